@@ -96,11 +96,11 @@ __global__ void __launch_bounds__(256) mm_tile_kernel(mm_dev a) {
     for (int i = 0; i < 4; i++) {
         const int m = m0 + ty * 4 + i;
         if (m >= row1) continue;
-        if (EPI == PIB_EPI_GLU_PAIR) {
+        if (pib_epi_pairs(EPI)) {
 #pragma unroll
             for (int j = 0; j < 4; j += 2) {
                 const int n = n0 + tx * 4 + j;
-                if (n + 1 < a.N) Y[(size_t) m * a.ldy + (n >> 1)] = pib_glu_pair<ROUND>(acc[i][j], acc[i][j + 1], a.e0);
+                if (n + 1 < a.N) Y[(size_t) m * a.ldy + (n >> 1)] = pib_glu_pair<EPI, ROUND>(acc[i][j], acc[i][j + 1], a.e0);
             }
             continue;
         }
@@ -135,7 +135,7 @@ template <> struct wvec<float> {
 // the rows [row0, row1) of problem z (at most B of them) against weight row n
 template <typename WT, bool ROUND, int EPI, int B>
 __device__ __forceinline__ void mv_rows_body(const mm_dev & a, bool xvec, int z, int n, int lane, int row0, int row1) {
-    constexpr int NR = EPI == PIB_EPI_GLU_PAIR ? 2 : 1;        // paired outputs: the warp walks the pair's two weight rows one after the other
+    constexpr int NR = pib_epi_pairs(EPI) ? 2 : 1;        // paired outputs: the warp walks the pair's two weight rows one after the other
     const float * X = a.X + (size_t) z * a.xz;
     float *       Y = a.Y + (size_t) z * a.yz;
     constexpr int V = wvec<WT>::N;
@@ -183,7 +183,7 @@ __device__ __forceinline__ void mv_rows_body(const mm_dev & a, bool xvec, int z,
 #pragma unroll
     for (int b = 0; b < B; b++) {
         if (lane == 0 && row0 + b < row1)
-            Y[(size_t) (row0 + b) * a.ldy + n] = EPI == PIB_EPI_GLU_PAIR ? pib_glu_pair<ROUND>(res[0][b], res[NR - 1][b], a.e0) : pib_epilogue<EPI, ROUND>(res[0][b], a.e0, a.e1);
+            Y[(size_t) (row0 + b) * a.ldy + n] = pib_epi_pairs(EPI) ? pib_glu_pair<EPI, ROUND>(res[0][b], res[NR - 1][b], a.e0) : pib_epilogue<EPI, ROUND>(res[0][b], a.e0, a.e1);
     }
 }
 
@@ -200,7 +200,7 @@ __global__ void __launch_bounds__(256) mv_rows_kernel(mm_dev a, bool xvec) {
     if (row1 - row0 > B) row1 = row0 + B;            // the host only picks this kernel when every z has at most B rows
     if (row0 >= row1) return;
     const int lane = threadIdx.x & 31, n = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-    if (n >= (EPI == PIB_EPI_GLU_PAIR ? a.N / 2 : a.N)) return;
+    if (n >= (pib_epi_pairs(EPI) ? a.N / 2 : a.N)) return;
     const int cnt = row1 - row0;
     if (B > 1 && a.zrange && cnt < B) {
         if (cnt == 1)                { mv_rows_body<WT, ROUND, EPI, 1>(a, xvec, z, n, lane, row0, row1); return; }
@@ -243,7 +243,7 @@ static int launch_mm(const pib_mm & a, const mm_dev & d, cudaStream_t st) {
     const bool vec_ok = a.ldw % V == 0 && a.wz % V == 0 && ((uintptr_t) a.W & 15) == 0;
     // few rows in all (with zrange: no problem z can own more than the total): a warp per weight row; problems without rows leave at once
     if (a.M <= MV_MAXB && vec_ok) {
-        dim3 grid((unsigned) (((EPI == PIB_EPI_GLU_PAIR ? a.N / 2 : a.N) + 7) / 8), 1, (unsigned) a.Z);
+        dim3 grid((unsigned) (((pib_epi_pairs(EPI) ? a.N / 2 : a.N) + 7) / 8), 1, (unsigned) a.Z);
         const bool xvec = a.ldx % 4 == 0 && a.xz % 4 == 0 && ((uintptr_t) a.X & 15) == 0;
         if (a.M == 1)      pib_launch(mv_rows_kernel<WT, ROUND, EPI, 1>, dim3(grid), dim3(256), (size_t) (0), st, d, xvec);
         else if (a.M == 2) pib_launch(mv_rows_kernel<WT, ROUND, EPI, 2>, dim3(grid), dim3(256), (size_t) (0), st, d, xvec);
@@ -277,9 +277,10 @@ int pib_dense_mm(const pib_mm & a, cudaStream_t st) {
         PIB_CHECK(cudaGetLastError());
         return PIB_OK;
     }
-    if (a.epi == PIB_EPI_GLU_PAIR && (a.N & 1)) { pib_set_error("dense matmul: paired outputs need an even number of weight rows"); return PIB_ERR_ARG; }
+    if (pib_epi_pairs(a.epi) && (a.N & 1)) { pib_set_error("dense matmul: paired outputs need an even number of weight rows"); return PIB_ERR_ARG; }
 #define MM_GO(WT, ROUND) (a.epi == PIB_EPI_RELU2 ? launch_mm<WT, ROUND, PIB_EPI_RELU2>(a, d, st) : a.epi == PIB_EPI_XIELU ? launch_mm<WT, ROUND, PIB_EPI_XIELU>(a, d, st) : \
                           a.epi == PIB_EPI_GLU_PAIR ? launch_mm<WT, ROUND, PIB_EPI_GLU_PAIR>(a, d, st) : \
+                          a.epi == PIB_EPI_GEGLU_PAIR ? launch_mm<WT, ROUND, PIB_EPI_GEGLU_PAIR>(a, d, st) : \
                                                     launch_mm<WT, ROUND, PIB_EPI_NONE>(a, d, st))
     if (a.wtype == PIB_TYPE_BF16) return MM_GO(__nv_bfloat16, true);
     if (a.wtype == PIB_TYPE_F32) return a.exact ? MM_GO(float, false) : MM_GO(float, true);

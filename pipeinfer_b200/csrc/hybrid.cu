@@ -28,6 +28,7 @@ struct pib_hybrid_ctx {
     float * x = nullptr, * h = nullptr, * y = nullptr, * proj = nullptr, * cq = nullptr, * q = nullptr, * qlat = nullptr, * lat = nullptr, * att = nullptr;
     float * rlog = nullptr, * wts = nullptr, * eup = nullptr, * edn = nullptr, * ysh = nullptr;
     float * h2 = nullptr, * cv = nullptr, * vfirst = nullptr, * mixes = nullptr;   // parallel layers: second norm (pre-norm layers: the stream's second buffer); convolved q | k | v; first mixing layer's values; token-shift mixes
+    float * rg = nullptr, * y2 = nullptr;       // gated frame: the residual gate's logits; the second branch's output
     float * cat = nullptr;                      // [stream ; embedding] rows of models whose layers are walked again
     int32_t * ids = nullptr, * perm = nullptr, * inv = nullptr, * counts = nullptr, * offs = nullptr;
     // batch bookkeeping: pinned staging ring + device copy
@@ -55,12 +56,14 @@ static const char * const HK_NAMES[] = { "cellmap", "embed_ln", "canon_conv", "m
                                          "embed_pair", "prenorm_shift", "loop_concat", "mm_loop_in", "mm_ssm_in", "ssm_conv", "mm_ssm_x", "mm_ssm_dt", "ssm_scan", "mm_ssm_o",
                                          "mm_dual_proj", "dual_prep", "decay_scan", "dual_gate", "mm_dual_o",
                                          "hyper_norm", "mm_mamba2_in", "mamba2_conv", "mamba2_prep", "mamba2_scan", "gated_group_norm", "mm_mamba2_o", "qkv_rope", "diff_combine",
-                                         "mm_gate_up" };
+                                         "mm_gate_up",
+                                         "gated_norm", "input_conv", "mm_res_gate", "mm_attn_mem_proj", "attn_mem_prep", "memory_scan", "attn_mem_gate", "mm_attn_mem_o" };
 enum { HK_CELLMAP, HK_EMBED, HK_CANON, HK_DQKV, HK_LPREP, HK_UQ, HK_ABSORB, HK_LATTN, HK_UV, HK_AO, HK_QFV, HK_GATES, HK_SCAN, HK_HO, HK_LNRES, HK_UP, HK_POLY, HK_DOWN,
        HK_ROUTER, HK_ROUTE, HK_SORT, HK_EUP, HK_EDOWN, HK_SUP, HK_SDOWN, HK_COMBINE, HK_FINAL, HK_HEAD, HK_SAMPLE, HK_LATTN_MM,
        HK_EMBSCALE, HK_NORM2, HK_QKV, HK_QKVCONV, HK_APREP, HK_KVATTN, HK_KVATTN_MM, HK_SHIFT, HK_RKVG, HK_DECAY, HK_DECAYACT, HK_WKVSCAN, HK_DPREP, HK_DSCAN, HK_GHNORM, HK_GLU,
        HK_PSUM, HK_EMBPAIR, HK_PRENORM, HK_CONCAT, HK_LOOPIN, HK_SSMIN, HK_SSMCONV, HK_SSMX, HK_SSMDT, HK_SSMSCAN, HK_SSMO, HK_DUALPROJ, HK_DUALPREP, HK_DECAYSCAN, HK_DUALGATE,
-       HK_DUALO, HK_HYPER, HK_M2IN, HK_M2CONV, HK_M2PREP, HK_M2SCAN, HK_GGNORM, HK_M2O, HK_QKVROPE, HK_DIFFCOMB, HK_GATEUP, HK_COUNT };
+       HK_DUALO, HK_HYPER, HK_M2IN, HK_M2CONV, HK_M2PREP, HK_M2SCAN, HK_GGNORM, HK_M2O, HK_QKVROPE, HK_DIFFCOMB, HK_GATEUP,
+       HK_GNORM, HK_INCONV, HK_RGATE, HK_AMPROJ, HK_AMPREP, HK_MEMSCAN, HK_AMGATE, HK_AMO, HK_COUNT };
 const char * pib_hybrid_kind_name(int k) { return k >= 0 && k < HK_COUNT ? HK_NAMES[k] : "?"; }
 
 // fetch and clear the records; returns the count (the stream is synchronised)
@@ -98,7 +101,7 @@ int pib_hybrid_ctx_init(pib_context * c, int n_slots) {
     x->rope.assign(hy->ropes.size(), nullptr);
     for (size_t i = 0; i < hy->ropes.size(); i++) {
         std::vector<float2> tab;
-        if (hy->ropes[i].factor > 0) pib_rope_table(tab, (int) c->n_ctx, hy->ropes[i]);                // scaled frequencies
+        if (hy->ropes[i].scaling != PIB_ROPE_PLAIN) pib_rope_table(tab, (int) c->n_ctx, hy->ropes[i]);                // scaled frequencies
         else rope_table_build(tab, (int) c->n_ctx, hy->ropes[i].dims, 4, hy->ropes[i].base, 1.0f);     // mode 4: every angle from its own power, in double
         HCK(cudaMalloc(&x->rope[i], std::max<size_t>(16, tab.size() * sizeof(float2))));
         HCK(cudaMemcpy(x->rope[i], tab.data(), tab.size() * sizeof(float2), cudaMemcpyHostToDevice));
@@ -148,9 +151,9 @@ static int grow_attn_mm(pib_context * c, size_t kw, size_t kx, int q_rows, int s
 static void free_scratch(pib_hybrid_ctx * x) {
     for (void * b : { (void *) x->x, (void *) x->h, (void *) x->y, (void *) x->proj, (void *) x->cq, (void *) x->q, (void *) x->qlat, (void *) x->lat, (void *) x->att,
                       (void *) x->rlog, (void *) x->wts, (void *) x->eup, (void *) x->edn, (void *) x->ysh, (void *) x->ids, (void *) x->perm, (void *) x->inv,
-                      (void *) x->counts, (void *) x->offs, (void *) x->h2, (void *) x->cv, (void *) x->vfirst, (void *) x->mixes, (void *) x->cat }) if (b) cudaFree(b);
+                      (void *) x->counts, (void *) x->offs, (void *) x->h2, (void *) x->cv, (void *) x->vfirst, (void *) x->mixes, (void *) x->cat, (void *) x->rg, (void *) x->y2 }) if (b) cudaFree(b);
     x->x = x->h = x->y = x->proj = x->cq = x->q = x->qlat = x->lat = x->att = x->rlog = x->wts = x->eup = x->edn = x->ysh = nullptr;
-    x->h2 = x->cv = x->vfirst = x->mixes = x->cat = nullptr;
+    x->h2 = x->cv = x->vfirst = x->mixes = x->cat = x->rg = x->y2 = nullptr;
     x->ids = x->perm = x->inv = x->counts = x->offs = nullptr;
     x->cap = 0;
 }
@@ -191,8 +194,9 @@ static int grow_scratch(pib_context * c, int T) {
                     fl(&x->qlat, (size_t) hy->w_lat) && fl(&x->lat, (size_t) hy->w_lat) && fl(&x->att, (size_t) hy->w_att) && fl(&x->rlog, (size_t) hy->w_router) &&
                     fl(&x->wts, (size_t) hy->w_pairs) && fl(&x->eup, (size_t) hy->w_eup) && fl(&x->edn, (size_t) hy->w_pairs * W) && fl(&x->ysh, hy->w_pairs ? W : 0) &&
                     in(&x->ids, n * hy->w_pairs) && in(&x->perm, n * hy->w_pairs) && in(&x->inv, n * hy->w_pairs) && in(&x->counts, (size_t) hy->w_router + 1) &&
-                    in(&x->offs, (size_t) hy->w_router + 2) && fl(&x->h2, hy->form == PIB_FORM_PARALLEL || hy->form == PIB_FORM_PRENORM ? W : 0) && fl(&x->cv, (size_t) hy->w_conv) &&
-                    fl(&x->vfirst, (size_t) hy->w_vfirst) && fl(&x->mixes, (size_t) hy->w_shift) && fl(&x->cat, (size_t) hy->w_cat);
+                    in(&x->offs, (size_t) hy->w_router + 2) && fl(&x->h2, hy->form == PIB_FORM_PARALLEL || hy->form == PIB_FORM_PRENORM || hy->form == PIB_FORM_GATED ? W : 0) && fl(&x->cv, (size_t) hy->w_conv) &&
+                    fl(&x->vfirst, (size_t) hy->w_vfirst) && fl(&x->mixes, (size_t) hy->w_shift) && fl(&x->cat, (size_t) hy->w_cat) &&
+                    fl(&x->rg, (size_t) hy->w_gate) && fl(&x->y2, (size_t) hy->w_y2);
     if (!ok) { cudaGetLastError(); free_scratch(x); pib_set_error("decode: out of memory for the work buffers of %d tokens", T); return PIB_ERR_NOMEM; }
     x->cap = (int) n;
     return PIB_OK;
@@ -232,9 +236,9 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
     auto wbytes = [](const pib_weight * w) { return (double) w->bytes; };
     auto mmfl = [&](const pib_weight * w) { return 2.0 * Td * (double) w->N * (double) w->K; };
     auto mmby = [&](const pib_weight * w) { return (double) w->bytes + 4.0 * Td * ((double) w->N + (double) w->K); };
-    auto key_pairs = [&](int window, int mask = PIB_MASK_WINDOW) {
+    auto key_pairs = [&](int window, int mask = PIB_MASK_WINDOW, int keep = 0) {
         double n = 0;
-        for (int i = 0; i < T; i++) n += mask == PIB_MASK_CHUNK ? B_pos_host[i] % window + 1 : std::min(B_pos_host[i] + 1, window);
+        for (int i = 0; i < T; i++) n += mask == PIB_MASK_CHUNK ? B_pos_host[i] % window + 1 : std::min<int64_t>(B_pos_host[i] + 1, (int64_t) window + keep);
         return n;
     };
     auto mm = [&](const pib_weight * w, const float * X, int ldx, float * Y, int ldy, int epi, float e0 = 0.f, float e1 = 0.f) {
@@ -299,7 +303,7 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
     // the attention of cached key / value heads over `q`: per-token kernel, or the matmul form for long portions in served mode
     auto kv_attend = [&](const pib_hlayer & L, float * cache, int row, float * out) -> int {
         const int H = L.heads * L.maps, G = L.kv_heads * L.maps, D = L.dim, V = L.vdim;      // query rows and key heads: one per map
-        const double keys = key_pairs(L.window, L.mask);
+        const double keys = key_pairs(L.window, L.mask, L.keep);
         const bool mm_ok = !exact && D % 8 == 0 && D >= 16 && V >= 16 && attn_mm_enabled();
         bool any_mm = false, any_simt = false;
         for (const pib_hseg & g : segs) { if (mm_ok && g.len >= MM_ATTN_MIN_LEN) any_mm = true; else any_simt = true; }
@@ -311,11 +315,13 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
             const int nb = (g.len + MM_ATTN_BLOCK - 1) / MM_ATTN_BLOCK, per = (g.len + nb - 1) / nb;      // blocks of equal size: none is left with a handful of rows
             for (int o = 0; o < g.len; o += per) {
                 const int nq = std::min(per, g.len - o), p0 = B_pos_host[g.start + o];
-                const int j0 = L.mask == PIB_MASK_CHUNK ? p0 - p0 % L.window : std::max(0, p0 - L.window + 1), NK = p0 + nq - j0;
+                int j0 = L.mask == PIB_MASK_CHUNK ? p0 - p0 % L.window : std::max(0, p0 - L.window + 1), n_front = 0;
+                if (L.keep > 0) { if (j0 <= L.keep) j0 = 0; else n_front = L.keep; }        // kept first positions: columns of their own in front of the window's
+                const int NK = n_front + p0 + nq - j0;
                 if ((rc = grow_attn_mm(c, (size_t) G * std::max(D, V), (size_t) 3 * G * D + V, nq * H, nq * H, NK)) != PIB_OK) return rc;
                 RC(HK_KVATTN_MM, 2.0 * nq * H * (double) NK * (D + 2.0 * V), 2.0 * NK * G * (D + 2.0 * V) + 8.0 * nq * H * (D + V) + 8.0 * nq * H * (double) NK,
-                   pib_kv_attention_mm(x->q, L, B, cache, row, x->cellmap + (size_t) g.slot * c->n_ctx, g.start + o, nq, j0, NK, x->am_kb, x->am_vt, x->am_q, x->am_s, x->am_p,
-                                       out, st));
+                   pib_kv_attention_mm(x->q, L, B, cache, row, x->cellmap + (size_t) g.slot * c->n_ctx, g.start + o, nq, j0, n_front, NK, x->am_kb, x->am_vt, x->am_q, x->am_s,
+                                       x->am_p, out, st));
                 nk += 5;
             }
         }
@@ -449,6 +455,27 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
         RC(HK_AO, mmfl(L.wo), mmby(L.wo), mm(L.wo, x->att, H * V, x->y, W, PIB_EPI_NONE));
         return PIB_OK;
     };
+    // attention beside a matrix memory: every projection in one matmul; norms, rotation and cache write beside the memory's gates in one kernel; windowed
+    // attention with kept first tokens; the memory's recurrence; gates and the memory's norms in one kernel; an output matmul per branch (x->y, x->y2),
+    // whose norms and mean ride on the frame's kernel
+    auto mixer_attn_mem = [&](const pib_hlayer & L, const float * hin) -> int {
+        const int H = L.heads, G = L.kv_heads, D = L.dim, V = L.vdim, H2 = L.heads2, D2 = L.dim2, V2 = L.vdim2, row = hy->cache_row[L.cache_id];
+        const int ldp = ((int) L.qkv->N + 3) & ~3, q2 = (H + G) * D + G * V, k2 = q2 + H2 * D2, v2 = k2 + H2 * D2, og = v2 + H2 * V2, hg = og + H2 * V2, gi = hg + H, gf = gi + H2;
+        const int mem_off = (H * V + 3) & ~3, ldo = (mem_off + H2 * V2 + 3) & ~3;
+        float * cache = x->cache[L.cache_id];
+        RC(HK_AMPROJ, mmfl(L.qkv), mmby(L.qkv), mm(L.qkv, hin, W, x->proj, ldp, PIB_EPI_NONE));
+        RC(HK_AMPREP, 0, 4.0 * Td * (2.0 * q2 + 6.0 * H2), pib_attn_mem_prep(x->proj, ldp, gi, gf, L, eps, B, x->rope[L.rope_id], x->q, cache, row, x->state, hy->state_floats, x->cq, st));
+        if ((rc = kv_attend(L, cache, row, x->lat)) != PIB_OK) return rc;
+        int parts = 0, per = 0;
+        if ((rc = split_plan(H2, D2, V2 + 1, parts, per)) != PIB_OK) return rc;
+        RC(HK_MEMSCAN, 5.0 * Td * H2 * D2 * (V2 + 1.0), 4.0 * Td * H2 * (2.0 * D2 + 2.0 * V2 + 3.0),
+           pib_memory_scan(x->proj, ldp, q2, k2, v2, x->cq, L, B, x->state, hy->state_floats, x->cv, st, x->split_buf, parts, per));
+        nk += parts ? 4 : 0;
+        RC(HK_AMGATE, 0, 4.0 * Td * (2.0 * H * V + 3.0 * H2 * V2 + 2.0 * H2 + H), pib_attn_mem_gate(x->lat, x->cv, x->cq, x->proj, ldp, hg, og, L, eps, T, x->att, ldo, mem_off, st));
+        RC(HK_AMO, mmfl(L.wo), mmby(L.wo), mm(L.wo, x->att, ldo, x->y, W, PIB_EPI_NONE));
+        RC(HK_AMO, mmfl(L.wo2), mmby(L.wo2), mm(L.wo2, x->att + mem_off, ldo, x->y2, W, PIB_EPI_NONE));
+        return PIB_OK;
+    };
     auto run_mixer = [&](const pib_hlayer & L, const float * hin) -> int {
         switch (L.mixer) {
             case PIB_MIXER_LATENT: return mixer_latent(L, hin);
@@ -460,6 +487,7 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
             case PIB_MIXER_DUAL:   return mixer_dual(L, hin);
             case PIB_MIXER_MAMBA2: return mixer_mamba2(L, hin);
             case PIB_MIXER_DIFF:   return mixer_diff(L, hin);
+            case PIB_MIXER_ATTN_MEM: return mixer_attn_mem(L, hin);
         }
         pib_set_error("decode: mixer %d", L.mixer);
         return PIB_ERR_UNSUPP;
@@ -499,7 +527,7 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
 
     RC(HK_CELLMAP, 0, 16.0 * Td, pib_cellmap_set(x->cellmap, (int) c->n_ctx, B, st));
     if (hy->form == PIB_FORM_HYPER)        RC(HK_EMBSCALE, 0, (2.0 + 4.0 * hy->streams) * Td * Wd, pib_embed_scale(m->tok_embd, B.tok, hy->embd_scale, T, W, x->x, st, hy->streams));
-    else if (hy->form == PIB_FORM_PARALLEL) RC(HK_EMBSCALE, 0, 6.0 * Td * Wd, pib_embed_scale(m->tok_embd, B.tok, hy->embd_scale, T, W, x->x, st));
+    else if (hy->form == PIB_FORM_PARALLEL || hy->form == PIB_FORM_GATED) RC(HK_EMBSCALE, 0, 6.0 * Td * Wd, pib_embed_scale(m->tok_embd, B.tok, hy->embd_scale, T, W, x->x, st));
     else if (hy->form == PIB_FORM_PRENORM) RC(HK_EMBPAIR, 0, (hy->loops ? 10.0 : 6.0) * Td * Wd, pib_embed_pair(m->tok_embd, B.tok, T, W, x->x, hy->loops ? x->cat : nullptr, st));
     else                                   RC(HK_EMBED, 0, 6.0 * Td * Wd, pib_embed_ln(m->tok_embd, B.tok, hy->embd_norm, eps, T, W, x->x, st));
     // pre-norm form: the stream is (have_x ? cur : 0) + pend_y + pend_b; the sum is formed by the next norm's kernel, which leaves it in the
@@ -515,10 +543,37 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
         if (upd) { std::swap(cur, other); have_x = true; pend_y = pend_b = nullptr; }
         return PIB_OK;
     };
+    // gated frame: what the sublayer before left is added by the kernel that norms the stream for the next one; in batches of single tokens that
+    // kernel also does the next input convolution.  x->h: the normed stream, x->h2: with its convolution added
+    pib_sublayer_out left;
+    auto gated = [&](const float * w, const float * conv, size_t tail_off) -> int {
+        const bool fused = conv && T == B.S;
+        RC(HK_GNORM, 0, 4.0 * Td * Wd * ((left.ya ? (left.wa ? 5.0 : 4.0) : 1.0) + (w ? 1.0 : 0.0) + (fused ? 2.0 * hy->taps : 0.0)),
+           pib_gated_norm(x->x, left, w, eps, W, w ? x->h : nullptr, fused ? conv : nullptr, hy->taps, B, x->state, hy->state_floats, tail_off, x->h2, st));
+        left = pib_sublayer_out();
+        if (conv && !fused) {
+            RC(HK_INCONV, 2.0 * Td * Wd * hy->taps, 8.0 * Td * Wd, pib_canon_conv(x->h, conv, hy->taps, B, x->state, hy->state_floats, tail_off, W, x->h2, st));
+            nk += hy->taps > 1;
+        }
+        return PIB_OK;
+    };
     for (int il = 0; il < m->n_layer; il++) {
         const pib_hlayer & L = hy->layers[il];
         int lds = 0;
-        if (hy->form == PIB_FORM_HYPER) {
+        if (hy->form == PIB_FORM_GATED) {
+            if ((rc = gated(L.norm1, L.canon, L.tail_off)) != PIB_OK) return rc;
+            RC(HK_RGATE, mmfl(L.rg1), mmby(L.rg1), mm(L.rg1, x->h, W, x->rg, W, PIB_EPI_NONE));
+            if ((rc = run_mixer(L, x->h2)) != PIB_OK) return rc;
+            left.ya = x->y; left.gl = x->rg; left.gb = L.rg1_b;
+            if (L.wo2) { left.wa = L.out_a; left.yb = x->y2; left.wb = L.out_b; left.mix = L.mix_a; }
+            if (L.mlp == PIB_MLP_GEGLU) {
+                if ((rc = gated(L.norm2, L.canon2, L.tail2_off)) != PIB_OK) return rc;
+                RC(HK_RGATE, mmfl(L.rg2), mmby(L.rg2), mm(L.rg2, x->h, W, x->rg, W, PIB_EPI_NONE));
+                RC(HK_GATEUP, mmfl(L.up), wbytes(L.up) + 4.0 * Td * (Wd + L.ff), mm(L.up, x->h2, W, x->proj, L.ff, PIB_EPI_GEGLU_PAIR));
+                RC(HK_DOWN, mmfl(L.down), mmby(L.down), mm(L.down, x->proj, L.ff, x->y, W, PIB_EPI_NONE));
+                left.ya = x->y; left.gl = x->rg; left.gb = L.rg2_b;
+            } else if (L.mlp != PIB_MLP_NONE) { pib_set_error("decode: feed-forward %d in a gated layer", L.mlp); return PIB_ERR_UNSUPP; }
+        } else if (hy->form == PIB_FORM_HYPER) {
             // the write of the sublayer before rides on the kernel that reads and norms the streams for the next one
             const int Sn = hy->streams;
             const double hby = (8.0 * Sn + 8.0) * Td * Wd;
@@ -575,6 +630,7 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
                 RC(HK_LNRES, 0, 12.0 * Td * Wd, pib_layer_norm(x->y, L.norm2, eps, T, W, x->x, 1, st));
             }
         }
+        if (getenv("PIB_HYBRID_DUMP") && hy->form == PIB_FORM_GATED && left.ya) { if ((rc = gated(nullptr, nullptr, 0)) != PIB_OK) return rc; }
         if (getenv("PIB_HYBRID_DUMP") && hy->form == PIB_FORM_HYPER) {   // debugging: the sum of the streams after every layer, one file per layer and decode
             if (pend_y) { RC(HK_HYPER, 0, 0, pib_hyper_norm(x->x, hy->streams, pend_y, pend_b, nullptr, nullptr, nullptr, eps, T, W, nullptr, st)); pend_y = pend_b = nullptr; }
             std::vector<float> xb((size_t) T * hy->streams * W), hb((size_t) T * W, 0.f);
@@ -596,7 +652,8 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
             if (FILE * f = fopen(path, "wb")) { fwrite(hb.data(), 4, hb.size(), f); fclose(f); }
         }
     }
-    if (hy->form == PIB_FORM_HYPER)         RC(HK_FINAL, 0, (4.0 * hy->streams + 8.0) * Td * Wd, pib_hyper_norm(x->x, hy->streams, pend_y, pend_b, nullptr, m->output_norm, hy->final_b, eps, T, W, x->h, st));
+    if (hy->form == PIB_FORM_GATED)         { if ((rc = gated(m->output_norm, nullptr, 0)) != PIB_OK) return rc; }
+    else if (hy->form == PIB_FORM_HYPER)    RC(HK_FINAL, 0, (4.0 * hy->streams + 8.0) * Td * Wd, pib_hyper_norm(x->x, hy->streams, pend_y, pend_b, nullptr, m->output_norm, hy->final_b, eps, T, W, x->h, st));
     else if (hy->form == PIB_FORM_PRENORM)  { if ((rc = prenorm(hy->final_g, nullptr, 0, false)) != PIB_OK) return rc; }
     else if (hy->form == PIB_FORM_PARALLEL) RC(HK_FINAL, 0, 8.0 * Td * Wd, pib_rms_norm2(x->x, m->output_norm, nullptr, eps, hy->logit_scale, T, W, x->h, nullptr, st));
     else                                    RC(HK_FINAL, 0, 8.0 * Td * Wd, pib_layer_norm(x->x, m->output_norm, eps, T, W, x->h, 0, st));

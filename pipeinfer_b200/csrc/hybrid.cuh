@@ -17,8 +17,13 @@
 //                  grouped RMS norm); differential attention (two softmax maps per head over the same values, subtracted, per-head unit
 //                  RMS; biases, partial rotation with YaRN-scaled frequencies); latent attention without a query latent or sink, rotated
 //                  in adjacent pairs
-//   more feed-forwards: dense clamped gated (the experts' activation of the mixtures above as one dense block)
-// Designs built from these parts: "Rapisun", "Fabivik", "Lulenex", "Putazen".  The parts take their sizes and constants as parameters so that another
+//   more feed-forwards: dense clamped gated (the experts' activation of the mixtures above as one dense block); dense gated with a gelu
+//   one more frame: sequential pre-norm with an input convolution in front of BOTH sublayers and a sigmoid gate per channel on what a
+//                  sublayer adds to the stream
+//   one more mixer: windowed softmax attention that also keeps the sequence's first tokens (one RMS norm over all query rows and one over
+//                  all key rows, capped scores, a sink of score 0, a gate per head) beside a matrix memory with exponential gates (mLSTM);
+//                  each branch has an output matrix of its own, their outputs are RMS-normed over the width and averaged
+// Designs built from these parts: "Rapisun", "Fabivik", "Lulenex", "Putazen", "Bobunex".  The parts take their sizes and constants as parameters so that another
 // layer-list design can name them too.
 //
 // What such a model adds to the runtime, beside what llama / falcon graphs use:
@@ -33,21 +38,25 @@
 #include "engine.cuh"
 
 enum { PIB_MIXER_LATENT = 1, PIB_MIXER_HGRN2 = 2, PIB_MIXER_SWA = 3, PIB_MIXER_WKV = 4, PIB_MIXER_DELTA = 5, PIB_MIXER_SSM = 6, PIB_MIXER_DUAL = 7,
-       PIB_MIXER_MAMBA2 = 8, PIB_MIXER_DIFF = 9 };
-enum { PIB_MLP_NONE = 0, PIB_MLP_POLYNORM = 1, PIB_MLP_MOE = 2, PIB_MLP_XIELU = 3, PIB_MLP_GLU = 4 };
+       PIB_MIXER_MAMBA2 = 8, PIB_MIXER_DIFF = 9, PIB_MIXER_ATTN_MEM = 10 };
+enum { PIB_MLP_NONE = 0, PIB_MLP_POLYNORM = 1, PIB_MLP_MOE = 2, PIB_MLP_XIELU = 3, PIB_MLP_GLU = 4, PIB_MLP_GEGLU = 5 };
 // which earlier positions j a token at p may read: the last `window` ones (p - window < j <= p), or those of its own chunk (j / window == p / window)
 enum { PIB_MASK_WINDOW = 0, PIB_MASK_CHUNK = 1 };
 // what a matmul does to an output on its way out: nothing; max(y, 0)^2; xIELU (y > 0: e0 y^2 + y/2, else e1 (exp(y) - 1 - y) + y/2)
 //   PIB_EPI_GLU_PAIR: outputs come in pairs (2 i: gate g, 2 i + 1: linear part u; the weight rows are stored interleaved); output i of a row with pitch ldy is
 //   a sigmoid(1.702 a) (b + 1), a = min(g, e0), b = clamp(u, -e0, e0).  N counts the weight rows (twice the outputs).
-enum { PIB_EPI_NONE = 0, PIB_EPI_RELU2 = 1, PIB_EPI_XIELU = 2, PIB_EPI_GLU_PAIR = 3 };
+//   PIB_EPI_GEGLU_PAIR: pairs as above; output i is gelu(g) u, gelu in its tanh form.
+enum { PIB_EPI_NONE = 0, PIB_EPI_RELU2 = 1, PIB_EPI_XIELU = 2, PIB_EPI_GLU_PAIR = 3, PIB_EPI_GEGLU_PAIR = 4 };
 // layer forms: x += LN(mixer(conv(x))), x += LN(ff(x))   |   x += mixer(N1(x)) + ff(N2(x)), N = RMS norm with weight (1 + w)
 //              x += mixer(shift(N(x))), x += ff(N(x)), N = RMS norm times one number, shift(h)_t = h_t + (h_{t-1} - h_t) * mu
 //              hyper-connections over S streams X_s: u = sum_s in_s X_s, y = sublayer(LN(u)) (LayerNorm with weight and bias),
 //              X_t <- sum_s mix[s][t] X_s + out_t y, for the mixer and then for the feed-forward; the model's output reads sum_s X_s
-enum { PIB_FORM_POSTNORM = 0, PIB_FORM_PARALLEL = 1, PIB_FORM_PRENORM = 2, PIB_FORM_HYPER = 3 };
+//              gated: h = N(x), x += sublayer(h + conv(h)) * sigmoid(R h + r), for the mixer and then for the feed-forward
+enum { PIB_FORM_POSTNORM = 0, PIB_FORM_PARALLEL = 1, PIB_FORM_PRENORM = 2, PIB_FORM_HYPER = 3, PIB_FORM_GATED = 4 };
 // how a rotation pairs coordinates: (i, i + dims / 2) or (2 i, 2 i + 1)
 enum { PIB_PAIR_HALF = 0, PIB_PAIR_ADJACENT = 1 };
+// how a rotation's frequencies are scaled (see pib_hybrid::Rope)
+enum { PIB_ROPE_PLAIN = 0, PIB_ROPE_YARN = 1, PIB_ROPE_BANDS = 2 };
 // mixture of experts: how the router's logits become weights, where a weight multiplies, what an expert computes
 enum { PIB_ROUTE_SOFTMAX_RENORM = 0, PIB_ROUTE_SIGMOID = 1 };
 enum { PIB_EXPERT_RELU2 = 0, PIB_EXPERT_GLU_CLAMP = 1 };
@@ -122,6 +131,23 @@ struct pib_hlayer {
     int   maps = 1;                                   // attention rows per head that share its values (1: ordinary attention)
     float diff_lambda = 0.f, diff_out = 1.f;
     int   rot_pairs = PIB_PAIR_HALF;
+    // ---- gated frame (PIB_FORM_GATED): residual gates' matrices and biases, the feed-forward's input convolution (the mixer's: canon, tail_off) ----
+    pib_weight * rg1 = nullptr, * rg2 = nullptr;      // [width][width]
+    float * rg1_b = nullptr, * rg2_b = nullptr, * canon2 = nullptr;
+    size_t  tail2_off = 0;
+    // ---- attention beside a matrix memory (PIB_MIXER_ATTN_MEM) ----
+    // attention: heads / kv_heads / dim / vdim / rot_dims / scale / window; q_norm [heads*dim] and k_norm [kv_heads*dim] are weights of ONE norm over all
+    // rows each; sink: zeros.  memory: heads2 x (dim2 -> vdim2), per head S [dim2][vdim2 + 1], whose last column is the normaliser n (its
+    // value is always 1), and the running maximum m: S <- e^(f + m - m') S + e^(i - m') k [v | 1]^T, m' = max(f + m, i).
+    // qkv rows: q (heads*dim) | k (kv_heads*dim) | v (kv_heads*vdim) | q2 (heads2*dim2) | k2 (heads2*dim2) | v2 (heads2*vdim2) | output gates (heads2*vdim2) |
+    // head gates (heads) | input gates (heads2) | forget gates (heads2); wo [width][heads*vdim], wo2 [width][heads2*vdim2]
+    int   keep = 0;                                   // the first `keep` positions are read from everywhere
+    float softcap = 0.f;                              // score <- softcap tanh(score / softcap) (0: none)
+    float gate_cap = 0.f;                             // the memory's gate logits, the same way
+    pib_weight * wo2 = nullptr;
+    float * i_bias = nullptr;                         // [heads2]  (forget gates: f_bias)
+    float * out_a = nullptr, * out_b = nullptr;       // [width]: weights of the branches' output norms
+    size_t  max_off = 0;                              // floats into a slot's state: m [heads2]   (state_off: the matrices)
     // ---- feed-forward ----
     int   ff = 0;
     pib_weight * up = nullptr, * down = nullptr;
@@ -156,12 +182,18 @@ struct pib_hybrid {
     // context; pairs below a = max(floor(d(fast)), 0) keep their frequency, pairs above b = min(ceil(d(slow)), dims - 1) have it divided by
     // the factor, and between them the blend r_i = clamp((i - a) / max(b - a, 0.001), 0, 1) gives f_i (r_i / factor + 1 - r_i).  The table's
     // cos and sin carry the magnitude 0.1 ln(factor) + 1.
-    struct Rope { float base; int dims; double factor = 0, original = 0, fast = 0, slow = 0; };
+    // Bands (Llama 3.1): waves that turn more than `fast` times over the original context keep their frequency, those that turn less than
+    // `slow` times have it divided by the factor, and a wave that turns n times in between gets f ((1 - s) / factor + s), s = (n - slow) / (fast - slow).
+    struct Rope {
+        float base; int dims; double factor = 0, original = 0, fast = 0, slow = 0; int scaling = PIB_ROPE_PLAIN;
+        bool operator==(const Rope & o) const { return base == o.base && dims == o.dims && factor == o.factor && original == o.original && fast == o.fast && slow == o.slow && scaling == o.scaling; }
+    };
     std::vector<Rope> ropes;
     // widest per-token scratch rows over all layers
     int     w_proj = 0, w_cq = 0, w_q = 0, w_lat = 0, w_att = 0, w_pairs = 0, w_eup = 0, w_router = 0;
     int     w_conv = 0, w_vfirst = 0, w_shift = 0;    // convolved q | k | v rows, the first mixing layer's values, the five token-shift mixes
     int     w_cat = 0;                                // [stream ; embedding] rows of a walk's opening
+    int     w_gate = 0, w_y2 = 0;                     // residual gates' logits, a second branch's output
 };
 
 struct pib_hybrid_ctx;
@@ -202,7 +234,12 @@ template <int EPI, bool FAST> __device__ __forceinline__ float pib_epilogue(floa
     }
     return v;
 }
-template <bool FAST> __device__ __forceinline__ float pib_glu_pair(float g, float u, float limit) {
+__host__ __device__ constexpr bool pib_epi_pairs(int epi) { return epi == PIB_EPI_GLU_PAIR || epi == PIB_EPI_GEGLU_PAIR; }
+template <int EPI, bool FAST> __device__ __forceinline__ float pib_glu_pair(float g, float u, float limit) {
+    if (EPI == PIB_EPI_GEGLU_PAIR) {      // 0.5 g (1 + tanh z) = g sigmoid(2 z)
+        const float z = 0.7978845608028654f * fmaf(0.044715f * g * g, g, g);
+        return (FAST ? g / (1.0f + __expf(-2.0f * z)) : 0.5f * g * (1.0f + tanhf(z))) * u;
+    }
     const float a = fminf(g, limit), b = fminf(fmaxf(u, -limit), limit);
     return a / (1.0f + (FAST ? __expf(-1.702f * a) : expf(-1.702f * a))) * (b + 1.0f);
 }
@@ -234,7 +271,7 @@ int pib_latent_attention(const float * q, int ldq, const float * qlat, const pib
 int pib_latent_attention_mm(const float * q, int ldq, const float * qlat, const pib_hlayer & L, const pib_hbatch & b, const float2 * rope, const float * cache, int cache_row,
                             const int32_t * map, int t0, int nq, int j0, int NK, void * Kb, void * Vt, float * Qc, float * S, void * P, float * ctx, cudaStream_t st);
 int pib_window_softmax(float * S, void * P, int NKp, int NK, int j0, int window, const int32_t * pos, int t0, int n_rows, int rows_per_z, int rep, const float * sink,
-                       cudaStream_t st, int mask = PIB_MASK_WINDOW);
+                       cudaStream_t st, int mask = PIB_MASK_WINDOW, int keep = 0, int n_front = 0, float softcap = 0.f);
 int pib_hgrn2_gates(float * qfv, int ld, const float * f_bias, const float * lower, int T, int HD, cudaStream_t st);
 int pib_hgrn2_scan(const float * qfv, int ld, const pib_hlayer & L, const pib_hbatch & b, float * state, size_t state_stride, const float * onorm, float eps,
                    float * out, cudaStream_t st);
@@ -250,7 +287,7 @@ int pib_rms_norm2(const float * x, const float * w1, const float * w2, float eps
 int pib_swa_prep(const float * cv, int ldc, const pib_hlayer & L, float eps, const pib_hbatch & b, float * q, float * cache, int cache_row, float * vfirst, cudaStream_t st);
 int pib_kv_attention(const float * q, const pib_hlayer & L, const pib_hbatch & b, const float * cache, int cache_row, const int32_t * cellmap, int n_ctx, float * out,
                      const int32_t * skip, cudaStream_t st);
-int pib_kv_attention_mm(const float * q, const pib_hlayer & L, const pib_hbatch & b, const float * cache, int cache_row, const int32_t * map, int t0, int nq, int j0, int NK,
+int pib_kv_attention_mm(const float * q, const pib_hlayer & L, const pib_hbatch & b, const float * cache, int cache_row, const int32_t * map, int t0, int nq, int j0, int n_front, int NK,
                         void * Kb, void * Vt, float * Qc, float * S, void * P, float * out, cudaStream_t st);
 int pib_token_shift(const float * h, const float * mu, int n_mix, const pib_hbatch & b, float * state, size_t state_stride, size_t shift_off, int W, float * mixes, cudaStream_t st);
 int pib_rows_act(float * z, int ld, int n, int T, int op, const float * bias, cudaStream_t st);           // op 0: tanh; 1: exp(-exp(z + bias))
@@ -281,4 +318,18 @@ int pib_hyper_norm(float * X, int S, const float * y, const float * hc_prev, con
 int pib_mamba2_prep(const float * proj, int ldp, int dt_off, const pib_hlayer & L, int T, float * dg, cudaStream_t st);
 int pib_gated_group_norm(float * y, const float * z, int ldz, int T, int C, int groups, const float * w, float eps, cudaStream_t st);
 int pib_qkv_rope(const float * proj, int ldp, const pib_hlayer & L, const pib_hbatch & b, const float2 * rope, float * q, float * cache, int cache_row, cudaStream_t st);
+// gated_kernels.cu
+struct pib_sublayer_out {            // what the sublayer before left for the stream: y = ya, or mix (RMS(ya) wa + RMS(yb) wb); x += y sigmoid(gl + gb)
+    const float * ya = nullptr, * wa = nullptr, * yb = nullptr, * wb = nullptr;
+    float mix = 1.f;
+    const float * gl = nullptr, * gb = nullptr;
+};
+int pib_gated_norm(float * x, const pib_sublayer_out & o, const float * w, float eps, int W, float * h, const float * conv, int taps, const pib_hbatch & b, float * state,
+                   size_t state_stride, size_t tail_off, float * hc, cudaStream_t st);
+int pib_attn_mem_prep(const float * proj, int ldp, int i_off, int f_off, const pib_hlayer & L, float eps, const pib_hbatch & b, const float2 * rope, float * q, float * cache,
+                      int cache_row, float * state, size_t state_stride, float * dg, cudaStream_t st);
+int pib_attn_mem_gate(const float * a, const float * mem, const float * dg, const float * proj, int ldp, int hg_off, int og_off, const pib_hlayer & L, float eps, int T, float * out,
+                      int ldo, int mem_off, cudaStream_t st);
+int pib_memory_scan(const float * proj, int ldp, int q_off, int k_off, int v_off, float * dg, const pib_hlayer & L, const pib_hbatch & b, float * state, size_t state_stride, float * out,
+                    cudaStream_t st, float * split_buf = nullptr, int parts = 0, int per = 0);   // mixer_kernels.cu
 int pib_diff_combine(const float * a, const pib_hlayer & L, float eps, int T, float * out, cudaStream_t st);

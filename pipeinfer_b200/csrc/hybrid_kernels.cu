@@ -346,20 +346,28 @@ __global__ void __launch_bounds__(128) lat_qcat_kernel(const float * __restrict_
     for (int i = threadIdx.x; i < rot_dim; i += blockDim.x) out[R + i] = rot_coord(qr, i, rot_dims, pairs, cs) * scale;
 }
 // one score row per (token, head), in place: keys outside [p - window + 1, p] (chunk mask: outside [p - p % window, p]) and the pad get weight 0, the sink (optional) one share of
-// the denominator.  Rows come in groups of rows_per_z (one group per problem of the score matmul), inside a group `rep` heads per token:
+// the denominator.  The first `keep` positions are read from everywhere: columns [0, n_front) are positions 0 .. n_front - 1 (n_front is 0 or keep), the columns
+// behind them positions j0, j0 + 1, ... (n_front 0: then j0 is 0 or nothing is kept).  softcap > 0: a score becomes softcap tanh(score / softcap) first.  Rows come in groups of rows_per_z (one group per problem of the score matmul), inside a group `rep` heads per token:
 // token t0 + (row % rows_per_z) / rep, head (row / rows_per_z) * rep + (row % rows_per_z) % rep.
 __global__ void __launch_bounds__(256) lat_softmax_kernel(float * __restrict__ S, __nv_bfloat16 * __restrict__ P, int NKp, int NK, int j0, int window,
-                                                          const int32_t * __restrict__ pos, int t0, int rows_per_z, int rep, const float * __restrict__ sink, int mask) {
+                                                          const int32_t * __restrict__ pos, int t0, int rows_per_z, int rep, const float * __restrict__ sink, int mask, int keep, int n_front,
+                                                          float softcap) {
     pib_pdl_wait();
     pib_pdl_trigger();
     __shared__ float red[32];
     const int row = blockIdx.x, rz = row % rows_per_z, t = t0 + rz / rep, h = (row / rows_per_z) * rep + rz % rep, p = pos[t];
     float *   s = S + (size_t) row * NKp;
     __nv_bfloat16 * pw = P + (size_t) row * 2 * NKp;   // [weights' bfloat16 part | what the rounding left]: the value matmul sees both, so the weights keep fp32 accuracy
-    const int lo = (mask == PIB_MASK_CHUNK ? p - p % window : max(0, p - window + 1)) - j0, hi = p - j0;            // valid columns [lo, hi]
+    const int lo = (mask == PIB_MASK_CHUNK ? p - p % window : max(0, p - window + 1)) - j0 + n_front, hi = p - j0 + n_front;            // valid columns [lo, hi] ...
+    const int ka = n_front > 0 ? n_front : min(keep, lo);                                                                              // ... and [0, ka)
     const float sk = sink ? sink[h] : -INFINITY;
     float m = sk;
-    for (int j = lo + (int) threadIdx.x; j <= hi; j += blockDim.x) m = fmaxf(m, s[j]);
+    for (int e = threadIdx.x; e < ka + hi - lo + 1; e += blockDim.x) {
+        const int j = e < ka ? e : lo + e - ka;
+        float v = s[j];
+        if (softcap > 0.f) { v = softcap * tanhf(v / softcap); s[j] = v; }
+        m = fmaxf(m, v);
+    }
     m = warp_max(m);
     __syncthreads();
     if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = m;
@@ -367,7 +375,7 @@ __global__ void __launch_bounds__(256) lat_softmax_kernel(float * __restrict__ S
     for (int i = 0; i < (int) (blockDim.x >> 5); i++) m = fmaxf(m, red[i]);
     float sum = 0.f;
     for (int j = threadIdx.x; j < NKp; j += blockDim.x) {
-        const float e = (j >= lo && j <= hi) ? expf(s[j] - m) : 0.f;
+        const float e = ((j >= lo && j <= hi) || j < ka) ? expf(s[j] - m) : 0.f;
         s[j] = e;
         sum += e;
     }
@@ -381,8 +389,8 @@ __global__ void __launch_bounds__(256) lat_softmax_kernel(float * __restrict__ S
     (void) NK; (void) hi;
 }
 int pib_window_softmax(float * S, void * P, int NKp, int NK, int j0, int window, const int32_t * pos, int t0, int n_rows, int rows_per_z, int rep, const float * sink,
-                       cudaStream_t st, int mask) {
-    pib_launch(lat_softmax_kernel, dim3(n_rows), dim3(256), (size_t) (0), st, S, (__nv_bfloat16 *) P, NKp, NK, j0, window, pos, t0, rows_per_z, rep, sink, mask);
+                       cudaStream_t st, int mask, int keep, int n_front, float softcap) {
+    pib_launch(lat_softmax_kernel, dim3(n_rows), dim3(256), (size_t) (0), st, S, (__nv_bfloat16 *) P, NKp, NK, j0, window, pos, t0, rows_per_z, rep, sink, mask, keep, n_front, softcap);
     CKL();
     return PIB_OK;
 }

@@ -107,11 +107,11 @@ int pib_swa_prep(const float * cv, int ldc, const pib_hlayer & L, float eps, con
 }
 
 // grid (token, head group); a block holds HPB query heads x KS key shares, one warp each.  A warp walks its share of the window
-// [max(0, p - window + 1), p] (chunk mask: of the token's chunk [p - p % window, p]) through the slot's position -> cell table, keeps a running maximum / denominator / weighted sum of value
+// [max(0, p - window + 1), p] (chunk mask: of the token's chunk [p - p % window, p]) and the kept first positions [0, keep) through the slot's position -> cell table, keeps a running maximum / denominator / weighted sum of value
 // rows, and the shares of a head are merged in shared memory.  A sink (optional) is one more logit without a row: the running state of
-// share 0 starts at (max = sink, denominator = 1).
+// share 0 starts at (max = sink, denominator = 1).  softcap > 0: a score becomes softcap tanh(score / softcap).
 template <int RPL>
-__global__ void __launch_bounds__(512) kv_attn_kernel(const float * __restrict__ q, int H, int G, int maps, int D, int V, float scale, int window, int mask, const float * __restrict__ sink,
+__global__ void __launch_bounds__(512) kv_attn_kernel(const float * __restrict__ q, int H, int G, int maps, int D, int V, float scale, int window, int mask, int keep, float softcap, const float * __restrict__ sink,
                                                       const int32_t * __restrict__ pos, const int32_t * __restrict__ slot, const float * __restrict__ cache, int cache_row,
                                                       const int32_t * __restrict__ cellmap, int n_ctx, int HPB, int KS, float * __restrict__ out,
                                                       const int32_t * __restrict__ skip) {
@@ -134,16 +134,19 @@ __global__ void __launch_bounds__(512) kv_attn_kernel(const float * __restrict__
         if (ks == 0 && sink) { m = sink[h]; l = 1.f; }
         const int32_t * map = cellmap + (size_t) slot[t] * n_ctx;
         const size_t ko = (size_t) (g * maps + mp) * D, vo = (size_t) G * maps * D + (size_t) g * V;
-        for (int j = lo + ks; j <= p; j += KS) {
+        const int nf = min(keep, lo), n_keys = nf + p - lo + 1;          // kept positions in front of the window, then the window
+        for (int e = ks; e < n_keys; e += KS) {
+            const int     j   = e < nf ? e : lo + e - nf;
             const float * row = cache + (size_t) map[j] * cache_row;
             float s = 0.f, c[RPL];
 #pragma unroll
             for (int i = 0; i < RPL; i++) { const int r = i * 32 + lane; if (r < D) s = fmaf(qv[i], row[ko + r], s); c[i] = r < V ? row[vo + r] : 0.f; }
             s = warp_sum(s);
-            const float mn = fmaxf(m, s), a = expf(m - mn), e = expf(s - mn);         // m == -inf only before the first key: a = 0
-            l = l * a + e;
+            if (softcap > 0.f) s = softcap * tanhf(s / softcap);
+            const float mn = fmaxf(m, s), a = expf(m - mn), w = expf(s - mn);         // m == -inf only before the first key: a = 0
+            l = l * a + w;
 #pragma unroll
-            for (int i = 0; i < RPL; i++) acc[i] = fmaf(acc[i], a, e * c[i]);
+            for (int i = 0; i < RPL; i++) acc[i] = fmaf(acc[i], a, w * c[i]);
             m = mn;
         }
         float * part = sm + (size_t) warp * (V + 2);
@@ -180,13 +183,13 @@ int pib_kv_attention(const float * q, const pib_hlayer & L, const pib_hbatch & b
     const int H = L.heads * L.maps, V = L.vdim, R = L.dim > L.vdim ? L.dim : L.vdim;
     const int HPB = (long long) b.T * H <= 1024 ? 1 : (H < 4 ? H : 4);
     int KS = 16 / HPB;
-    if (L.window < 64) KS = 1;
+    if (L.window + L.keep < 64) KS = 1;
     const size_t smem = (size_t) HPB * KS * (V + 2) * 4;
     dim3 grid((unsigned) b.T, (unsigned) ((H + HPB - 1) / HPB));
     const int threads = HPB * KS * 32;
 #define KA_GO(RPL) do {                                                                                                              \
         if (smem > 48 * 1024) cudaFuncSetAttribute(kv_attn_kernel<RPL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int) smem);   \
-        pib_launch(kv_attn_kernel<RPL>, dim3(grid), dim3(threads), (size_t) smem, st, q, H, L.kv_heads, L.maps, L.dim, V, L.scale, L.window, L.mask, (const float *) L.sink, b.pos, b.slot, cache, \
+        pib_launch(kv_attn_kernel<RPL>, dim3(grid), dim3(threads), (size_t) smem, st, q, H, L.kv_heads, L.maps, L.dim, V, L.scale, L.window, L.mask, L.keep, L.softcap, (const float *) L.sink, b.pos, b.slot, cache, \
                    cache_row, cellmap, n_ctx, HPB, KS, out, skip);                                                                  \
     } while (0)
     if (R <= 32) KA_GO(1); else if (R <= 64) KA_GO(2); else if (R <= 128) KA_GO(4); else if (R <= 256) KA_GO(8); else if (R <= 512) KA_GO(16);
@@ -204,12 +207,13 @@ int pib_kv_attention(const float * q, const pib_hlayer & L, const pib_hbatch & b
 // [hi | lo] against the values twice side by side.  These kernels prepare the operands -- keys [G][NKp][3 D], values transposed
 // [G][V][2 NKp], query rows [G][nq * rep][3 D], all bfloat16 -- and put the outputs [G][nq * rep][V] back in token order.
 __device__ __forceinline__ void mk_split(float x, __nv_bfloat16 & hi, __nv_bfloat16 & lo) { hi = __float2bfloat16_rn(x); lo = __float2bfloat16_rn(x - __bfloat162float(hi)); }
-__global__ void __launch_bounds__(128) kv_gather_kernel(const float * __restrict__ cache, int cache_row, const int32_t * __restrict__ map, int j0, int NK, int NKp, int G, int maps,
+// columns [0, n_front) are positions 0 .. n_front - 1, the columns behind them positions j0, j0 + 1, ...
+__global__ void __launch_bounds__(128) kv_gather_kernel(const float * __restrict__ cache, int cache_row, const int32_t * __restrict__ map, int j0, int n_front, int NK, int NKp, int G, int maps,
                                                         int D, int V, __nv_bfloat16 * __restrict__ Kb, __nv_bfloat16 * __restrict__ Vt) {
     pib_pdl_wait();
     pib_pdl_trigger();
     const int j = blockIdx.x, GK = G * maps;          // one problem per (key / value head, map): its own keys, the head's values
-    const float * row = j < NK ? cache + (size_t) map[j0 + j] * cache_row : nullptr;
+    const float * row = j < NK ? cache + (size_t) map[j < n_front ? j : j0 + j - n_front] * cache_row : nullptr;
     for (int i = threadIdx.x; i < GK * D; i += blockDim.x) {
         __nv_bfloat16 hi, lo;
         mk_split(row ? row[i] : 0.f, hi, lo);
@@ -249,11 +253,11 @@ __global__ void __launch_bounds__(128) kv_token_order_kernel(const float * __res
     float * dst = out + ((size_t) (t0 + ti) * H + h) * V;
     for (int i = threadIdx.x; i < V; i += blockDim.x) dst[i] = src[i];
 }
-int pib_kv_attention_mm(const float * q, const pib_hlayer & L, const pib_hbatch & b, const float * cache, int cache_row, const int32_t * map, int t0, int nq, int j0, int NK,
+int pib_kv_attention_mm(const float * q, const pib_hlayer & L, const pib_hbatch & b, const float * cache, int cache_row, const int32_t * map, int t0, int nq, int j0, int n_front, int NK,
                         void * Kb, void * Vt, float * Qc, float * S, void * P, float * out, cudaStream_t st) {
     const int maps = L.maps, H = L.heads * maps, G = L.kv_heads, GK = G * maps, D = L.dim, V = L.vdim, rep = L.heads / G, NKp = (NK + 7) & ~7, M = nq * rep;
     if (maps > 1 && L.sink) { pib_set_error("attention: a sink with several maps per head"); return PIB_ERR_UNSUPP; }
-    pib_launch(kv_gather_kernel, dim3(NKp), dim3(128), (size_t) 0, st, cache, cache_row, map, j0, NK, NKp, G, maps, D, V, (__nv_bfloat16 *) Kb, (__nv_bfloat16 *) Vt);
+    pib_launch(kv_gather_kernel, dim3(NKp), dim3(128), (size_t) 0, st, cache, cache_row, map, j0, n_front, NK, NKp, G, maps, D, V, (__nv_bfloat16 *) Kb, (__nv_bfloat16 *) Vt);
     CKL();
     pib_launch(kv_query_rows_kernel, dim3((unsigned) nq, (unsigned) H), dim3(128), (size_t) 0, st, q, (__nv_bfloat16 *) Qc, H, maps, rep, nq, D, t0, L.scale);
     CKL();
@@ -262,7 +266,7 @@ int pib_kv_attention_mm(const float * q, const pib_hlayer & L, const pib_hbatch 
     a.Y = S; a.ldy = NKp; a.yz = (int64_t) M * NKp; a.M = M; a.N = NK; a.K = 3 * D; a.Z = GK;
     int rc = pib_dense_mm(a, st);
     if (rc != PIB_OK) return rc;
-    if ((rc = pib_window_softmax(S, P, NKp, NK, j0, L.window, b.pos, t0, GK * M, M, rep, L.sink, st, L.mask)) != PIB_OK) return rc;
+    if ((rc = pib_window_softmax(S, P, NKp, NK, j0, L.window, b.pos, t0, GK * M, M, rep, L.sink, st, L.mask, L.keep, n_front, L.softcap)) != PIB_OK) return rc;
     pib_mm v;
     v.W = Vt; v.wtype = PIB_TYPE_BF16; v.ldw = 2 * NKp; v.wz = (int64_t) V * 2 * NKp; v.X = (const float *) P; v.ldx = 2 * NKp; v.xz = (int64_t) M * 2 * NKp; v.x_bf16 = 1;
     v.Y = Qc; v.ldy = V; v.yz = (int64_t) M * V; v.M = M; v.N = V; v.K = 2 * NKp; v.Z = GK;              // the query rows are used up: the outputs take their place
@@ -364,6 +368,8 @@ int pib_delta_prep(float * cv, int ldc, const pib_hlayer & L, const float * proj
 //   MODE 2 (constant decay): s_d <- c s_d + k_d v,  o = sum_d a_d s_d  (read after the write; c one number per head)   row = [a D | k D | v LS_VT | dot]
 //   MODE 3 (one decay per head and token, Mamba-2): s_d <- c s_d + (dt k_d) v,  o = sum_d a_d s_d + u v  (read after the write; u one number per head)
 //                                                                                                           row = [a D | k D | v LS_VT | c, dt | dot]
+//   MODE 4 (matrix memory): s_d <- c s_d + (w k_d) v,  o = sum_d a_d s_d  (read after the write); one more column, whose value is always 1 and which v's
+//                           rows do not hold (its sums are the normaliser's)                                  row = [a D | k D | v LS_VT | c, w | dot]
 // What does not depend on the matrix or the column -- dot = sum_d a_d u_d k_d (MODE 0), sum_d a_d k_d (MODE 1) -- is formed once per token
 // when its chunk has landed; in MODE 1 the read-out is taken from the sums over the matrix before the write (one round of shuffles for
 // both sums), and the next token's rows are already in registers while the sums of this one cross the lanes.
@@ -372,7 +378,7 @@ int pib_delta_prep(float * cv, int ldc, const pib_hlayer & L, const float * proj
 struct ls_args {
     const float * a; int lda, a_hs;          // query-like rows: a[t * lda + group * a_hs + d]
     const float * k; int ldk, k_hs;
-    const float * w; int ldw;                // MODE 0: decay rows w[t * ldw + h * D + d];   MODE 1: bg rows [beta (H) | g (H)], ldw = 2 H;   MODE 2: decay [H];   MODE 3: rows [dt (H) | c (H)]
+    const float * w; int ldw;                // MODE 0: decay rows w[t * ldw + h * D + d];   MODE 1: bg rows [beta (H) | g (H)], ldw = 2 H;   MODE 2: decay [H];   MODE 3, 4: rows [dt (H) | c (H)]
     const float * v; int ldv;                // v[t * ldv + h * V + j]
     const float * u;                         // MODE 0: bonus [H][D];   MODE 3: skip [H]
     int H, G, D, V, chunk;
@@ -394,9 +400,10 @@ __global__ void __launch_bounds__(16 * LS_VT) lin_scan_kernel(ls_args A) {
     pib_pdl_trigger();
     extern __shared__ float hs[];
     const int sg = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * LS_VT, part = threadIdx.x & 15, vl = threadIdx.x >> 4, vd = v0 + vl;
-    const int D = FULL ? 16 * RPT : A.D, V = A.V, H = A.H, grp = h / (H / A.G), CH = A.chunk;
+    const int D = FULL ? 16 * RPT : A.D, Vv = A.V, V = MODE == 4 ? A.V + 1 : A.V, H = A.H, grp = h / (H / A.G), CH = A.chunk;
     const int s0 = A.seg_start[sg], n = A.seg_len[sg];
-    const int vbase = MODE == 0 ? 3 * D : 2 * D, dot_off = vbase + LS_VT + ((MODE == 1 || MODE == 3) ? 2 : 0), row_f = (dot_off + 4) & ~3;
+    constexpr bool TWO = MODE == 1 || MODE == 3 || MODE == 4;      // two numbers per head and token beside the rows
+    const int vbase = MODE == 0 ? 3 * D : 2 * D, dot_off = vbase + LS_VT + (TWO ? 2 : 0), row_f = (dot_off + 4) & ~3;
     const float cdec = MODE == 2 ? A.w[h] : 0.f, skip = MODE == 3 ? A.u[h] : 0.f;
     const bool vok = vd < V;
     float * S = A.state + (size_t) A.seg_slot[sg] * A.state_stride + A.state_off + (size_t) h * D * V;
@@ -420,13 +427,13 @@ __global__ void __launch_bounds__(16 * LS_VT) lin_scan_kernel(ls_args A) {
                 const float * src = which == 0 ? A.a + tt * A.lda + (size_t) grp * A.a_hs : which == 1 ? A.k + tt * A.ldk + (size_t) grp * A.k_hs : A.w + tt * A.ldw + (size_t) h * D;
                 asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(base + 4u * (uint32_t) (t * row_f + which * D + 4 * i)), "l"(src + 4 * i) : "memory");
             }
-            constexpr int NS = LS_VT + ((MODE == 1 || MODE == 3) ? 2 : 0);
+            constexpr int NS = LS_VT + (TWO ? 2 : 0);
             for (int p = threadIdx.x; p < nc * NS; p += blockDim.x) {
                 const int t = p / NS, j = p - t * NS;
                 const size_t tt = (size_t) (s0 + c0 + t);
                 const uint32_t dst = base + 4u * (uint32_t) (t * row_f + vbase + j);
                 if (j < LS_VT) {
-                    if (v0 + j < V) asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(dst), "l"(A.v + tt * A.ldv + (size_t) h * V + v0 + j) : "memory");
+                    if (v0 + j < Vv) asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(dst), "l"(A.v + tt * A.ldv + (size_t) h * Vv + v0 + j) : "memory");
                 } else {
                     asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(dst), "l"(A.w + tt * A.ldw + (j == LS_VT ? H : 0) + h) : "memory");
                 }
@@ -444,9 +451,9 @@ __global__ void __launch_bounds__(16 * LS_VT) lin_scan_kernel(ls_args A) {
                 asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(dst + 4u * (D + e)), "l"(kr + e) : "memory");
                 if (MODE == 0) asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(dst + 4u * (2 * D + e)), "l"(A.w + tt * A.ldw + (size_t) h * D + e) : "memory");
             }
-            if (threadIdx.x < LS_VT && v0 + (int) threadIdx.x < V)
-                asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(dst + 4u * (vbase + threadIdx.x)), "l"(A.v + tt * A.ldv + (size_t) h * V + v0 + threadIdx.x) : "memory");
-            if ((MODE == 1 || MODE == 3) && threadIdx.x >= 32 && threadIdx.x < 34) {       // g, then beta (MODE 3: the decay, then dt)
+            if (threadIdx.x < LS_VT && v0 + (int) threadIdx.x < Vv)
+                asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(dst + 4u * (vbase + threadIdx.x)), "l"(A.v + tt * A.ldv + (size_t) h * Vv + v0 + threadIdx.x) : "memory");
+            if (TWO && threadIdx.x >= 32 && threadIdx.x < 34) {       // g, then beta (MODE 3: the decay, then dt)
                 const int which = threadIdx.x - 32;
                 asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(dst + 4u * (vbase + LS_VT + which)), "l"(A.w + tt * A.ldw + (which == 0 ? H : 0) + h) : "memory");
             }
@@ -485,7 +492,7 @@ __global__ void __launch_bounds__(16 * LS_VT) lin_scan_kernel(ls_args A) {
         for (int t = 0; t < nc; t++, op += ostride) {
             const float * sc = qp - part + vbase;            // this token's scalars
             const float * qn = t + 1 < nc ? qp + row_f : qp; // the next token's rows (the last token reads its own again)
-            const float v = vok ? sc[vl] : 0.f, dot = sc[dot_off - vbase];
+            const float v = MODE == 4 && vd == Vv ? 1.0f : vok ? sc[vl] : 0.f, dot = sc[dot_off - vbase];
             float an[RPT], kn[RPT], wn[RPT];
             if (MODE == 0) {
                 float acc = 0.f;
@@ -509,7 +516,7 @@ __global__ void __launch_bounds__(16 * LS_VT) lin_scan_kernel(ls_args A) {
                 }
                 acc = ls_sum16(acc);
                 if (part == 0 && vok) *op = fmaf(cdec, acc, v * dot);       // sum_d a_d (c s_d + k_d v)
-            } else if (MODE == 3) {
+            } else if (MODE == 3 || MODE == 4) {
                 const float dec = sc[LS_VT], kv = sc[LS_VT + 1] * v;
                 float acc = 0.f;
 #pragma unroll
@@ -520,7 +527,7 @@ __global__ void __launch_bounds__(16 * LS_VT) lin_scan_kernel(ls_args A) {
                     an[r] = ok ? qn[16 * r] : 0.f; kn[r] = ok ? qn[D + 16 * r] : 0.f; wn[r] = 0.f;
                 }
                 acc = ls_sum16(acc);
-                if (part == 0 && vok) *op = fmaf(dec, acc, fmaf(kv, dot, skip * v));      // sum_d a_d (c s_d + dt k_d v) + u v
+                if (part == 0 && vok) *op = fmaf(dec, acc, MODE == 3 ? fmaf(kv, dot, skip * v) : kv * dot);      // sum_d a_d (c s_d + dt k_d v) + u v
             } else {
                 const float g = sc[LS_VT], beta = sc[LS_VT + 1];
                 float sk = 0.f, sa = 0.f;
@@ -550,8 +557,9 @@ __global__ void __launch_bounds__(16 * LS_VT) lin_scan_kernel(ls_args A) {
 
 static int lin_scan(int mode, ls_args & A, int S, cudaStream_t st) {
     if (A.D > 256) { pib_set_error("recurrence: dim %d not supported (up to 256)", A.D); return PIB_ERR_UNSUPP; }
-    dim3 grid((unsigned) S, (unsigned) A.H, (unsigned) ((A.V + LS_VT - 1) / LS_VT));
-    const size_t row_f = ((size_t) (mode == 0 ? 3 * A.D : 2 * A.D) + LS_VT + ((mode == 1 || mode == 3) ? 2 : 0) + 4) & ~(size_t) 3;
+    const int Vt = A.V + (mode == 4 ? 1 : 0);
+    dim3 grid((unsigned) S, (unsigned) A.H, (unsigned) ((Vt + LS_VT - 1) / LS_VT));
+    const size_t row_f = ((size_t) (mode == 0 ? 3 * A.D : 2 * A.D) + LS_VT + ((mode == 1 || mode == 3 || mode == 4) ? 2 : 0) + 4) & ~(size_t) 3;
     {   // 16-byte staging copies need every operand row to start on a 16-byte boundary
         static const int on = getenv("PIB_SCAN_VEC") ? atoi(getenv("PIB_SCAN_VEC")) : 1;
         auto al = [](const void * p) { return ((uintptr_t) p & 15) == 0; };
@@ -567,7 +575,7 @@ static int lin_scan(int mode, ls_args & A, int S, cudaStream_t st) {
                                     pib_launch(lin_scan_kernel<RPT, MODE, FULL>, dim3(grid), dim3(16 * LS_VT), (size_t) smem, st, A); } while (0)
 #define LS_PICK(MODE) do { if (A.D == 64) LS_GO(4, MODE, true); else if (A.D == 128) LS_GO(8, MODE, true); else if (A.D <= 32) LS_GO(2, MODE, false); \
                            else if (A.D <= 64) LS_GO(4, MODE, false); else if (A.D <= 128) LS_GO(8, MODE, false); else LS_GO(16, MODE, false); } while (0)
-    if (mode == 0) LS_PICK(0); else if (mode == 1) LS_PICK(1); else if (mode == 2) LS_PICK(2); else LS_PICK(3);
+    if (mode == 0) LS_PICK(0); else if (mode == 1) LS_PICK(1); else if (mode == 2) LS_PICK(2); else if (mode == 3) LS_PICK(3); else LS_PICK(4);
 #undef LS_PICK
 #undef LS_GO
     CKL();
@@ -686,7 +694,7 @@ size_t pib_decay_split_bytes(const pib_hlayer & L, int parts) { return pib_scan_
 static int scan_in_parts(int mode, ls_args A, const float * q, int ldq, const float * decay, const float * cum, int ldc, const pib_hbatch & b, float * state, size_t state_stride,
                          size_t state_off, float * split_buf, int parts, int per, cudaStream_t st) {
     if (b.S != 1) { pib_set_error("recurrence in parts: the batch must be one segment"); return PIB_ERR_ARG; }
-    const int H = A.H, D = A.D, V = A.V, E = H * D * V;
+    const int H = A.H, D = A.D, V = A.V + (mode == 4 ? 1 : 0), E = H * D * V;
     float * Lm = split_buf, * F = split_buf + (size_t) parts * E;
     int32_t * table = reinterpret_cast<int32_t *>(split_buf + (size_t) 2 * parts * E);
     const int64_t n = (int64_t) parts * E;
@@ -753,6 +761,21 @@ int pib_mamba2_scan(const float * xbc, int ldc, float * dg, const pib_hlayer & L
     pib_launch(cum_decay_kernel, dim3((unsigned) ((parts * H + 127) / 128)), dim3(128), (size_t) 0, st, dg + 2 * H, 3 * H, H, b.T, per, parts);
     CKL();
     return scan_in_parts(3, A, xbc + I + GN, ldc, nullptr, dg + 2 * H, 3 * H, b, state, state_stride, L.state_off, split_buf, parts, per, st);
+}
+
+// matrix memory: rows proj[t] hold q (H*D) at q_off, k (H*D) at k_off, v (H*V) at v_off; dg[t] = [e^(i - m) (H) | decay (H) | log decay (H) | e^-m (H)]
+// (pib_attn_mem_prep); the matrices are [H][D][V + 1], out [T][H][V + 1] = [S^T q | n . q].  Parts as for Mamba-2.
+int pib_memory_scan(const float * proj, int ldp, int q_off, int k_off, int v_off, float * dg, const pib_hlayer & L, const pib_hbatch & b, float * state, size_t state_stride, float * out,
+                    cudaStream_t st, float * split_buf, int parts, int per) {
+    const int H = L.heads2;
+    ls_args A;
+    A.a = proj + q_off; A.lda = ldp; A.a_hs = L.dim2; A.k = proj + k_off; A.ldk = ldp; A.k_hs = L.dim2; A.w = dg; A.ldw = 4 * H; A.v = proj + v_off; A.ldv = ldp; A.u = nullptr;
+    A.H = H; A.G = H; A.D = L.dim2; A.V = L.vdim2; A.seg_start = b.seg_start; A.seg_len = b.seg_len; A.seg_slot = b.seg_slot;
+    A.state = state; A.state_stride = state_stride; A.state_off = L.state_off; A.out = out;
+    if (parts < 2 || !split_buf) return lin_scan(4, A, b.S, st);
+    pib_launch(cum_decay_kernel, dim3((unsigned) ((parts * H + 127) / 128)), dim3(128), (size_t) 0, st, dg + 2 * H, 4 * H, H, b.T, per, parts);
+    CKL();
+    return scan_in_parts(4, A, proj + q_off, ldp, nullptr, dg + 2 * H, 4 * H, b, state, state_stride, L.state_off, split_buf, parts, per, st);
 }
 
 // one warp per (token, head): o <- o / sqrt(mean(o^2) + eps) * w[(h * w_hs) + i] * silu(gate[t * ldg + h * V + i])

@@ -200,7 +200,8 @@ struct TensorSource {
             else if (ends(name, "lower")) v = 0.45f + 0.45f * u;
             else if (ends(name, ".act")) v = (i == 0 ? 0.6f : i == 1 ? 0.3f : i == 2 ? 0.2f : 0.05f);
             else if (ends(name, "sink") || ends(name, "f.b")) v = u;
-            else if (ends(name, "canon1")) v = 0.3f * u;
+            else if (ends(name, "canon1") || ends(name, "canon2")) v = 0.3f * u;
+            else if (ends(name, ".out") && name.find(".mix.") != std::string::npos) v = 1.0f + 0.2f * u;
             else if (name == "embed") v = 1.7f * u;
             else v = amp * u;
             out[i] = __bfloat162float(__float2bfloat16_rn(v));
@@ -229,10 +230,28 @@ static pib_weight * upload_mat(const std::vector<float> & v, int64_t N, int64_t 
     return w;
 }
 
+// gate row i and up row i next to each other: the matmul's paired epilogue forms the activation on the way out
+static pib_weight * upload_gate_up(TensorSource & src, const std::string & pre, int ff, int W, int dtype, pib_model * m) {
+    std::vector<float> v, all((size_t) 2 * ff * W);
+    const char * names[2] = { "gate", "up" };
+    for (int k = 0; k < 2; k++) {
+        if (!src.get(pre + names[k], { (int64_t) ff, (int64_t) W }, v)) return nullptr;
+        for (int64_t i = 0; i < ff; i++) memcpy(&all[(size_t) (2 * i + k) * W], &v[(size_t) i * W], (size_t) W * 4);
+    }
+    return upload_mat(all, 2 * (int64_t) ff, W, dtype, m);
+}
+
 static double jnum(const Json * o, const char * k, double dflt, bool * ok = nullptr) {
     const Json * v = o ? o->get(k) : nullptr;
     if (!v || v->kind != Json::NUM) { if (ok) *ok = false; return dflt; }
     return v->num;
+}
+
+// the rotation table of these constants: one per distinct set
+static int rope_index(pib_hybrid * hy, const pib_hybrid::Rope & r) {
+    for (size_t i = 0; i < hy->ropes.size(); i++) if (hy->ropes[i] == r) return (int) i;
+    hy->ropes.push_back(r);
+    return (int) hy->ropes.size() - 1;
 }
 
 // ---- the Rapisun builder ----------------------------------------------------------------------------------------------------------
@@ -863,13 +882,7 @@ static pib_model * build_putazen(const Json & cfg, TensorSource & src, int dtype
             VEC(L.norm2, p + "norm2", W);
             VEC(L.norm2_b, p + "norm2.b", W);
             if (!hyper(p + "hc2.", L.hc2)) return nullptr;
-            // gate row i and up row i next to each other: the matmul's paired epilogue forms the activation on the way out
-            std::vector<float> all((size_t) 2 * L.ff * W);
-            GET(pm + "gate", (int64_t) L.ff, W);
-            for (int64_t i = 0; i < L.ff; i++) memcpy(&all[(size_t) (2 * i) * W], &v[(size_t) i * W], (size_t) W * 4);
-            GET(pm + "up", (int64_t) L.ff, W);
-            for (int64_t i = 0; i < L.ff; i++) memcpy(&all[(size_t) (2 * i + 1) * W], &v[(size_t) i * W], (size_t) W * 4);
-            if (!(L.up = upload_mat(all, 2 * (int64_t) L.ff, W, dtype, m))) return nullptr;
+            if (!(L.up = upload_gate_up(src, pm, L.ff, W, dtype, m))) return nullptr;
             MAT(L.down, pm + "down", W, L.ff);
             widen(hy->w_proj, (int64_t) L.ff);
         }
@@ -897,14 +910,10 @@ static pib_model * build_putazen(const Json & cfg, TensorSource & src, int dtype
             const Json * mx = layers->arr[(size_t) il].get("mixer"), * rt = mx ? mx->get("rot") : nullptr, * sc = rt ? rt->get("scaling") : nullptr;
             if (L.mixer == PIB_MIXER_DIFF && sc && !sc->is_null()) {
                 r.factor = jnum(sc, "factor", 1.0); r.original = jnum(sc, "original", 1.0); r.fast = jnum(sc, "fast", 32.0); r.slow = jnum(sc, "slow", 1.0);
+                r.scaling = PIB_ROPE_YARN;
                 if (!(r.factor > 0) || !(r.original > 0) || !(r.fast > 0) || !(r.slow > 0)) { pib_set_error("model: layer %d: rot.scaling", il); return nullptr; }
             }
-            L.rope_id = -1;
-            for (size_t i = 0; i < hy->ropes.size(); i++) {
-                const pib_hybrid::Rope & o = hy->ropes[i];
-                if (o.base == r.base && o.dims == r.dims && o.factor == r.factor && o.original == r.original && o.fast == r.fast && o.slow == r.slow) L.rope_id = (int) i;
-            }
-            if (L.rope_id < 0) { L.rope_id = (int) hy->ropes.size(); hy->ropes.push_back(r); }
+            L.rope_id = rope_index(hy, r);
         }
         hy->layers.push_back(L);
     }
@@ -917,9 +926,140 @@ static pib_model * build_putazen(const Json & cfg, TensorSource & src, int dtype
     return mp.release();
 }
 
+// ---- the Bobunex builder ----------------------------------------------------------------------------------------------------------
+// Sequential pre-norm layers with an input convolution in front of both sublayers and a sigmoid gate per channel on what each adds to the
+// stream; the mixer "parallel" (windowed softmax attention that keeps the first tokens, beside a matrix memory with exponential gates; the
+// mean of their normed outputs); dense feed-forwards gated with a gelu.  Sizes the configuration leaves out come from the tensors' shapes.
+// Tensor names: '<layer>.norm1|norm2|canon1|canon2', '<layer>.rg1|rg2' (+ '.b'), '<layer>.mix.left|right.*', '<layer>.mlp.gate|up|down', 'final.norm', 'embed', 'head'.
+static pib_model * build_bobunex(const Json & cfg, TensorSource & src, int dtype) {
+    std::unique_ptr<pib_model, void (*)(pib_model *)> mp(new pib_model(), pib_model_free);
+    pib_model * m = mp.get();
+    pib_hybrid * hy = new pib_hybrid();
+    m->hy = hy;
+    m->arch = 2; m->name = "Bobunex";
+    bool ok = true;
+    const int W = (int) jnum(&cfg, "width", 0, &ok), V = (int) jnum(&cfg, "vocab", 0, &ok);
+    const Json * layers = cfg.get("layers");
+    if (!ok || W <= 0 || V <= 0 || !layers || layers->kind != Json::ARR || layers->arr.empty()) { pib_set_error("model: config.json needs width, vocab and layers"); return nullptr; }
+    hy->dtype = dtype;
+    hy->form = PIB_FORM_GATED;
+    hy->eps = (float) jnum(cfg.get("norm"), "eps", 1e-5);
+    hy->embd_scale = (float) jnum(cfg.get("embedding"), "scale", 1.0);
+    hy->taps = (int) jnum(cfg.get("canon"), "taps", (double) src.dim("l0.canon1", 1, 1));
+    if (hy->taps < 1) { pib_set_error("model: canon.taps %d", hy->taps); return nullptr; }
+    m->n_embd = W; m->n_vocab = V; m->n_layer = (int) layers->arr.size(); m->layer_begin = 0; m->layer_end = m->n_layer;
+    m->wtype = dtype; m->n_ctx_train = 1 << 20; m->n_head = 1; m->n_head_kv = 1; m->tok_bos = -1; m->tok_eos = -1;
+    std::vector<float> v;
+#define GET(name, ...) do { if (!src.get((name), { __VA_ARGS__ }, v)) return nullptr; } while (0)
+#define VEC(dst, name, n) do { GET(name, (int64_t) (n)); if (!((dst) = upload_f32v(v))) return nullptr; } while (0)
+#define MAT(dst, name, N, K) do { GET(name, (int64_t) (N), (int64_t) (K)); if (!((dst) = upload_mat(v, (N), (K), dtype, m))) return nullptr; } while (0)
+#define APPEND(all, name, N, K) do { GET(name, (int64_t) (N), (int64_t) (K)); (all).insert((all).end(), v.begin(), v.end()); } while (0)
+    MAT(m->tok_embd, "embed", V, W);
+    VEC(m->output_norm, "final.norm", W);
+    MAT(m->output, "head", V, W);
+    hy->layers.resize(m->n_layer);
+    hy->w_gate = hy->w_y2 = W;
+    const size_t tail = (size_t) (hy->taps - 1) * W;
+    size_t state = 0;
+    auto widen = [](int & a, int64_t b) { if (b > a) a = (int) b; };
+    for (int il = 0; il < m->n_layer; il++) {
+        const Json & jl = layers->arr[il];
+        pib_hlayer & L = hy->layers[il];
+        const std::string p = "l" + std::to_string(il) + ".", pl = p + "mix.left.", pr = p + "mix.right.", pm = p + "mlp.";
+        const Json * ty = jl.get("type"), * mx = jl.get("mixer"), * ml = jl.get("mlp");
+        if (!ty || ty->kind != Json::STR || !mx) { pib_set_error("model: layer %d needs type and mixer", il); return nullptr; }
+        if (ty->str != "parallel") { pib_set_error("model: layer %d: unknown mixer '%s'", il, ty->str.c_str()); return nullptr; }
+        const Json * a = mx->get("left"), * b = mx->get("right");
+        if (!a || !b) { pib_set_error("model: layer %d: the mixer needs left and right", il); return nullptr; }
+        // ---- the frame ----
+        VEC(L.norm1, p + "norm1", W);
+        GET(p + "canon1", W, (int64_t) hy->taps);
+        if (!(L.canon = upload_f32v(v))) return nullptr;
+        MAT(L.rg1, p + "rg1", W, W);
+        VEC(L.rg1_b, p + "rg1.b", W);
+        L.tail_off = state; state += tail;
+        // ---- the attention branch ----
+        L.mixer = PIB_MIXER_ATTN_MEM;
+        L.heads = (int) jnum(a, "heads", (double) src.dim(pl + "g", 0, 0));
+        L.dim = (int) jnum(a, "dim", L.heads > 0 ? (double) (src.dim(pl + "q", 0, 0) / L.heads) : 0.0);
+        L.kv_heads = (int) jnum(a, "kv_heads", L.dim > 0 ? (double) src.dim(pl + "k", 0, (int64_t) L.heads * L.dim) / L.dim : 0.0);
+        L.vdim = (int) jnum(a, "vdim", L.kv_heads > 0 ? (double) src.dim(pl + "v", 0, (int64_t) L.kv_heads * L.dim) / L.kv_heads : 0.0);
+        if (L.heads <= 0 || L.dim <= 0 || L.vdim <= 0 || L.kv_heads <= 0 || L.heads % L.kv_heads) { pib_set_error("model: layer %d: left heads / kv_heads / dim / vdim", il); return nullptr; }
+        L.scale = (float) jnum(a, "scale", 1.0 / sqrt((double) L.dim));
+        L.softcap = (float) jnum(a, "softcap", 0.0);
+        const Json * mk = a->get("mask"), * rt = a->get("rot"), * sc = rt ? rt->get("scaling") : nullptr;
+        L.window = (int) std::min(jnum(mk, "size", 0.0), (double) (1 << 30));
+        if (L.window <= 0) L.window = 1 << 30;                              // no mask: every earlier token is seen
+        L.keep = (int) std::min(std::max(jnum(mk, "keep_first", 0.0), 0.0), (double) (1 << 29));
+        L.rot_base = (float) jnum(rt, "base", 10000.0); L.rot_dims = rt && !rt->is_null() ? (int) jnum(rt, "dims", (double) L.dim) : 0;
+        if (L.rot_dims < 0 || L.rot_dims > L.dim || (L.rot_dims & 1)) { pib_set_error("model: layer %d: rot.dims %d of %d", il, L.rot_dims, L.dim); return nullptr; }
+        pib_hybrid::Rope rope = { L.rot_base, L.rot_dims };
+        if (sc && !sc->is_null()) {
+            rope.scaling = PIB_ROPE_BANDS;
+            rope.factor = jnum(sc, "factor", 1.0); rope.original = jnum(sc, "original", 1.0); rope.fast = jnum(sc, "high", 4.0); rope.slow = jnum(sc, "low", 1.0);
+            if (!(rope.factor > 0) || !(rope.original > 0)) { pib_set_error("model: layer %d: rot.scaling", il); return nullptr; }
+        }
+        L.rope_id = rope_index(hy, rope);
+        // ---- the memory branch ----
+        L.heads2 = (int) jnum(b, "heads", (double) src.dim(pr + "i.b", 0, 0));
+        L.dim2 = (int) jnum(b, "dim", L.heads2 > 0 ? (double) (src.dim(pr + "q", 0, 0) / L.heads2) : 0.0);
+        L.vdim2 = (int) jnum(b, "vdim", L.heads2 > 0 ? (double) (src.dim(pr + "v", 0, (int64_t) L.heads2 * L.dim2) / L.heads2) : 0.0);
+        L.gate_cap = (float) jnum(b, "gate_cap", 0.0);
+        if (L.heads2 <= 0 || L.dim2 <= 0 || L.vdim2 <= 0) { pib_set_error("model: layer %d: right heads / dim / vdim", il); return nullptr; }
+        const int64_t H = L.heads, G = L.kv_heads, D = L.dim, Vd = L.vdim, H2 = L.heads2, D2 = L.dim2, V2 = L.vdim2;
+        const int64_t rows = (H + G) * D + G * Vd + 2 * H2 * D2 + 2 * H2 * V2 + H + 2 * H2;
+        std::vector<float> all;
+        APPEND(all, pl + "q", H * D, W); APPEND(all, pl + "k", G * D, W); APPEND(all, pl + "v", G * Vd, W);
+        APPEND(all, pr + "q", H2 * D2, W); APPEND(all, pr + "k", H2 * D2, W); APPEND(all, pr + "v", H2 * V2, W); APPEND(all, pr + "g", H2 * V2, W);
+        APPEND(all, pl + "g", H, W); APPEND(all, pr + "i", H2, W); APPEND(all, pr + "f", H2, W);
+        if (!(L.qkv = upload_mat(all, rows, W, dtype, m))) return nullptr;
+        VEC(L.q_norm, pl + "q.norm", H * D);
+        VEC(L.k_norm, pl + "k.norm", G * D);
+        v.assign((size_t) H, 0.f);                                          // a sink of score 0 for every head
+        if (!(L.sink = upload_f32v(v))) return nullptr;
+        VEC(L.i_bias, pr + "i.b", H2);
+        VEC(L.f_bias, pr + "f.b", H2);
+        VEC(L.onorm, pr + "norm", H2 * V2);
+        MAT(L.wo, pl + "o", W, H * Vd);
+        MAT(L.wo2, pr + "o", W, H2 * V2);
+        VEC(L.out_a, pl + "out", W);
+        VEC(L.out_b, pr + "out", W);
+        L.mix_a = L.mix_b = 0.5f;
+        L.state_off = state; state += (size_t) (H2 * D2 * (V2 + 1));
+        L.max_off = state; state += (size_t) H2;
+        L.cache_id = hy->n_cache++;
+        hy->cache_row.push_back((int) (G * (D + Vd)));
+        widen(hy->w_proj, (rows + 3) & ~(int64_t) 3); widen(hy->w_q, H * D); widen(hy->w_lat, H * Vd); widen(hy->w_conv, H2 * (V2 + 1)); widen(hy->w_cq, 4 * H2);
+        widen(hy->w_att, ((H * Vd + 3) & ~(int64_t) 3) + ((H2 * V2 + 3) & ~(int64_t) 3));
+        // ---- the feed-forward ----
+        if (ml && !ml->is_null()) {
+            const Json * kind = ml->get("kind");
+            if (kind && kind->str != "dense") { pib_set_error("model: layer %d: unknown mlp kind", il); return nullptr; }
+            L.mlp = PIB_MLP_GEGLU; L.ff = (int) jnum(ml, "ff", (double) src.dim(pm + "up", 0, 0));
+            if (L.ff <= 0) { pib_set_error("model: layer %d: mlp.ff", il); return nullptr; }
+            VEC(L.norm2, p + "norm2", W);
+            GET(p + "canon2", W, (int64_t) hy->taps);
+            if (!(L.canon2 = upload_f32v(v))) return nullptr;
+            MAT(L.rg2, p + "rg2", W, W);
+            VEC(L.rg2_b, p + "rg2.b", W);
+            L.tail2_off = state; state += tail;
+            if (!(L.up = upload_gate_up(src, pm, L.ff, W, dtype, m))) return nullptr;
+            MAT(L.down, pm + "down", W, L.ff);
+            widen(hy->w_proj, (int64_t) L.ff);
+        }
+    }
+    hy->state_floats = state ? state : 4;
+#undef GET
+#undef VEC
+#undef MAT
+#undef APPEND
+    return mp.release();
+}
+
 // ---- registry: config.json "architecture" -> builder ---------------------------------------------------------------------------------
 struct DirArch { const char * name; pib_model * (*build)(const Json &, TensorSource &, int); };
-static const DirArch DIR_ARCHS[] = { { "Rapisun", build_rapisun }, { "Fabivik", build_fabivik }, { "Lulenex", build_lulenex }, { "Putazen", build_putazen } };
+static const DirArch DIR_ARCHS[] = { { "Rapisun", build_rapisun }, { "Fabivik", build_fabivik }, { "Lulenex", build_lulenex }, { "Putazen", build_putazen },
+                                     { "Bobunex", build_bobunex } };
 
 static pib_model * build_from_config(const Json & cfg, TensorSource & src, int dtype) {
     const Json * a = cfg.get("architecture");
@@ -956,9 +1096,9 @@ void pib_hybrid_model_free(pib_model * m) {
     for (pib_hlayer & L : hy->layers) {
         if (L.weights_of >= 0) continue;                  // a later walk of the same layer: the tensors are the first walk's
         for (float * f : { L.norm1, L.norm2, L.canon, L.dq_norm, L.dkv_norm, L.sink, L.f_bias, L.lower, L.onorm, L.conv, L.q_norm, L.k_norm, L.mu, L.w0, L.bonus, L.a_log,
-                           L.dt_bias, L.shift, L.conv_b, L.ssm_a, L.ssm_d, L.proj_bias, L.o_bias, L.decay, L.hc1, L.hc2, L.norm1_b, L.norm2_b }) if (f) cudaFree(f);
+                           L.dt_bias, L.shift, L.conv_b, L.ssm_a, L.ssm_d, L.proj_bias, L.o_bias, L.decay, L.hc1, L.hc2, L.norm1_b, L.norm2_b, L.rg1_b, L.rg2_b, L.canon2, L.i_bias, L.out_a, L.out_b }) if (f) cudaFree(f);
         for (pib_weight * w : { L.dqkv, L.uq, L.ukT, L.uv, L.wo, L.qfv, L.up, L.down, L.e_up, L.e_down, L.router, L.s_up, L.s_down, L.qkv, L.rkvg, L.w1, L.w2, L.ssm_in, L.ssm_x,
-                                L.ssm_dt }) if (w) pib_weight_free(w);
+                                L.ssm_dt, L.rg1, L.rg2, L.wo2 }) if (w) pib_weight_free(w);
     }
     if (hy->embd_norm) cudaFree(hy->embd_norm);
     if (hy->final_b) cudaFree(hy->final_b);

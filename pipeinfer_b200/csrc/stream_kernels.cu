@@ -3,7 +3,7 @@
 //   hyper-connections: every token carries S streams X_s [W].  A sublayer reads u = sum_s in_s X_s through a LayerNorm with weight and
 //       bias, and its output y is written back as X_t <- sum_s mix[s][t] X_s + out_t y.  One kernel does the write of the sublayer before
 //       and the read + norm of the next one, so the streams cross memory once per sublayer.
-//   rotation tables with YaRN-scaled frequencies
+//   rotation tables with scaled frequencies (YaRN; bands of wavelengths)
 //   Mamba-2: step sizes and decays per head and token; the gate silu(z) in front of an RMS norm over equal parts of the channels
 //   differential attention: biases + rotation + cache write of q | k | v rows with several maps per head; a1 - lambda a2 and the unit RMS
 #include "hybrid.cuh"
@@ -101,8 +101,16 @@ void pib_rope_table(std::vector<float2> & tab, int n_pos, const pib_hybrid::Rope
     std::vector<double> f((size_t) half);
     double mag = 1.0;
     for (int i = 0; i < half; i++) f[(size_t) i] = pow((double) r.base, -2.0 * i / (double) r.dims);
-    if (r.factor > 0) {
-        const double two_pi = 6.283185307179586476925286766559;
+    const double two_pi = 6.283185307179586476925286766559;
+    if (r.scaling == PIB_ROPE_BANDS) {
+        for (double & v : f) {
+            const double turns = r.original * v / two_pi;
+            if (turns > r.fast) continue;
+            if (turns < r.slow) { v /= r.factor; continue; }
+            const double s = r.fast > r.slow ? (turns - r.slow) / (r.fast - r.slow) : 1.0;
+            v = (1.0 - s) * v / r.factor + s * v;
+        }
+    } else if (r.scaling == PIB_ROPE_YARN) {
         auto dim_of = [&](double turns) { return r.dims * log(r.original / (two_pi * turns)) / (2.0 * log((double) r.base)); };
         const double lo = std::max(floor(dim_of(r.fast)), 0.0), hi = std::min(ceil(dim_of(r.slow)), (double) (r.dims - 1));
         for (int i = 0; i < half; i++) {
