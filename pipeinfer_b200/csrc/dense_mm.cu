@@ -211,6 +211,22 @@ __global__ void __launch_bounds__(256) mv_rows_kernel(mm_dev a, bool xvec) {
     mv_rows_body<WT, ROUND, EPI, B>(a, xvec, z, n, lane, row0, row1);
 }
 
+// two independent few-row matmuls in one launch (decode steps: a launch costs as much as a small matrix): blocks [0, blocks_a) walk a's weight rows,
+// the others b's
+template <typename WT, bool ROUND, int EPI_B, int B>
+__global__ void __launch_bounds__(256) mv_pair_kernel(mm_dev a, mm_dev b, bool xva, bool xvb, int blocks_a) {
+    pib_pdl_wait();
+    pib_pdl_trigger();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, per = blockDim.x >> 5;
+    if ((int) blockIdx.x < blocks_a) {
+        const int n = blockIdx.x * per + warp;
+        if (n < a.N) mv_rows_body<WT, ROUND, PIB_EPI_NONE, B>(a, xva, 0, n, lane, 0, a.M);
+    } else {
+        const int n = (blockIdx.x - blocks_a) * per + warp;
+        if (n < (pib_epi_pairs(EPI_B) ? b.N / 2 : b.N)) mv_rows_body<WT, ROUND, EPI_B, B>(b, xvb, 0, n, lane, 0, b.M);
+    }
+}
+
 // ---- few outputs, many rows (a router's logits over a prompt): one warp per row m, lanes stride over k, NB accumulators per lane ----
 // float32 weights and activations, no rounding; the weight matrix (N x K floats) stays in L1 / L2 while every warp walks it.
 template <int NB>
@@ -287,6 +303,37 @@ int pib_dense_mm(const pib_mm & a, cudaStream_t st) {
 #undef MM_GO
     pib_set_error("dense matmul: weight type %d", a.wtype);
     return PIB_ERR_UNSUPP;
+}
+
+// a (no epilogue) and b (none or PIB_EPI_GEGLU_PAIR) do not depend on each other; up to MV_MAXB rows they share a launch, else they follow one another
+template <typename WT, bool ROUND, int EPI_B>
+static void launch_pair(const mm_dev & a, const mm_dev & b, bool xva, bool xvb, cudaStream_t st) {
+    const int ba = (a.N + 7) / 8, bb = ((pib_epi_pairs(EPI_B) ? b.N / 2 : b.N) + 7) / 8;
+    const dim3 grid((unsigned) (ba + bb));
+    if (a.M == 1)      pib_launch(mv_pair_kernel<WT, ROUND, EPI_B, 1>, grid, dim3(256), (size_t) 0, st, a, b, xva, xvb, ba);
+    else if (a.M == 2) pib_launch(mv_pair_kernel<WT, ROUND, EPI_B, 2>, grid, dim3(256), (size_t) 0, st, a, b, xva, xvb, ba);
+    else if (a.M <= 4) pib_launch(mv_pair_kernel<WT, ROUND, EPI_B, 4>, grid, dim3(256), (size_t) 0, st, a, b, xva, xvb, ba);
+    else if (a.M <= 8) pib_launch(mv_pair_kernel<WT, ROUND, EPI_B, 8>, grid, dim3(256), (size_t) 0, st, a, b, xva, xvb, ba);
+    else               pib_launch(mv_pair_kernel<WT, ROUND, EPI_B, MV_MAXB>, grid, dim3(256), (size_t) 0, st, a, b, xva, xvb, ba);
+}
+int pib_dense_mm_pair(const pib_mm & a, const pib_mm & b, cudaStream_t st) {
+    const int V = a.wtype == PIB_TYPE_BF16 ? 8 : 4;
+    auto plain = [&](const pib_mm & m) { return m.Z == 1 && !m.xrows && !m.zrange && !m.x_bf16 && m.ldw % V == 0 && ((uintptr_t) m.W & 15) == 0; };
+    if (a.M < 1 || a.M > MV_MAXB || a.M != b.M || a.wtype != b.wtype || a.exact != b.exact || !plain(a) || !plain(b) || a.epi != PIB_EPI_NONE ||
+        (b.epi != PIB_EPI_NONE && b.epi != PIB_EPI_GEGLU_PAIR) || (pib_epi_pairs(b.epi) && (b.N & 1)) || (a.exact && a.wtype != PIB_TYPE_F32)) {
+        const int rc = pib_dense_mm(a, st);
+        return rc != PIB_OK ? rc : pib_dense_mm(b, st);
+    }
+    auto dev = [](const pib_mm & m) { return mm_dev{ m.W, m.ldw, m.wz, m.X, m.ldx, m.xz, nullptr, 1, m.Y, m.ldy, m.yz, m.M, m.N, m.K, nullptr, m.e0, m.e1 }; };
+    auto xvec = [](const pib_mm & m) { return m.ldx % 4 == 0 && ((uintptr_t) m.X & 15) == 0; };
+#define PAIR_GO(WT, ROUND) do { if (b.epi == PIB_EPI_NONE) launch_pair<WT, ROUND, PIB_EPI_NONE>(dev(a), dev(b), xvec(a), xvec(b), st); \
+                                else launch_pair<WT, ROUND, PIB_EPI_GEGLU_PAIR>(dev(a), dev(b), xvec(a), xvec(b), st); } while (0)
+    if (a.wtype == PIB_TYPE_BF16) PAIR_GO(__nv_bfloat16, true);
+    else if (a.exact) PAIR_GO(float, false);
+    else PAIR_GO(float, true);
+#undef PAIR_GO
+    PIB_CHECK(cudaGetLastError());
+    return PIB_OK;
 }
 
 pib_weight * pib_dense_upload(int type, const void * host, int64_t N, int64_t K) {

@@ -47,7 +47,7 @@ template <int VEC> __device__ __forceinline__ void gf_store(float * p, const gf_
     else *p = r.v[0];
 }
 template <int VEC, int NV>
-__global__ void __launch_bounds__(1024) gated_norm_kernel(gf_args A) {
+__global__ void __launch_bounds__(NV >= 4 ? 512 : 1024) gated_norm_kernel(gf_args A) {
     pib_pdl_wait();
     pib_pdl_trigger();
     __shared__ float2 red[32];
@@ -142,9 +142,8 @@ int pib_gated_norm(float * x, const pib_sublayer_out & o, const float * w, float
     const int vec = W % 4 == 0 ? 4 : 1, pieces = (W + vec - 1) / vec, want = b.T > 32 ? 256 : 1024;      // decode steps: one piece per thread, as many loads in flight as there are
     int nv = 1;
     while (nv < 8 && (pieces + nv - 1) / nv > want) nv *= 2;
-    while (nv < 8 && (pieces + nv - 1) / nv > 1024) nv *= 2;
     const int threads = ((pieces + nv - 1) / nv + 31) & ~31;
-    if (threads > 1024) { pib_set_error("gated norm: width %d not supported", W); return PIB_ERR_UNSUPP; }
+    if (threads > (nv >= 4 ? 512 : 1024)) { pib_set_error("gated norm: width %d not supported", W); return PIB_ERR_UNSUPP; }
 #define GF_GO(VEC, NV) pib_launch(gated_norm_kernel<VEC, NV>, dim3((unsigned) b.T), dim3((unsigned) threads), (size_t) 0, st, A)
     if (vec == 4) { if (nv == 1) GF_GO(4, 1); else if (nv == 2) GF_GO(4, 2); else if (nv == 4) GF_GO(4, 4); else GF_GO(4, 8); }
     else          { if (nv == 1) GF_GO(1, 1); else if (nv == 2) GF_GO(1, 2); else if (nv == 4) GF_GO(1, 4); else GF_GO(1, 8); }
@@ -154,16 +153,16 @@ int pib_gated_norm(float * x, const pib_sublayer_out & o, const float * w, float
 }
 
 // ---- attention beside a matrix memory: what follows the projections -----------------------------------------------------------------------
-// Blocks [0, T): one token each.  proj[t] = [q (nq = H*D) | k (nk = G*D) | v (nv = G*V) | ...]: q / rms(q) q_norm and k / rms(k) k_norm (one root mean
+// Blocks [S, S + T): one token each.  proj[t] = [q (nq = H*D) | k (nk = G*D) | v (nv = G*V) | ...]: q / rms(q) q_norm and k / rms(k) k_norm (one root mean
 // square over ALL rows of q, one over all of k), then the first rot_dims coordinates of every D-wide row turn (pairs (i, i + rot_dims / 2)); q[t] gets
 // the query rows, the token's cell [k | v].
-// Blocks [T, T + S): the memory's gates of one segment, a warp per head.  i = cap tanh((proj[i_off + h] + i_bias) / cap), f = log sigmoid(cap tanh((proj[f_off + h] +
+// Blocks [0, S) (first, since they take longest): the memory's gates of one segment, a warp per head.  i = cap tanh((proj[i_off + h] + i_bias) / cap), f = log sigmoid(cap tanh((proj[f_off + h] +
 // f_bias) / cap)); the running maximum m' = max(f + m, i) starts from the slot's and is left there.  It composes like a pair (F, M): m -> max(F + m, M),
-// (F1, M1) then (F2, M2) = (F1 + F2, max(M1 + F2, M2)), so a warp takes 32 tokens per trip with an inclusive scan over its lanes.
+// (F1, M1) then (F2, M2) = (F1 + F2, max(M1 + F2, M2)), so a warp takes 32 K tokens per trip: K in a row per lane, an inclusive scan over the lanes.
 // dg[t] = [e^(i - m') (H2) | e^(f + m - m') (H2) | f + m - m' (H2) | e^-m' (H2)].  Every factor is formed from the maxima as stored, so their rounding cancels
 // between the factors of neighbouring tokens.
 struct amp_args {
-    const float * proj; int ldp, T;
+    const float * proj; int ldp, S;
     int nq, nk, nv, D, rot_dims;
     const float * q_norm, * k_norm; float eps;
     const int32_t * pos, * cell; const float2 * rope;
@@ -174,13 +173,14 @@ struct amp_args {
     float * dg;
 };
 __device__ __forceinline__ float gk_capped(float z, float cap) { return cap > 0.f ? cap * tanhf(z / cap) : z; }
-__global__ void __launch_bounds__(1024) attn_mem_prep_kernel(amp_args A) {
+template <int K>
+__global__ void __launch_bounds__(K == 1 ? 1024 : 256) attn_mem_prep_kernel(amp_args A) {
     pib_pdl_wait();
     pib_pdl_trigger();
     __shared__ float2 red[32];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
-    if ((int) blockIdx.x < A.T) {
-        const int t = blockIdx.x, half = A.rot_dims / 2, nqk = A.nq + A.nk;
+    if ((int) blockIdx.x >= A.S) {
+        const int t = blockIdx.x - A.S, half = A.rot_dims / 2, nqk = A.nq + A.nk;
         const float * p = A.proj + (size_t) t * A.ldp;
         float sq = 0.f, sk = 0.f;
         for (int e = threadIdx.x; e < nqk; e += blockDim.x) { const float v = p[e]; if (e < A.nq) sq = fmaf(v, v, sq); else sk = fmaf(v, v, sk); }
@@ -208,32 +208,51 @@ __global__ void __launch_bounds__(1024) attn_mem_prep_kernel(amp_args A) {
         }
         return;
     }
-    const int sg = blockIdx.x - A.T, s0 = A.seg_start[sg], n = A.seg_len[sg], H = A.H2;
+    const int sg = blockIdx.x, s0 = A.seg_start[sg], n = A.seg_len[sg], H = A.H2;
     for (int h = warp; h < H; h += nw) {
         float * mslot = A.state + (size_t) A.seg_slot[sg] * A.state_stride + A.max_off + h;
         float m0 = *mslot;
         const float ib = A.i_bias[h], fb = A.f_bias[h];
-        float zi = lane < n ? A.proj[(size_t) (s0 + lane) * A.ldp + A.i_off + h] : 0.f, zf = lane < n ? A.proj[(size_t) (s0 + lane) * A.ldp + A.f_off + h] : 0.f;
-        for (int t0 = 0; t0 < n; t0 += 32) {
-            const bool ok = t0 + lane < n;
-            const float gi = gk_capped(zi + ib, A.cap), z = gk_capped(zf + fb, A.cap);
-            const float gf = fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
-            const int tn = t0 + 32 + lane;                       // the next trip's logits are on their way while this one is scanned
-            zi = tn < n ? A.proj[(size_t) (s0 + tn) * A.ldp + A.i_off + h] : 0.f; zf = tn < n ? A.proj[(size_t) (s0 + tn) * A.ldp + A.f_off + h] : 0.f;
-            float F = ok ? gf : 0.f, M = ok ? gi : -INFINITY;    // lanes behind the end pass the maximum on unchanged
+        float zi[K], zf[K];
+        auto fetch = [&](int t0) {
+#pragma unroll
+            for (int k = 0; k < K; k++) {
+                const int t = t0 + lane * K + k;
+                const float * p = A.proj + (size_t) (s0 + t) * A.ldp + h;
+                zi[k] = t < n ? p[A.i_off] : 0.f; zf[k] = t < n ? p[A.f_off] : 0.f;
+            }
+        };
+        fetch(0);
+        for (int t0 = 0; t0 < n; t0 += 32 * K) {
+            float gi[K], gf[K];
+            float F = 0.f, M = -INFINITY;                        // tokens behind the end pass the maximum on unchanged
+#pragma unroll
+            for (int k = 0; k < K; k++) {
+                const float z = gk_capped(zf[k] + fb, A.cap);
+                gi[k] = gk_capped(zi[k] + ib, A.cap);
+                gf[k] = fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
+                if (t0 + lane * K + k < n) { M = fmaxf(M + gf[k], gi[k]); F += gf[k]; }
+            }
+            if (t0 + 32 * K < n) fetch(t0 + 32 * K);             // the next trip's logits are on their way while this one is scanned
 #pragma unroll
             for (int o = 1; o < 32; o <<= 1) {
                 const float Fp = __shfl_up_sync(0xffffffffu, F, o), Mp = __shfl_up_sync(0xffffffffu, M, o);
                 if (lane >= o) { M = fmaxf(Mp + F, M); F += Fp; }
             }
-            const float m = fmaxf(F + m0, M);
-            float prev = __shfl_up_sync(0xffffffffu, m, 1);
-            if (lane == 0) prev = m0;
-            m0 = __shfl_sync(0xffffffffu, m, 31);
-            if (ok) {
-                float * d = A.dg + (size_t) (s0 + t0 + lane) * 4 * H + h;
-                const float ld = (gf + prev) - m;
-                d[0] = expf(gi - m); d[H] = expf(ld); d[2 * H] = ld; d[3 * H] = expf(-m);
+            const float last = fmaxf(F + m0, M);
+            float m = __shfl_up_sync(0xffffffffu, last, 1);      // the maximum in front of this lane's tokens
+            if (lane == 0) m = m0;
+            m0 = __shfl_sync(0xffffffffu, last, 31);
+#pragma unroll
+            for (int k = 0; k < K; k++) {
+                const int t = t0 + lane * K + k;
+                if (t < n) {
+                    // the lane's last token takes the scan's number, so that the next lane's first factor starts from the same one
+                    const float mn = k == K - 1 ? last : fmaxf(gf[k] + m, gi[k]), ld = (gf[k] + m) - mn;
+                    float * d = A.dg + (size_t) (s0 + t) * 4 * H + h;
+                    d[0] = expf(gi[k] - mn); d[H] = expf(ld); d[2 * H] = ld; d[3 * H] = expf(-mn);
+                    m = mn;
+                }
             }
         }
         if (lane == 0) *mslot = m0;
@@ -242,10 +261,11 @@ __global__ void __launch_bounds__(1024) attn_mem_prep_kernel(amp_args A) {
 int pib_attn_mem_prep(const float * proj, int ldp, int i_off, int f_off, const pib_hlayer & L, float eps, const pib_hbatch & b, const float2 * rope, float * q, float * cache,
                       int cache_row, float * state, size_t state_stride, float * dg, cudaStream_t st) {
     const int nq = L.heads * L.dim, nk = L.kv_heads * L.dim, nv = L.kv_heads * L.vdim, n_all = nq + nk + nv;
-    amp_args A = { proj, ldp, b.T, nq, nk, nv, L.dim, L.rot_dims, L.q_norm, L.k_norm, eps, b.pos, b.cell, rope, q, cache, cache_row, L.heads2, i_off, f_off, L.i_bias, L.f_bias,
+    amp_args A = { proj, ldp, b.S, nq, nk, nv, L.dim, L.rot_dims, L.q_norm, L.k_norm, eps, b.pos, b.cell, rope, q, cache, cache_row, L.heads2, i_off, f_off, L.i_bias, L.f_bias,
                    L.gate_cap, b.seg_start, b.seg_len, b.seg_slot, state, state_stride, L.max_off, dg };
-    const int threads = b.T > 32 ? 256 : n_all >= 2048 ? 1024 : n_all >= 1024 ? 512 : 256;
-    pib_launch(attn_mem_prep_kernel, dim3((unsigned) (b.T + b.S)), dim3(threads), (size_t) 0, st, A);
+    const int threads = b.T > 32 || b.T > b.S ? 256 : n_all >= 2048 ? 1024 : n_all >= 1024 ? 512 : 256;
+    if (b.T == b.S) pib_launch(attn_mem_prep_kernel<1>, dim3((unsigned) (b.T + b.S)), dim3(threads), (size_t) 0, st, A);
+    else            pib_launch(attn_mem_prep_kernel<8>, dim3((unsigned) (b.T + b.S)), dim3(threads), (size_t) 0, st, A);
     CKL();
     return PIB_OK;
 }

@@ -57,13 +57,13 @@ static const char * const HK_NAMES[] = { "cellmap", "embed_ln", "canon_conv", "m
                                          "mm_dual_proj", "dual_prep", "decay_scan", "dual_gate", "mm_dual_o",
                                          "hyper_norm", "mm_mamba2_in", "mamba2_conv", "mamba2_prep", "mamba2_scan", "gated_group_norm", "mm_mamba2_o", "qkv_rope", "diff_combine",
                                          "mm_gate_up",
-                                         "gated_norm", "input_conv", "mm_res_gate", "mm_attn_mem_proj", "attn_mem_prep", "memory_scan", "attn_mem_gate", "mm_attn_mem_o" };
+                                         "gated_norm", "input_conv", "mm_res_gate", "mm_attn_mem_proj", "attn_mem_prep", "memory_scan", "attn_mem_gate", "mm_attn_mem_o", "mm_gate_pair" };
 enum { HK_CELLMAP, HK_EMBED, HK_CANON, HK_DQKV, HK_LPREP, HK_UQ, HK_ABSORB, HK_LATTN, HK_UV, HK_AO, HK_QFV, HK_GATES, HK_SCAN, HK_HO, HK_LNRES, HK_UP, HK_POLY, HK_DOWN,
        HK_ROUTER, HK_ROUTE, HK_SORT, HK_EUP, HK_EDOWN, HK_SUP, HK_SDOWN, HK_COMBINE, HK_FINAL, HK_HEAD, HK_SAMPLE, HK_LATTN_MM,
        HK_EMBSCALE, HK_NORM2, HK_QKV, HK_QKVCONV, HK_APREP, HK_KVATTN, HK_KVATTN_MM, HK_SHIFT, HK_RKVG, HK_DECAY, HK_DECAYACT, HK_WKVSCAN, HK_DPREP, HK_DSCAN, HK_GHNORM, HK_GLU,
        HK_PSUM, HK_EMBPAIR, HK_PRENORM, HK_CONCAT, HK_LOOPIN, HK_SSMIN, HK_SSMCONV, HK_SSMX, HK_SSMDT, HK_SSMSCAN, HK_SSMO, HK_DUALPROJ, HK_DUALPREP, HK_DECAYSCAN, HK_DUALGATE,
        HK_DUALO, HK_HYPER, HK_M2IN, HK_M2CONV, HK_M2PREP, HK_M2SCAN, HK_GGNORM, HK_M2O, HK_QKVROPE, HK_DIFFCOMB, HK_GATEUP,
-       HK_GNORM, HK_INCONV, HK_RGATE, HK_AMPROJ, HK_AMPREP, HK_MEMSCAN, HK_AMGATE, HK_AMO, HK_COUNT };
+       HK_GNORM, HK_INCONV, HK_RGATE, HK_AMPROJ, HK_AMPREP, HK_MEMSCAN, HK_AMGATE, HK_AMO, HK_GATE_PAIR, HK_COUNT };
 const char * pib_hybrid_kind_name(int k) { return k >= 0 && k < HK_COUNT ? HK_NAMES[k] : "?"; }
 
 // fetch and clear the records; returns the count (the stream is synchronised)
@@ -241,12 +241,25 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
         for (int i = 0; i < T; i++) n += mask == PIB_MASK_CHUNK ? B_pos_host[i] % window + 1 : std::min<int64_t>(B_pos_host[i] + 1, (int64_t) window + keep);
         return n;
     };
-    auto mm = [&](const pib_weight * w, const float * X, int ldx, float * Y, int ldy, int epi, float e0 = 0.f, float e1 = 0.f) {
+    auto mm_of = [&](const pib_weight * w, const float * X, int ldx, float * Y, int ldy, int epi, float e0 = 0.f, float e1 = 0.f) {
         pib_mm a;
         a.W = w->base; a.wtype = w->type; a.ldw = w->K; a.X = X; a.ldx = ldx; a.Y = Y; a.ldy = ldy; a.M = T; a.N = (int) w->N; a.K = (int) w->K; a.epi = epi;
         a.e0 = e0; a.e1 = e1;
         a.exact = exact || w->type == PIB_TYPE_F32;
-        return pib_dense_mm(a, st);
+        return a;
+    };
+    auto mm = [&](const pib_weight * w, const float * X, int ldx, float * Y, int ldy, int epi, float e0 = 0.f, float e1 = 0.f) { return pib_dense_mm(mm_of(w, X, ldx, Y, ldy, epi, e0, e1), st); };
+    // gated frame: the residual gate's matmul x->rg = R x->h shares a launch with the sublayer's first one in decode steps
+    const bool pairs = T <= 16;
+    const pib_weight * gate_w = nullptr;              // a gate whose matmul is still to be launched
+    auto with_gate = [&](int kind, double fl, double by, const pib_mm & b) -> int {
+        if (gate_w && pairs) { RC(HK_GATE_PAIR, fl + mmfl(gate_w), by + mmby(gate_w), pib_dense_mm_pair(mm_of(gate_w, x->h, W, x->rg, W, PIB_EPI_NONE), b, st)); }
+        else {
+            if (gate_w) RC(HK_RGATE, mmfl(gate_w), mmby(gate_w), mm(gate_w, x->h, W, x->rg, W, PIB_EPI_NONE));
+            RC(kind, fl, by, pib_dense_mm(b, st));
+        }
+        gate_w = nullptr;
+        return PIB_OK;
     };
     // ---- mixers: read hin [T][W], leave their output in x->y ----
     auto mixer_latent = [&](const pib_hlayer & L, const float * hin) -> int {
@@ -463,7 +476,7 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
         const int ldp = ((int) L.qkv->N + 3) & ~3, q2 = (H + G) * D + G * V, k2 = q2 + H2 * D2, v2 = k2 + H2 * D2, og = v2 + H2 * V2, hg = og + H2 * V2, gi = hg + H, gf = gi + H2;
         const int mem_off = (H * V + 3) & ~3, ldo = (mem_off + H2 * V2 + 3) & ~3;
         float * cache = x->cache[L.cache_id];
-        RC(HK_AMPROJ, mmfl(L.qkv), mmby(L.qkv), mm(L.qkv, hin, W, x->proj, ldp, PIB_EPI_NONE));
+        if ((rc = with_gate(HK_AMPROJ, mmfl(L.qkv), mmby(L.qkv), mm_of(L.qkv, hin, W, x->proj, ldp, PIB_EPI_NONE))) != PIB_OK) return rc;
         RC(HK_AMPREP, 0, 4.0 * Td * (2.0 * q2 + 6.0 * H2), pib_attn_mem_prep(x->proj, ldp, gi, gf, L, eps, B, x->rope[L.rope_id], x->q, cache, row, x->state, hy->state_floats, x->cq, st));
         if ((rc = kv_attend(L, cache, row, x->lat)) != PIB_OK) return rc;
         int parts = 0, per = 0;
@@ -472,8 +485,12 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
            pib_memory_scan(x->proj, ldp, q2, k2, v2, x->cq, L, B, x->state, hy->state_floats, x->cv, st, x->split_buf, parts, per));
         nk += parts ? 4 : 0;
         RC(HK_AMGATE, 0, 4.0 * Td * (2.0 * H * V + 3.0 * H2 * V2 + 2.0 * H2 + H), pib_attn_mem_gate(x->lat, x->cv, x->cq, x->proj, ldp, hg, og, L, eps, T, x->att, ldo, mem_off, st));
-        RC(HK_AMO, mmfl(L.wo), mmby(L.wo), mm(L.wo, x->att, ldo, x->y, W, PIB_EPI_NONE));
-        RC(HK_AMO, mmfl(L.wo2), mmby(L.wo2), mm(L.wo2, x->att + mem_off, ldo, x->y2, W, PIB_EPI_NONE));
+        if (pairs) RC(HK_AMO, mmfl(L.wo) + mmfl(L.wo2), mmby(L.wo) + mmby(L.wo2),
+                      pib_dense_mm_pair(mm_of(L.wo, x->att, ldo, x->y, W, PIB_EPI_NONE), mm_of(L.wo2, x->att + mem_off, ldo, x->y2, W, PIB_EPI_NONE), st));
+        else {
+            RC(HK_AMO, mmfl(L.wo), mmby(L.wo), mm(L.wo, x->att, ldo, x->y, W, PIB_EPI_NONE));
+            RC(HK_AMO, mmfl(L.wo2), mmby(L.wo2), mm(L.wo2, x->att + mem_off, ldo, x->y2, W, PIB_EPI_NONE));
+        }
         return PIB_OK;
     };
     auto run_mixer = [&](const pib_hlayer & L, const float * hin) -> int {
@@ -562,14 +579,15 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
         int lds = 0;
         if (hy->form == PIB_FORM_GATED) {
             if ((rc = gated(L.norm1, L.canon, L.tail_off)) != PIB_OK) return rc;
-            RC(HK_RGATE, mmfl(L.rg1), mmby(L.rg1), mm(L.rg1, x->h, W, x->rg, W, PIB_EPI_NONE));
+            gate_w = L.rg1;
+            if (L.mixer != PIB_MIXER_ATTN_MEM) { RC(HK_RGATE, mmfl(L.rg1), mmby(L.rg1), mm(L.rg1, x->h, W, x->rg, W, PIB_EPI_NONE)); gate_w = nullptr; }      // the other mixers launch their matmuls alone
             if ((rc = run_mixer(L, x->h2)) != PIB_OK) return rc;
             left.ya = x->y; left.gl = x->rg; left.gb = L.rg1_b;
             if (L.wo2) { left.wa = L.out_a; left.yb = x->y2; left.wb = L.out_b; left.mix = L.mix_a; }
             if (L.mlp == PIB_MLP_GEGLU) {
                 if ((rc = gated(L.norm2, L.canon2, L.tail2_off)) != PIB_OK) return rc;
-                RC(HK_RGATE, mmfl(L.rg2), mmby(L.rg2), mm(L.rg2, x->h, W, x->rg, W, PIB_EPI_NONE));
-                RC(HK_GATEUP, mmfl(L.up), wbytes(L.up) + 4.0 * Td * (Wd + L.ff), mm(L.up, x->h2, W, x->proj, L.ff, PIB_EPI_GEGLU_PAIR));
+                gate_w = L.rg2;
+                if ((rc = with_gate(HK_GATEUP, mmfl(L.up), wbytes(L.up) + 4.0 * Td * (Wd + L.ff), mm_of(L.up, x->h2, W, x->proj, L.ff, PIB_EPI_GEGLU_PAIR))) != PIB_OK) return rc;
                 RC(HK_DOWN, mmfl(L.down), mmby(L.down), mm(L.down, x->proj, L.ff, x->y, W, PIB_EPI_NONE));
                 left.ya = x->y; left.gl = x->rg; left.gb = L.rg2_b;
             } else if (L.mlp != PIB_MLP_NONE) { pib_set_error("decode: feed-forward %d in a gated layer", L.mlp); return PIB_ERR_UNSUPP; }

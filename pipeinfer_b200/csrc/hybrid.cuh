@@ -245,6 +245,7 @@ template <int EPI, bool FAST> __device__ __forceinline__ float pib_glu_pair(floa
 }
 #endif
 int pib_dense_mm(const pib_mm & a, cudaStream_t st);
+int pib_dense_mm_pair(const pib_mm & a, const pib_mm & b, cudaStream_t st);   // two independent matmuls; in decode steps one launch
 int pib_dense_mm_check(cudaStream_t st, int enqueue);   // dense_mma.cu: the error word of the bounded waits (1: copy it in stream order, 0: read the copy)
 pib_weight * pib_dense_upload(int type, const void * host, int64_t N, int64_t K);   // type: PIB_TYPE_BF16 / PIB_TYPE_F32, row-major [N][K]
 

@@ -108,6 +108,49 @@ __global__ void __launch_bounds__(256) canon_kernel(const float * __restrict__ x
     }
 }
 
+// the same for prompts: a thread takes one channel of CANON_RUN tokens in a row, all inputs of the run in flight at once, each read once (and
+// the taps - 1 in front of the run again)
+#define CANON_RUN 8
+template <int TAPS>
+__global__ void __launch_bounds__(256) canon_run_kernel(const float * __restrict__ x, int ldu, const float * __restrict__ w, const int32_t * __restrict__ seg, const int32_t * __restrict__ seg_start,
+                                                        const int32_t * __restrict__ seg_slot, const float * __restrict__ state, size_t state_stride, size_t tail_off, int T, int W,
+                                                        float * __restrict__ h, int ldo, int flags, const float * __restrict__ bias) {
+    pib_pdl_wait();
+    pib_pdl_trigger();
+    const int t0 = blockIdx.x * CANON_RUN, c = blockIdx.y * blockDim.x + threadIdx.x;
+    if (c >= W) return;
+    float in[TAPS - 1 + CANON_RUN], wc[TAPS];
+    const int first = seg_start[seg[t0]];
+#pragma unroll
+    for (int k = 0; k < TAPS - 1 + CANON_RUN; k++) {
+        const int tau = t0 - (TAPS - 1) + k;
+        in[k] = (tau < T && (k >= TAPS - 1 || tau >= first)) ? x[(size_t) tau * ldu + c] : 0.f;
+    }
+#pragma unroll
+    for (int j = 0; j < TAPS; j++) wc[j] = w[(size_t) c * TAPS + j];
+    const float b = bias ? bias[c] : 0.f;
+#pragma unroll
+    for (int r = 0; r < CANON_RUN; r++) {
+        const int t = t0 + r;
+        if (t >= T) break;
+        const int sg = seg[t], s0 = seg_start[sg];
+        float acc = ((flags & CONV_ADD_INPUT) ? in[TAPS - 1 + r] : 0.f) + b;
+        if (t - (TAPS - 1) >= s0) {
+#pragma unroll
+            for (int j = 0; j < TAPS; j++) acc = fmaf(wc[j], in[r + j], acc);
+        } else {
+            const float * tail = state + (size_t) seg_slot[sg] * state_stride + tail_off;
+#pragma unroll
+            for (int j = 0; j < TAPS; j++) {
+                const int tau = t - (TAPS - 1) + j;
+                acc = fmaf(wc[j], tau >= s0 ? in[r + j] : tail[(size_t) (TAPS - 1 + tau - s0) * W + c], acc);
+            }
+        }
+        if (flags & CONV_SILU) acc = acc / (1.0f + expf(-acc));
+        h[(size_t) t * ldo + c] = acc;
+    }
+}
+
 // after canon_kernel, when some segment has more than one token: the last taps-1 inputs of every segment become its slot's tail (old tail
 // rows move up when the segment is shorter)
 __global__ void __launch_bounds__(256) canon_tail_kernel(const float * __restrict__ x, int ldu, int taps, const int32_t * __restrict__ seg_start, const int32_t * __restrict__ seg_len,
@@ -139,7 +182,13 @@ int pib_chan_conv(const float * u, int ldu, const float * w, int taps, const pib
     const int flags = (add_input ? CONV_ADD_INPUT : 0) | (silu ? CONV_SILU : 0) | (b.T == b.S ? CONV_MOVE_TAIL : 0);
     // few tokens (decode steps): a token's channels go to several blocks, so that more than a handful of SMs have loads in flight
     const unsigned ny = b.T > 32 ? 1u : (unsigned) std::min(16, (C + 255) / 256);
-    pib_launch(canon_kernel, dim3((unsigned) b.T, ny), dim3(256), (size_t) (0), st, u, ldu, w, taps, b.seg, b.seg_start, b.seg_slot, state, state_stride, tail_off, C, out, ldo, flags, bias);
+    const dim3 runs((unsigned) ((b.T + CANON_RUN - 1) / CANON_RUN), (unsigned) ((C + 255) / 256));
+#define CANON_GO(TAPS) pib_launch(canon_run_kernel<TAPS>, runs, dim3(256), (size_t) 0, st, u, ldu, w, b.seg, b.seg_start, b.seg_slot, (const float *) state, state_stride, tail_off, b.T, C, out, ldo, flags, bias)
+    if (b.T > 32 && b.T > b.S && taps == 2) CANON_GO(2);
+    else if (b.T > 32 && b.T > b.S && taps == 3) CANON_GO(3);
+    else if (b.T > 32 && b.T > b.S && taps == 4) CANON_GO(4);
+#undef CANON_GO
+    else pib_launch(canon_kernel, dim3((unsigned) b.T, ny), dim3(256), (size_t) (0), st, u, ldu, w, taps, b.seg, b.seg_start, b.seg_slot, state, state_stride, tail_off, C, out, ldo, flags, bias);
     CKL();
     if (taps > 1 && b.T > b.S) { pib_launch(canon_tail_kernel, dim3(b.S), dim3(256), (size_t) (0), st, u, ldu, taps, b.seg_start, b.seg_len, b.seg_slot, state, state_stride, tail_off, C); CKL(); }
     return PIB_OK;

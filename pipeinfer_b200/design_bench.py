@@ -1,9 +1,10 @@
-"""`bench.py --design rapisun | fabivik | lulenex | putazen`: prefill and decode throughput of a layer-list design at sizes that resemble a real
+"""`bench.py --design rapisun | fabivik | lulenex | putazen | bobunex`: prefill and decode throughput of a layer-list design at sizes that resemble a real
 model's layers (random weights drawn in the loader from a seed), beside the closest existing model of the library at equal width / depth /
 vocabulary -- for Rapisun the llama architecture in Q4_K (prompts on its tcgen05 GEMM, decoding on its tensor-core GEMVs), for Fabivik
 the Rapisun design (the other layer-list model: same runtime, same dense matmuls), for Lulenex the Fabivik design (attention over cached
 key / value heads and recurrences on the same kernels), for Putazen the Lulenex design (a state-space scan beside attention over cached
-key / value heads, a dense feed-forward in every layer, a layer walked twice) -- plus the share and the roofline fraction of every kind of launch.  Everything goes through llama_decode on host batches; times are medians of CUDA-side
+key / value heads, a dense feed-forward in every layer, a layer walked twice), for Bobunex the Lulenex design too (softmax attention beside a
+linear recurrence in one mixer) -- plus the share and the roofline fraction of every kind of launch.  Everything goes through llama_decode on host batches; times are medians of CUDA-side
 work as seen by the caller (llama_decode returns after the run's event), the per-kind numbers come from CUDA events around each
 launch (llama_pib_profile_layer).  One JSON line on stdout."""
 import ctypes as C
@@ -80,9 +81,18 @@ def putazen_config(width, vocab, blocks, heads, ff, kv_rank, **_):
             "loop": {"start": 1, "stop": 2, "times": 2}}
 
 
+def bobunex_config(width, vocab, blocks, heads, window, ff, **_):
+    """4 * blocks layers: windowed attention with kept first tokens beside a matrix memory, a gelu-gated feed-forward in every layer"""
+    two = {"left": {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "mask": {"size": window, "keep_first": 4}, "softcap": 50.0,
+                    "rot": {"base": 500000.0, "dims": 64, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}}, "scale": 1.0 / math.sqrt(128)},
+           "right": {"heads": max(1, heads // 2), "dim": 128, "vdim": 128, "gate_cap": 15.0}}
+    return {"architecture": "Bobunex", "width": width, "vocab": vocab, "canon": {"taps": 4}, "norm": {"eps": 1e-5}, "embedding": {"scale": 1.0},
+            "layers": [{"type": "parallel", "mixer": two, "mlp": {"kind": "dense", "ff": ff}}] * (4 * blocks)}
+
+
 # design -> (its name, its configuration, the comparator's key)
 DESIGNS = {"rapisun": ("Rapisun", design_config, "llama_q4k"), "fabivik": ("Fabivik", fabivik_config, "rapisun"), "lulenex": ("Lulenex", lulenex_config, "fabivik"),
-           "putazen": ("Putazen", putazen_config, "lulenex")}
+           "putazen": ("Putazen", putazen_config, "lulenex"), "bobunex": ("Bobunex", bobunex_config, "lulenex")}
 COMPARATORS = {"llama_q4k": "llama architecture, Q4_K", "rapisun": "Rapisun (layer-list design of this library), same width / depth / vocabulary / experts",
                "fabivik": "Fabivik (layer-list design of this library), same width / layer runs / vocabulary",
                "lulenex": "Lulenex (layer-list design of this library), same width / layer runs / vocabulary / feed-forward width"}
