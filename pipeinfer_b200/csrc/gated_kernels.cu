@@ -153,16 +153,17 @@ int pib_gated_norm(float * x, const pib_sublayer_out & o, const float * w, float
 }
 
 // ---- attention beside a matrix memory: what follows the projections -----------------------------------------------------------------------
-// Blocks [S, S + T): one token each.  proj[t] = [q (nq = H*D) | k (nk = G*D) | v (nv = G*V) | ...]: q / rms(q) q_norm and k / rms(k) k_norm (one root mean
+// Tokens (attn_rows_kernel; in batches of single tokens blocks of attn_mem_prep_kernel): one block each.  proj[t] = [q (nq = H*D) | k (nk = G*D) | v (nv = G*V) | ...]: q / rms(q) q_norm and k / rms(k) k_norm (one root mean
 // square over ALL rows of q, one over all of k), then the first rot_dims coordinates of every D-wide row turn (pairs (i, i + rot_dims / 2)); q[t] gets
 // the query rows, the token's cell [k | v].
-// Blocks [0, S) (first, since they take longest): the memory's gates of one segment, a warp per head.  i = cap tanh((proj[i_off + h] + i_bias) / cap), f = log sigmoid(cap tanh((proj[f_off + h] +
+// Gates (attn_mem_prep_kernel): a block takes a few heads of one segment.  i = cap tanh((proj[i_off + h] + i_bias) / cap), f = log sigmoid(cap tanh((proj[f_off + h] +
 // f_bias) / cap)); the running maximum m' = max(f + m, i) starts from the slot's and is left there.  It composes like a pair (F, M): m -> max(F + m, M),
-// (F1, M1) then (F2, M2) = (F1 + F2, max(M1 + F2, M2)), so a warp takes 32 K tokens per trip: K in a row per lane, an inclusive scan over the lanes.
+// (F1, M1) then (F2, M2) = (F1 + F2, max(M1 + F2, M2)), so a warp takes 32 K tokens per trip: K in a row per lane, an inclusive scan over the lanes (and, with
+// several warps per head, over the warps).
 // dg[t] = [e^(i - m') (H2) | e^(f + m - m') (H2) | f + m - m' (H2) | e^-m' (H2)].  Every factor is formed from the maxima as stored, so their rounding cancels
 // between the factors of neighbouring tokens.
 struct amp_args {
-    const float * proj; int ldp, S;
+    const float * proj; int ldp, gate_blocks, groups;
     int nq, nk, nv, D, rot_dims;
     const float * q_norm, * k_norm; float eps;
     const int32_t * pos, * cell; const float2 * rope;
@@ -173,99 +174,182 @@ struct amp_args {
     float * dg;
 };
 __device__ __forceinline__ float gk_capped(float z, float cap) { return cap > 0.f ? cap * tanhf(z / cap) : z; }
-template <int K>
+// one token: a warp per head row, VEC neighbouring coordinates per lane
+template <int VEC>
+__device__ __forceinline__ void amp_token(const amp_args & A, int t, float2 * red) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5, D = A.D, half = A.rot_dims / 2, nqk = A.nq + A.nk;
+    const float * p = A.proj + (size_t) t * A.ldp;
+    float sq = 0.f, sk = 0.f;
+    for (int e = threadIdx.x * VEC; e < nqk; e += blockDim.x * VEC) {
+        const gf_vec<VEC> v = gf_load<VEC>(p + e);
+        float s = 0.f;
+#pragma unroll
+        for (int i = 0; i < VEC; i++) s = fmaf(v.v[i], v.v[i], s);
+        if (e < A.nq) sq += s; else sk += s;
+    }
+    const float2 s = gk_block_sum2(sq, sk, red);
+    const float rq = 1.0f / sqrtf(s.x / A.nq + A.eps), rk = 1.0f / sqrtf(s.y / A.nk + A.eps);
+    const float2 * cs = A.rope + (size_t) A.pos[t] * half;
+    float * row = A.cache + (size_t) A.cell[t] * A.cache_row;
+    for (int e0 = warp * D; e0 < nqk; e0 += nw * D) {
+        const bool    isq = e0 < A.nq;
+        const float * w   = isq ? A.q_norm + e0 : A.k_norm + (e0 - A.nq), * src = p + e0;
+        float *       dst = isq ? A.q + (size_t) t * A.nq + e0 : row + (e0 - A.nq);
+        const float   r   = isq ? rq : rk;
+        for (int i = lane * VEC; i < D; i += 32 * VEC) {
+            gf_vec<VEC> v = gf_load<VEC>(src + i);
+            const gf_vec<VEC> wv = gf_load<VEC>(w + i);
+#pragma unroll
+            for (int j = 0; j < VEC; j++) v.v[j] = v.v[j] * r * wv.v[j];
+            if (i < A.rot_dims) {
+                const bool first = i < half;
+                const int  pi = first ? i + half : i - half, ci = first ? i : pi;
+                const gf_vec<VEC> o = gf_load<VEC>(src + pi), wo = gf_load<VEC>(w + pi);
+#pragma unroll
+                for (int j = 0; j < VEC; j++) {
+                    const float2 c = cs[ci + j];
+                    const float  x = o.v[j] * r * wo.v[j];
+                    v.v[j] = first ? v.v[j] * c.x - x * c.y : v.v[j] * c.x + x * c.y;
+                }
+            }
+            gf_store<VEC>(dst + i, v);
+        }
+    }
+    for (int e = threadIdx.x * VEC; e < A.nv; e += blockDim.x * VEC) gf_store<VEC>(row + A.nk + e, gf_load<VEC>(p + nqk + e));
+}
+// K == 1: tokens and gates of a batch of single tokens; K == 8: the gates alone
+template <int K, int VEC>
 __global__ void __launch_bounds__(K == 1 ? 1024 : 256) attn_mem_prep_kernel(amp_args A) {
     pib_pdl_wait();
     pib_pdl_trigger();
-    __shared__ float2 red[32];
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
-    if ((int) blockIdx.x >= A.S) {
-        const int t = blockIdx.x - A.S, half = A.rot_dims / 2, nqk = A.nq + A.nk;
-        const float * p = A.proj + (size_t) t * A.ldp;
-        float sq = 0.f, sk = 0.f;
-        for (int e = threadIdx.x; e < nqk; e += blockDim.x) { const float v = p[e]; if (e < A.nq) sq = fmaf(v, v, sq); else sk = fmaf(v, v, sk); }
-        const float2 s = gk_block_sum2(sq, sk, red);
-        const float rq = 1.0f / sqrtf(s.x / A.nq + A.eps), rk = 1.0f / sqrtf(s.y / A.nk + A.eps);
-        const float2 * cs = A.rope + (size_t) A.pos[t] * half;
-        float * row = A.cache + (size_t) A.cell[t] * A.cache_row;
-        for (int e = threadIdx.x; e < nqk + A.nv; e += blockDim.x) {
-            float v = p[e];
-            if (e < nqk) {
-                const bool    isq = e < A.nq;
-                const float * w = isq ? A.q_norm : A.k_norm - A.nq;
-                const float   r = isq ? rq : rk;
-                const int     i = (isq ? e : e - A.nq) % A.D;
-                v = v * r * w[e];
-                if (i < A.rot_dims) {
-                    const bool   first = i < half;
-                    const int    pe = first ? e + half : e - half;
-                    const float2 c = cs[first ? i : i - half];
-                    const float  o = p[pe] * r * w[pe];
-                    v = first ? v * c.x - o * c.y : v * c.x + o * c.y;
-                }
-            }
-            if (e < A.nq) A.q[(size_t) t * A.nq + e] = v; else row[e - A.nq] = v;
-        }
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    if (K == 1 && (int) blockIdx.x >= A.gate_blocks) {
+        __shared__ float2 red[32];
+        amp_token<VEC>(A, blockIdx.x - A.gate_blocks, red);
         return;
     }
-    const int sg = blockIdx.x, s0 = A.seg_start[sg], n = A.seg_len[sg], H = A.H2;
-    for (int h = warp; h < H; h += nw) {
-        float * mslot = A.state + (size_t) A.seg_slot[sg] * A.state_stride + A.max_off + h;
-        float m0 = *mslot;
-        const float ib = A.i_bias[h], fb = A.f_bias[h];
-        float zi[K], zf[K];
-        auto fetch = [&](int t0) {
+    // K == 1 (single tokens): a block takes 8 heads of one segment, a warp per head.  K == 8: a block takes two heads, four warps each on neighbouring runs of
+    // 256 tokens; logits come in, and factors leave, through shared memory with neighbouring lanes on neighbouring heads
+    static_assert(K == 1 || K == 8, "tokens per lane");
+    constexpr int WPH = K == 1 ? 1 : 4, HPB = 8 / WPH, RUN = 32 * K, TT = WPH * RUN, PITCH = TT + TT / 8 + 1;      // token t sits at t + t / 8: a lane's 8 tokens start 9 words behind its neighbour's
+    __shared__ float buf[K == 1 ? 1 : 4 * HPB * PITCH];
+    __shared__ float2 agg[8];
+    if (warp >= 8) return;                                       // (only K == 1 has more threads, and no barrier below)
+    const int sg = blockIdx.x / A.groups, h0 = (blockIdx.x % A.groups) * HPB, s0 = A.seg_start[sg], n = A.seg_len[sg], H = A.H2;
+    const int hw = warp / WPH, part = warp % WPH, h = h0 + hw;   // this warp's head and its run of every tile
+    if (K == 1 && h >= H) return;
+    float * mslot = A.state + (size_t) A.seg_slot[sg] * A.state_stride + A.max_off + (h < H ? h : 0);
+    float m0 = *mslot;
+    const float ib = A.i_bias[h < H ? h : 0], fb = A.f_bias[h < H ? h : 0];
+    const int hl = threadIdx.x % HPB, tl = threadIdx.x / HPB;    // staging: head, first token (steps of 256 / HPB tokens)
+    constexpr int STEP = 256 / HPB, NS = K == 1 ? 1 : TT / STEP;
+    float pi[NS], pf[NS];
+    auto fetch = [&](int t0) {
 #pragma unroll
-            for (int k = 0; k < K; k++) {
-                const int t = t0 + lane * K + k;
-                const float * p = A.proj + (size_t) (s0 + t) * A.ldp + h;
-                zi[k] = t < n ? p[A.i_off] : 0.f; zf[k] = t < n ? p[A.f_off] : 0.f;
+        for (int k = 0; k < NS; k++) {
+            const int  t  = K == 1 ? t0 + lane : t0 + tl + STEP * k, hh = K == 1 ? h : h0 + hl;
+            const bool ok = t < n && hh < H;
+            const float * p = A.proj + (size_t) (s0 + t) * A.ldp + hh;
+            pi[k] = ok ? p[A.i_off] : 0.f; pf[k] = ok ? p[A.f_off] : 0.f;
+        }
+    };
+    fetch(0);
+    for (int t0 = 0; t0 < n; t0 += TT) {
+        float gi[K], gf[K];
+        const int  base = part * RUN + lane * K;                 // this lane's first token of the tile
+        const int  pos  = hw * PITCH + base + base / 8;
+        if (K > 1) {
+            __syncthreads();                                     // the trip before has left the buffer
+#pragma unroll
+            for (int k = 0; k < NS; k++) {
+                const int t = tl + STEP * k;
+                buf[hl * PITCH + t + t / 8] = pi[k]; buf[(HPB + hl) * PITCH + t + t / 8] = pf[k];
             }
-        };
-        fetch(0);
-        for (int t0 = 0; t0 < n; t0 += 32 * K) {
-            float gi[K], gf[K];
-            float F = 0.f, M = -INFINITY;                        // tokens behind the end pass the maximum on unchanged
+            __syncthreads();
+        }
+        float F = 0.f, M = -INFINITY;                            // tokens behind the end pass the maximum on unchanged
 #pragma unroll
-            for (int k = 0; k < K; k++) {
-                const float z = gk_capped(zf[k] + fb, A.cap);
-                gi[k] = gk_capped(zi[k] + ib, A.cap);
-                gf[k] = fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
-                if (t0 + lane * K + k < n) { M = fmaxf(M + gf[k], gi[k]); F += gf[k]; }
+        for (int k = 0; k < K; k++) {
+            const float zi = K == 1 ? pi[0] : buf[pos + k], zf = K == 1 ? pf[0] : buf[HPB * PITCH + pos + k];
+            const float z = gk_capped(zf + fb, A.cap);
+            gi[k] = gk_capped(zi + ib, A.cap);
+            gf[k] = fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
+            if (t0 + base + k < n) { M = fmaxf(M + gf[k], gi[k]); F += gf[k]; }
+        }
+        if (t0 + TT < n) fetch(t0 + TT);                         // the next trip's logits are on their way while this one is scanned
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const float Fp = __shfl_up_sync(0xffffffffu, F, o), Mp = __shfl_up_sync(0xffffffffu, M, o);
+            if (lane >= o) { M = fmaxf(Mp + F, M); F += Fp; }
+        }
+        float in = m0;                                           // the maximum in front of this warp's run
+        if (K > 1) {
+            if (lane == 31) agg[warp] = make_float2(F, M);
+            __syncthreads();                                     // (and every warp has read its logits)
+            float m = m0;
+#pragma unroll
+            for (int j = 0; j < WPH; j++) {
+                if (j == part) in = m;
+                const float2 r = agg[hw * WPH + j];
+                m = fmaxf(r.x + m, r.y);
             }
-            if (t0 + 32 * K < n) fetch(t0 + 32 * K);             // the next trip's logits are on their way while this one is scanned
+            m0 = m;
+        }
+        const float last = fmaxf(F + in, M);
+        float m = __shfl_up_sync(0xffffffffu, last, 1);          // the maximum in front of this lane's tokens
+        if (lane == 0) m = in;
+        if (K == 1) m0 = __shfl_sync(0xffffffffu, last, 31);
 #pragma unroll
-            for (int o = 1; o < 32; o <<= 1) {
-                const float Fp = __shfl_up_sync(0xffffffffu, F, o), Mp = __shfl_up_sync(0xffffffffu, M, o);
-                if (lane >= o) { M = fmaxf(Mp + F, M); F += Fp; }
+        for (int k = 0; k < K; k++) {
+            // the lane's last token takes the scan's number, so that the next lane's first factor starts from the same one
+            const float mn = k == K - 1 ? last : fmaxf(gf[k] + m, gi[k]), ld = (gf[k] + m) - mn, f0 = expf(gi[k] - mn), f1 = expf(ld), f3 = expf(-mn);
+            if (K == 1) {
+                if (t0 + base < n) { float * d = A.dg + (size_t) (s0 + t0 + base) * 4 * H + h; d[0] = f0; d[H] = f1; d[2 * H] = ld; d[3 * H] = f3; }
+            } else {
+                float * o = buf + pos + k;
+                o[0] = f0; o[HPB * PITCH] = f1; o[2 * HPB * PITCH] = ld; o[3 * HPB * PITCH] = f3;
             }
-            const float last = fmaxf(F + m0, M);
-            float m = __shfl_up_sync(0xffffffffu, last, 1);      // the maximum in front of this lane's tokens
-            if (lane == 0) m = m0;
-            m0 = __shfl_sync(0xffffffffu, last, 31);
+            m = mn;
+        }
+        if (K > 1) {
+            __syncthreads();
 #pragma unroll
-            for (int k = 0; k < K; k++) {
-                const int t = t0 + lane * K + k;
-                if (t < n) {
-                    // the lane's last token takes the scan's number, so that the next lane's first factor starts from the same one
-                    const float mn = k == K - 1 ? last : fmaxf(gf[k] + m, gi[k]), ld = (gf[k] + m) - mn;
-                    float * d = A.dg + (size_t) (s0 + t) * 4 * H + h;
-                    d[0] = expf(gi[k] - mn); d[H] = expf(ld); d[2 * H] = ld; d[3 * H] = expf(-mn);
-                    m = mn;
+            for (int k = 0; k < NS; k++) {
+                const int t = tl + STEP * k;
+                if (t0 + t < n && h0 + hl < H) {
+                    float * d = A.dg + (size_t) (s0 + t0 + t) * 4 * H + h0 + hl;
+#pragma unroll
+                    for (int j = 0; j < 4; j++) d[j * H] = buf[(HPB * j + hl) * PITCH + t + t / 8];
                 }
             }
         }
-        if (lane == 0) *mslot = m0;
     }
+    if (lane == 0 && part == 0 && h < H) *mslot = m0;
+}
+template <int VEC>
+__global__ void __launch_bounds__(256) attn_rows_kernel(amp_args A) {
+    pib_pdl_wait();
+    pib_pdl_trigger();
+    __shared__ float2 red[32];
+    amp_token<VEC>(A, blockIdx.x, red);
 }
 int pib_attn_mem_prep(const float * proj, int ldp, int i_off, int f_off, const pib_hlayer & L, float eps, const pib_hbatch & b, const float2 * rope, float * q, float * cache,
                       int cache_row, float * state, size_t state_stride, float * dg, cudaStream_t st) {
-    const int nq = L.heads * L.dim, nk = L.kv_heads * L.dim, nv = L.kv_heads * L.vdim, n_all = nq + nk + nv;
-    amp_args A = { proj, ldp, b.S, nq, nk, nv, L.dim, L.rot_dims, L.q_norm, L.k_norm, eps, b.pos, b.cell, rope, q, cache, cache_row, L.heads2, i_off, f_off, L.i_bias, L.f_bias,
+    const int nq = L.heads * L.dim, nk = L.kv_heads * L.dim, nv = L.kv_heads * L.vdim, n_all = nq + nk + nv, hpb = b.T == b.S ? 8 : 2, groups = (L.heads2 + hpb - 1) / hpb;
+    amp_args A = { proj, ldp, b.S * groups, groups, nq, nk, nv, L.dim, L.rot_dims, L.q_norm, L.k_norm, eps, b.pos, b.cell, rope, q, cache, cache_row, L.heads2, i_off, f_off, L.i_bias, L.f_bias,
                    L.gate_cap, b.seg_start, b.seg_len, b.seg_slot, state, state_stride, L.max_off, dg };
-    const int threads = b.T > 32 || b.T > b.S ? 256 : n_all >= 2048 ? 1024 : n_all >= 1024 ? 512 : 256;
-    if (b.T == b.S) pib_launch(attn_mem_prep_kernel<1>, dim3((unsigned) (b.T + b.S)), dim3(threads), (size_t) 0, st, A);
-    else            pib_launch(attn_mem_prep_kernel<8>, dim3((unsigned) (b.T + b.S)), dim3(threads), (size_t) 0, st, A);
+    auto al = [](const void * p) { return ((uintptr_t) p & 15) == 0; };
+    const bool vec = L.dim % 4 == 0 && (L.rot_dims / 2) % 4 == 0 && nv % 4 == 0 && ldp % 4 == 0 && cache_row % 4 == 0 && al(proj) && al(q) && al(cache);
+    if (b.T == b.S) {
+        const dim3 grid((unsigned) (b.T + b.S * groups)), threads(b.T > 32 ? 256u : n_all >= 2048 ? 1024u : n_all >= 1024 ? 512u : 256u);
+        if (vec) pib_launch(attn_mem_prep_kernel<1, 4>, grid, threads, (size_t) 0, st, A);
+        else     pib_launch(attn_mem_prep_kernel<1, 1>, grid, threads, (size_t) 0, st, A);
+    } else {
+        pib_launch(attn_mem_prep_kernel<8, 1>, dim3((unsigned) (b.S * groups)), dim3(256), (size_t) 0, st, A);
+        CKL();
+        if (vec) pib_launch(attn_rows_kernel<4>, dim3((unsigned) b.T), dim3(256), (size_t) 0, st, A);
+        else     pib_launch(attn_rows_kernel<1>, dim3((unsigned) b.T), dim3(256), (size_t) 0, st, A);
+    }
     CKL();
     return PIB_OK;
 }

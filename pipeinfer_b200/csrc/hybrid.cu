@@ -40,6 +40,7 @@ struct pib_hybrid_ctx {
     // operands of the matmul form of the attention: keys [NK][row] and transposed latents [R][NKp] (bfloat16), query rows, score rows
     void * am_kb = nullptr, * am_vt = nullptr, * am_p = nullptr; float * am_q = nullptr, * am_s = nullptr;
     size_t am_kb_cap = 0, am_vt_cap = 0, am_q_cap = 0, am_s_cap = 0, am_p_cap = 0;
+    void * chunk_buf = nullptr; size_t chunk_cap = 0;      // operands of a recurrence's matmul form
     float * split_buf = nullptr; size_t split_cap = 0;     // a long segment of the constant-decay recurrence in parts: the parts' matrices and table
     std::string kv_error;                       // set when a cache op arrived that the states cannot follow
     // per-launch timing (llama_pib_profile_layer(ctx, >= 0) switches it on): CUDA events around every launch of every layer
@@ -57,13 +58,13 @@ static const char * const HK_NAMES[] = { "cellmap", "embed_ln", "canon_conv", "m
                                          "mm_dual_proj", "dual_prep", "decay_scan", "dual_gate", "mm_dual_o",
                                          "hyper_norm", "mm_mamba2_in", "mamba2_conv", "mamba2_prep", "mamba2_scan", "gated_group_norm", "mm_mamba2_o", "qkv_rope", "diff_combine",
                                          "mm_gate_up",
-                                         "gated_norm", "input_conv", "mm_res_gate", "mm_attn_mem_proj", "attn_mem_prep", "memory_scan", "attn_mem_gate", "mm_attn_mem_o", "mm_gate_pair" };
+                                         "gated_norm", "input_conv", "mm_res_gate", "mm_attn_mem_proj", "attn_mem_prep", "memory_scan", "attn_mem_gate", "mm_attn_mem_o", "mm_gate_pair", "memory_scan_mm" };
 enum { HK_CELLMAP, HK_EMBED, HK_CANON, HK_DQKV, HK_LPREP, HK_UQ, HK_ABSORB, HK_LATTN, HK_UV, HK_AO, HK_QFV, HK_GATES, HK_SCAN, HK_HO, HK_LNRES, HK_UP, HK_POLY, HK_DOWN,
        HK_ROUTER, HK_ROUTE, HK_SORT, HK_EUP, HK_EDOWN, HK_SUP, HK_SDOWN, HK_COMBINE, HK_FINAL, HK_HEAD, HK_SAMPLE, HK_LATTN_MM,
        HK_EMBSCALE, HK_NORM2, HK_QKV, HK_QKVCONV, HK_APREP, HK_KVATTN, HK_KVATTN_MM, HK_SHIFT, HK_RKVG, HK_DECAY, HK_DECAYACT, HK_WKVSCAN, HK_DPREP, HK_DSCAN, HK_GHNORM, HK_GLU,
        HK_PSUM, HK_EMBPAIR, HK_PRENORM, HK_CONCAT, HK_LOOPIN, HK_SSMIN, HK_SSMCONV, HK_SSMX, HK_SSMDT, HK_SSMSCAN, HK_SSMO, HK_DUALPROJ, HK_DUALPREP, HK_DECAYSCAN, HK_DUALGATE,
        HK_DUALO, HK_HYPER, HK_M2IN, HK_M2CONV, HK_M2PREP, HK_M2SCAN, HK_GGNORM, HK_M2O, HK_QKVROPE, HK_DIFFCOMB, HK_GATEUP,
-       HK_GNORM, HK_INCONV, HK_RGATE, HK_AMPROJ, HK_AMPREP, HK_MEMSCAN, HK_AMGATE, HK_AMO, HK_GATE_PAIR, HK_COUNT };
+       HK_GNORM, HK_INCONV, HK_RGATE, HK_AMPROJ, HK_AMPREP, HK_MEMSCAN, HK_AMGATE, HK_AMO, HK_GATE_PAIR, HK_MEMSCAN_MM, HK_COUNT };
 const char * pib_hybrid_kind_name(int k) { return k >= 0 && k < HK_COUNT ? HK_NAMES[k] : "?"; }
 
 // fetch and clear the records; returns the count (the stream is synchronised)
@@ -128,6 +129,7 @@ int pib_hybrid_slots_free(const pib_context * c) { return c->hy ? c->hy->slots.n
 
 #define SCAN_SPLIT_MIN 256
 static bool scan_split_enabled() { static const int on = getenv("PIB_SCAN_SPLIT") ? atoi(getenv("PIB_SCAN_SPLIT")) : 1; return on != 0; }
+static bool chunk_scan_enabled() { static const int on = getenv("PIB_SCAN_MM") ? atoi(getenv("PIB_SCAN_MM")) : 1; return on != 0; }
 static bool attn_mm_enabled() { static const int on = getenv("PIB_ATTN_MM") ? atoi(getenv("PIB_ATTN_MM")) : 1; return on != 0; }
 
 // operands of the matmul form of an attention: key rows of `kw` (+ `kx` extra) bfloat16 each, transposed values [kw][2 NKp], query and
@@ -148,6 +150,15 @@ static int grow_attn_mm(pib_context * c, size_t kw, size_t kx, int q_rows, int s
     return PIB_OK;
 }
 
+static int grow_chunk(pib_context * c, size_t need) {
+    pib_hybrid_ctx * x = c->hy;
+    if (need <= x->chunk_cap) return PIB_OK;
+    cudaStreamSynchronize(c->stream);
+    if (x->chunk_buf) cudaFree(x->chunk_buf);
+    x->chunk_cap = need + need / 8;
+    if (cudaMalloc(&x->chunk_buf, x->chunk_cap) != cudaSuccess) { cudaGetLastError(); x->chunk_buf = nullptr; x->chunk_cap = 0; pib_set_error("decode: out of memory for the recurrence's operands"); return PIB_ERR_NOMEM; }
+    return PIB_OK;
+}
 static void free_scratch(pib_hybrid_ctx * x) {
     for (void * b : { (void *) x->x, (void *) x->h, (void *) x->y, (void *) x->proj, (void *) x->cq, (void *) x->q, (void *) x->qlat, (void *) x->lat, (void *) x->att,
                       (void *) x->rlog, (void *) x->wts, (void *) x->eup, (void *) x->edn, (void *) x->ysh, (void *) x->ids, (void *) x->perm, (void *) x->inv,
@@ -164,7 +175,7 @@ void pib_hybrid_ctx_free(pib_context * c) {
     free_scratch(x);
     if (x->state) cudaFree(x->state);
     if (x->cellmap) cudaFree(x->cellmap);
-    for (void * p : { x->am_kb, x->am_vt, x->am_p, (void *) x->am_q, (void *) x->am_s, (void *) x->split_buf }) if (p) cudaFree(p);
+    for (void * p : { x->am_kb, x->am_vt, x->am_p, (void *) x->am_q, (void *) x->am_s, (void *) x->split_buf, x->chunk_buf }) if (p) cudaFree(p);
     for (float * p : x->cache) if (p) cudaFree(p);
     for (float2 * p : x->rope) if (p) cudaFree(p);
     for (int i = 0; i < pib_hybrid_ctx::RING; i++) { if (x->meta_host[i]) cudaFreeHost(x->meta_host[i]); if (x->meta_ev[i]) cudaEventDestroy(x->meta_ev[i]); }
@@ -210,6 +221,8 @@ static int grow_scratch(pib_context * c, int T) {
 #define MM_ATTN_MIN_LEN 128
 #define MM_ATTN_MIN_ROW 192
 #define MM_ATTN_BLOCK   512
+// a recurrence's matmul form works through a segment in blocks of at most MM_SCAN_BLOCK tokens (its operands take a few hundred MB per block)
+#define MM_SCAN_BLOCK   2048
 struct pib_hseg { int start, len, seq, slot; bool fresh; };
 
 
@@ -478,12 +491,32 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
         float * cache = x->cache[L.cache_id];
         if ((rc = with_gate(HK_AMPROJ, mmfl(L.qkv), mmby(L.qkv), mm_of(L.qkv, hin, W, x->proj, ldp, PIB_EPI_NONE))) != PIB_OK) return rc;
         RC(HK_AMPREP, 0, 4.0 * Td * (2.0 * q2 + 6.0 * H2), pib_attn_mem_prep(x->proj, ldp, gi, gf, L, eps, B, x->rope[L.rope_id], x->q, cache, row, x->state, hy->state_floats, x->cq, st));
+        nk += T > B.S;
         if ((rc = kv_attend(L, cache, row, x->lat)) != PIB_OK) return rc;
-        int parts = 0, per = 0;
-        if ((rc = split_plan(H2, D2, V2 + 1, parts, per)) != PIB_OK) return rc;
-        RC(HK_MEMSCAN, 5.0 * Td * H2 * D2 * (V2 + 1.0), 4.0 * Td * H2 * (2.0 * D2 + 2.0 * V2 + 3.0),
-           pib_memory_scan(x->proj, ldp, q2, k2, v2, x->cq, L, B, x->state, hy->state_floats, x->cv, st, x->split_buf, parts, per));
-        nk += parts ? 4 : 0;
+        // long segments in served mode: chunks as matmuls; the others token by token (one long segment alone: in parts)
+        const bool mm_ok = !exact && pib_chunk_scan_fits(D2, V2) && chunk_scan_enabled();
+        double tok_mm = 0;
+        for (const pib_hseg & g : segs) if (mm_ok && g.len >= MM_ATTN_MIN_LEN) tok_mm += g.len;
+        const double tok_fl = 5.0 * H2 * D2 * (V2 + 1.0), tok_by = 4.0 * H2 * (2.0 * D2 + 2.0 * V2 + 3.0);
+        if (tok_mm < Td) {
+            int parts = 0, per = 0;
+            if (D2 <= 256 && (rc = split_plan(H2, D2, V2 + 1, parts, per)) != PIB_OK) return rc;
+            RC(HK_MEMSCAN, (Td - tok_mm) * tok_fl, (Td - tok_mm) * tok_by,
+               pib_memory_scan(x->proj, ldp, q2, k2, v2, x->cq, L, B, x->state, hy->state_floats, x->cv, st, x->split_buf, parts, per, tok_mm > 0 ? B.mmflag : nullptr));
+            nk += parts ? 4 : 0;
+        }
+        for (const pib_hseg & g : segs) {
+            if (!mm_ok || g.len < MM_ATTN_MIN_LEN) continue;
+            for (int o = 0; o < g.len; o += MM_SCAN_BLOCK) {
+                pib_chunk_scan a;
+                a.q = x->proj + q2; a.k = x->proj + k2; a.v = x->proj + v2; a.ldq = a.ldk = a.ldv = ldp; a.weight = x->cq; a.log_decay = x->cq + 2 * H2; a.ldg = 4 * H2;
+                a.H = a.G = H2; a.D = D2; a.V = V2; a.ones = 1; a.t0 = g.start + o; a.n = std::min(MM_SCAN_BLOCK, g.len - o);
+                a.state = x->state + (size_t) g.slot * hy->state_floats + L.state_off; a.out = x->cv;
+                if ((rc = grow_chunk(c, pib_chunk_scan_bytes(a))) != PIB_OK) return rc;
+                RC(HK_MEMSCAN_MM, a.n * tok_fl, a.n * tok_by, pib_chunk_scan_run(a, x->chunk_buf, st));
+                nk += 6;
+            }
+        }
         RC(HK_AMGATE, 0, 4.0 * Td * (2.0 * H * V + 3.0 * H2 * V2 + 2.0 * H2 + H), pib_attn_mem_gate(x->lat, x->cv, x->cq, x->proj, ldp, hg, og, L, eps, T, x->att, ldo, mem_off, st));
         if (pairs) RC(HK_AMO, mmfl(L.wo) + mmfl(L.wo2), mmby(L.wo) + mmby(L.wo2),
                       pib_dense_mm_pair(mm_of(L.wo, x->att, ldo, x->y, W, PIB_EPI_NONE), mm_of(L.wo2, x->att + mem_off, ldo, x->y2, W, PIB_EPI_NONE), st));

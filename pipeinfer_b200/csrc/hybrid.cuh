@@ -332,5 +332,16 @@ int pib_attn_mem_prep(const float * proj, int ldp, int i_off, int f_off, const p
 int pib_attn_mem_gate(const float * a, const float * mem, const float * dg, const float * proj, int ldp, int hg_off, int og_off, const pib_hlayer & L, float eps, int T, float * out,
                       int ldo, int mem_off, cudaStream_t st);
 int pib_memory_scan(const float * proj, int ldp, int q_off, int k_off, int v_off, float * dg, const pib_hlayer & L, const pib_hbatch & b, float * state, size_t state_stride, float * out,
-                    cudaStream_t st, float * split_buf = nullptr, int parts = 0, int per = 0);   // mixer_kernels.cu
+                    cudaStream_t st, float * split_buf = nullptr, int parts = 0, int per = 0, const int32_t * skip = nullptr);   // mixer_kernels.cu
+// chunk_scan.cu: n tokens of one segment (batch rows t0 ..) of a recurrence with one decay per head and token, as matmuls (served mode)
+struct pib_chunk_scan {
+    const float * q = nullptr, * k = nullptr, * v = nullptr; int ldq = 0, ldk = 0, ldv = 0;   // rows [G][D], [G][D], [H][V] per token
+    const float * weight = nullptr, * log_decay = nullptr; int ldg = 0;                       // [T][..H..] each
+    int H = 0, G = 0, D = 0, V = 0, ones = 0, t0 = 0, n = 0;                                  // ones: one more value column, always 1
+    float * state = nullptr;                                                                  // the segment's matrices [H][D][V (+ 1)]
+    float * out = nullptr;                                                                    // [T][H][V (+ 1)]
+};
+bool   pib_chunk_scan_fits(int D, int V);
+size_t pib_chunk_scan_bytes(const pib_chunk_scan & a);
+int    pib_chunk_scan_run(const pib_chunk_scan & a, void * buf, cudaStream_t st);
 int pib_diff_combine(const float * a, const pib_hlayer & L, float eps, int T, float * out, cudaStream_t st);

@@ -437,9 +437,58 @@ __global__ void __launch_bounds__(256) lat_softmax_kernel(float * __restrict__ S
     }
     (void) NK; (void) hi;
 }
+// the same for rows of up to 512 NR columns: a thread keeps its NR pairs of neighbouring columns in registers, so that a row is read once
+// (only where a key is seen) and its weights leave in one pass
+template <int NR>
+__global__ void __launch_bounds__(256) row_softmax_kernel(const float * __restrict__ S, __nv_bfloat16 * __restrict__ P, int NKp, int j0, int window, const int32_t * __restrict__ pos, int t0,
+                                                          int rows_per_z, int rep, const float * __restrict__ sink, int mask, int keep, int n_front, float softcap) {
+    pib_pdl_wait();
+    pib_pdl_trigger();
+    __shared__ float red[32];
+    const int row = blockIdx.x, rz = row % rows_per_z, t = t0 + rz / rep, h = (row / rows_per_z) * rep + rz % rep, p = pos[t];
+    const float *   s  = S + (size_t) row * NKp;
+    __nv_bfloat16 * pw = P + (size_t) row * 2 * NKp;
+    const int lo = (mask == PIB_MASK_CHUNK ? p - p % window : max(0, p - window + 1)) - j0 + n_front, hi = p - j0 + n_front, ka = n_front > 0 ? n_front : min(keep, lo);
+    const float sk = sink ? sink[h] : -INFINITY, icap = softcap > 0.f ? 1.0f / softcap : 0.f;
+    float2 v[NR];
+    float  m = sk;
+#pragma unroll
+    for (int i = 0; i < NR; i++) {
+        const int  j = 2 * ((int) threadIdx.x + 256 * i);
+        const bool a = (j >= lo && j <= hi) || j < ka, b = (j + 1 >= lo && j + 1 <= hi) || j + 1 < ka;
+        v[i] = make_float2(-INFINITY, -INFINITY);
+        if (a || b) {
+            const float2 x = *reinterpret_cast<const float2 *>(s + j);
+            if (a) v[i].x = softcap > 0.f ? softcap * tanhf(x.x * icap) : x.x;
+            if (b) v[i].y = softcap > 0.f ? softcap * tanhf(x.y * icap) : x.y;
+            m = fmaxf(m, fmaxf(v[i].x, v[i].y));
+        }
+    }
+    m = warp_max(m);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = m;
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < 8; i++) m = fmaxf(m, red[i]);
+    float sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < NR; i++) { v[i].x = expf(v[i].x - m); v[i].y = expf(v[i].y - m); sum += v[i].x + v[i].y; }      // exp(-inf) = 0 outside the mask
+    const float inv = 1.0f / (block_sum(sum, red) + (sink ? expf(sk - m) : 0.f));
+#pragma unroll
+    for (int i = 0; i < NR; i++) {
+        const int j = 2 * ((int) threadIdx.x + 256 * i);
+        if (j >= NKp) break;
+        const float x = v[i].x * inv, y = v[i].y * inv;
+        const __nv_bfloat16 hx = __float2bfloat16_rn(x), hy = __float2bfloat16_rn(y);
+        *reinterpret_cast<__nv_bfloat162 *>(pw + j) = __halves2bfloat162(hx, hy);
+        *reinterpret_cast<__nv_bfloat162 *>(pw + NKp + j) = __floats2bfloat162_rn(x - __bfloat162float(hx), y - __bfloat162float(hy));
+    }
+}
 int pib_window_softmax(float * S, void * P, int NKp, int NK, int j0, int window, const int32_t * pos, int t0, int n_rows, int rows_per_z, int rep, const float * sink,
                        cudaStream_t st, int mask, int keep, int n_front, float softcap) {
-    pib_launch(lat_softmax_kernel, dim3(n_rows), dim3(256), (size_t) (0), st, S, (__nv_bfloat16 *) P, NKp, NK, j0, window, pos, t0, rows_per_z, rep, sink, mask, keep, n_front, softcap);
+#define SM_GO(NR) pib_launch(row_softmax_kernel<NR>, dim3(n_rows), dim3(256), (size_t) 0, st, (const float *) S, (__nv_bfloat16 *) P, NKp, j0, window, pos, t0, rows_per_z, rep, sink, mask, keep, n_front, softcap)
+    if (NKp <= 512) SM_GO(1); else if (NKp <= 1024) SM_GO(2); else if (NKp <= 2048) SM_GO(4); else if (NKp <= 4096) SM_GO(8);
+#undef SM_GO
+    else pib_launch(lat_softmax_kernel, dim3(n_rows), dim3(256), (size_t) (0), st, S, (__nv_bfloat16 *) P, NKp, NK, j0, window, pos, t0, rows_per_z, rep, sink, mask, keep, n_front, softcap);
     CKL();
     return PIB_OK;
 }

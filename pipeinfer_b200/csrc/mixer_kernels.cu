@@ -208,22 +208,48 @@ int pib_kv_attention(const float * q, const pib_hlayer & L, const pib_hbatch & b
 // [G][V][2 NKp], query rows [G][nq * rep][3 D], all bfloat16 -- and put the outputs [G][nq * rep][V] back in token order.
 __device__ __forceinline__ void mk_split(float x, __nv_bfloat16 & hi, __nv_bfloat16 & lo) { hi = __float2bfloat16_rn(x); lo = __float2bfloat16_rn(x - __bfloat162float(hi)); }
 // columns [0, n_front) are positions 0 .. n_front - 1, the columns behind them positions j0, j0 + 1, ...
-__global__ void __launch_bounds__(128) kv_gather_kernel(const float * __restrict__ cache, int cache_row, const int32_t * __restrict__ map, int j0, int n_front, int NK, int NKp, int G, int maps,
+// grid (32 columns, problem (key / value head, map), 2): z = 0 the keys, z = 1 the values, which go through shared memory to come out transposed
+__global__ void __launch_bounds__(256) kv_gather_kernel(const float * __restrict__ cache, int cache_row, const int32_t * __restrict__ map, int j0, int n_front, int NK, int NKp, int G, int maps,
                                                         int D, int V, __nv_bfloat16 * __restrict__ Kb, __nv_bfloat16 * __restrict__ Vt) {
     pib_pdl_wait();
     pib_pdl_trigger();
-    const int j = blockIdx.x, GK = G * maps;          // one problem per (key / value head, map): its own keys, the head's values
-    const float * row = j < NK ? cache + (size_t) map[j < n_front ? j : j0 + j - n_front] * cache_row : nullptr;
-    for (int i = threadIdx.x; i < GK * D; i += blockDim.x) {
-        __nv_bfloat16 hi, lo;
-        mk_split(row ? row[i] : 0.f, hi, lo);
-        __nv_bfloat16 * k = Kb + ((size_t) (i / D) * NKp + j) * 3 * D + i % D;
-        k[0] = hi; k[D] = hi; k[2 * D] = lo;
+    __shared__ float tile[32][33];
+    const int c0 = blockIdx.x * 32, z = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, GK = G * maps;
+    const float * rows[4];                            // this warp's four columns (keys)
+#pragma unroll
+    for (int r = 0; r < 4; r++) {
+        const int j = c0 + warp + 8 * r;
+        rows[r] = j < NK ? cache + (size_t) map[j < n_front ? j : j0 + j - n_front] * cache_row : nullptr;
     }
-    for (int i = threadIdx.x; i < GK * V; i += blockDim.x) {
-        const int z = i / V, c = i % V;
-        const __nv_bfloat16 v = __float2bfloat16_rn(row ? row[(size_t) GK * D + (size_t) (z / maps) * V + c] : 0.f);
-        Vt[(size_t) i * 2 * NKp + j] = v; Vt[(size_t) i * 2 * NKp + NKp + j] = v;
+    if (blockIdx.z == 0) {
+        for (int i = lane; i < D; i += 32) {
+#pragma unroll
+            for (int r = 0; r < 4; r++) {
+                const int j = c0 + warp + 8 * r;
+                if (j >= NKp) continue;
+                __nv_bfloat16 hi, lo;
+                mk_split(rows[r] ? rows[r][(size_t) z * D + i] : 0.f, hi, lo);
+                __nv_bfloat16 * k = Kb + ((size_t) z * NKp + j) * 3 * D + i;
+                k[0] = hi; k[D] = hi; k[2 * D] = lo;
+            }
+        }
+        return;
+    }
+    const size_t vo = (size_t) GK * D + (size_t) (z / maps) * V;
+    for (int v0 = 0; v0 < V; v0 += 32) {
+#pragma unroll
+        for (int r = 0; r < 4; r++) tile[lane][warp + 8 * r] = rows[r] && v0 + lane < V ? rows[r][vo + v0 + lane] : 0.f;
+        __syncthreads();
+#pragma unroll
+        for (int r = 0; r < 4; r++) {
+            const int c = v0 + warp + 8 * r;
+            if (c < V && c0 + lane < NKp) {
+                const __nv_bfloat16 v = __float2bfloat16_rn(tile[warp + 8 * r][lane]);
+                __nv_bfloat16 * p = Vt + ((size_t) z * V + c) * 2 * NKp + c0 + lane;
+                p[0] = v; p[NKp] = v;
+            }
+        }
+        __syncthreads();
     }
 }
 // query row h of a token (maps rows per head, next to each other) belongs to problem z = (head / rep) * maps + h % maps, row ti * rep + head % rep
@@ -232,34 +258,38 @@ __device__ __forceinline__ size_t kv_problem_row(int h, int maps, int rep, int n
     return (size_t) z * nq * rep + (size_t) ti * rep + hq % rep;
 }
 // Qc[z][ti * rep + hr] = [hi | lo | hi] of scale * q[t0 + ti][h]
-__global__ void __launch_bounds__(128) kv_query_rows_kernel(const float * __restrict__ q, __nv_bfloat16 * __restrict__ Qc, int H, int maps, int rep, int nq, int D, int t0, float scale) {
+__global__ void __launch_bounds__(256) kv_query_rows_kernel(const float * __restrict__ q, __nv_bfloat16 * __restrict__ Qc, int H, int maps, int rep, int nq, int D, int t0, float scale) {
     pib_pdl_wait();
     pib_pdl_trigger();
-    const int ti = blockIdx.x, h = blockIdx.y;
-    const float * src = q + ((size_t) (t0 + ti) * H + h) * D;
-    __nv_bfloat16 * dst = Qc + kv_problem_row(h, maps, rep, nq, ti) * 3 * D;
-    for (int i = threadIdx.x; i < D; i += blockDim.x) {
-        __nv_bfloat16 hi, lo;
-        mk_split(src[i] * scale, hi, lo);
-        dst[i] = hi; dst[D + i] = lo; dst[2 * D + i] = hi;
+    const int ti = blockIdx.x;
+    for (int h = threadIdx.x >> 5; h < H; h += blockDim.x >> 5) {           // a warp per query row
+        const float * src = q + ((size_t) (t0 + ti) * H + h) * D;
+        __nv_bfloat16 * dst = Qc + kv_problem_row(h, maps, rep, nq, ti) * 3 * D;
+        for (int i = threadIdx.x & 31; i < D; i += 32) {
+            __nv_bfloat16 hi, lo;
+            mk_split(src[i] * scale, hi, lo);
+            dst[i] = hi; dst[D + i] = lo; dst[2 * D + i] = hi;
+        }
     }
 }
 // out[t0 + ti][h][V] = O[z][ti * rep + hr][V]
-__global__ void __launch_bounds__(128) kv_token_order_kernel(const float * __restrict__ O, float * __restrict__ out, int H, int maps, int rep, int nq, int V, int t0) {
+__global__ void __launch_bounds__(256) kv_token_order_kernel(const float * __restrict__ O, float * __restrict__ out, int H, int maps, int rep, int nq, int V, int t0) {
     pib_pdl_wait();
     pib_pdl_trigger();
-    const int ti = blockIdx.x, h = blockIdx.y;
-    const float * src = O + kv_problem_row(h, maps, rep, nq, ti) * V;
-    float * dst = out + ((size_t) (t0 + ti) * H + h) * V;
-    for (int i = threadIdx.x; i < V; i += blockDim.x) dst[i] = src[i];
+    const int ti = blockIdx.x;
+    for (int h = threadIdx.x >> 5; h < H; h += blockDim.x >> 5) {
+        const float * src = O + kv_problem_row(h, maps, rep, nq, ti) * V;
+        float * dst = out + ((size_t) (t0 + ti) * H + h) * V;
+        for (int i = threadIdx.x & 31; i < V; i += 32) dst[i] = src[i];
+    }
 }
 int pib_kv_attention_mm(const float * q, const pib_hlayer & L, const pib_hbatch & b, const float * cache, int cache_row, const int32_t * map, int t0, int nq, int j0, int n_front, int NK,
                         void * Kb, void * Vt, float * Qc, float * S, void * P, float * out, cudaStream_t st) {
     const int maps = L.maps, H = L.heads * maps, G = L.kv_heads, GK = G * maps, D = L.dim, V = L.vdim, rep = L.heads / G, NKp = (NK + 7) & ~7, M = nq * rep;
     if (maps > 1 && L.sink) { pib_set_error("attention: a sink with several maps per head"); return PIB_ERR_UNSUPP; }
-    pib_launch(kv_gather_kernel, dim3(NKp), dim3(128), (size_t) 0, st, cache, cache_row, map, j0, n_front, NK, NKp, G, maps, D, V, (__nv_bfloat16 *) Kb, (__nv_bfloat16 *) Vt);
+    pib_launch(kv_gather_kernel, dim3((unsigned) ((NKp + 31) / 32), (unsigned) GK, 2), dim3(256), (size_t) 0, st, cache, cache_row, map, j0, n_front, NK, NKp, G, maps, D, V, (__nv_bfloat16 *) Kb, (__nv_bfloat16 *) Vt);
     CKL();
-    pib_launch(kv_query_rows_kernel, dim3((unsigned) nq, (unsigned) H), dim3(128), (size_t) 0, st, q, (__nv_bfloat16 *) Qc, H, maps, rep, nq, D, t0, L.scale);
+    pib_launch(kv_query_rows_kernel, dim3((unsigned) nq), dim3(256), (size_t) 0, st, q, (__nv_bfloat16 *) Qc, H, maps, rep, nq, D, t0, L.scale);
     CKL();
     pib_mm a;
     a.W = Kb; a.wtype = PIB_TYPE_BF16; a.ldw = 3 * D; a.wz = (int64_t) NKp * 3 * D; a.X = Qc; a.ldx = 3 * D; a.xz = (int64_t) M * 3 * D; a.x_bf16 = 1;
@@ -271,7 +301,7 @@ int pib_kv_attention_mm(const float * q, const pib_hlayer & L, const pib_hbatch 
     v.W = Vt; v.wtype = PIB_TYPE_BF16; v.ldw = 2 * NKp; v.wz = (int64_t) V * 2 * NKp; v.X = (const float *) P; v.ldx = 2 * NKp; v.xz = (int64_t) M * 2 * NKp; v.x_bf16 = 1;
     v.Y = Qc; v.ldy = V; v.yz = (int64_t) M * V; v.M = M; v.N = V; v.K = 2 * NKp; v.Z = GK;              // the query rows are used up: the outputs take their place
     if ((rc = pib_dense_mm(v, st)) != PIB_OK) return rc;
-    pib_launch(kv_token_order_kernel, dim3((unsigned) nq, (unsigned) H), dim3(128), (size_t) 0, st, (const float *) Qc, out, H, maps, rep, nq, V, t0);
+    pib_launch(kv_token_order_kernel, dim3((unsigned) nq), dim3(256), (size_t) 0, st, (const float *) Qc, out, H, maps, rep, nq, V, t0);
     CKL();
     return PIB_OK;
 }
@@ -385,6 +415,7 @@ struct ls_args {
     const int32_t * seg_start, * seg_len, * seg_slot;
     float * state; size_t state_stride, state_off;
     float * out;                             // [T][H][V]
+    const int32_t * skip = nullptr;          // [T] (optional): a segment whose first token is flagged is walked elsewhere
     int vec16;                               // set by lin_scan: the operand rows start on 16-byte boundaries and D is a multiple of 4 (staged in 16-byte pieces)
 };
 __device__ __forceinline__ float ls_sum16(float x) {
@@ -402,6 +433,7 @@ __global__ void __launch_bounds__(16 * LS_VT) lin_scan_kernel(ls_args A) {
     const int sg = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * LS_VT, part = threadIdx.x & 15, vl = threadIdx.x >> 4, vd = v0 + vl;
     const int D = FULL ? 16 * RPT : A.D, Vv = A.V, V = MODE == 4 ? A.V + 1 : A.V, H = A.H, grp = h / (H / A.G), CH = A.chunk;
     const int s0 = A.seg_start[sg], n = A.seg_len[sg];
+    if (A.skip && A.skip[s0]) return;
     constexpr bool TWO = MODE == 1 || MODE == 3 || MODE == 4;      // two numbers per head and token beside the rows
     const int vbase = MODE == 0 ? 3 * D : 2 * D, dot_off = vbase + LS_VT + (TWO ? 2 : 0), row_f = (dot_off + 4) & ~3;
     const float cdec = MODE == 2 ? A.w[h] : 0.f, skip = MODE == 3 ? A.u[h] : 0.f;
@@ -556,7 +588,8 @@ __global__ void __launch_bounds__(16 * LS_VT) lin_scan_kernel(ls_args A) {
 }
 
 static int lin_scan(int mode, ls_args & A, int S, cudaStream_t st) {
-    if (A.D > 256) { pib_set_error("recurrence: dim %d not supported (up to 256)", A.D); return PIB_ERR_UNSUPP; }
+    const int most = mode == 4 ? 512 : 256;
+    if (A.D > most) { pib_set_error("recurrence: dim %d not supported (up to %d)", A.D, most); return PIB_ERR_UNSUPP; }
     const int Vt = A.V + (mode == 4 ? 1 : 0);
     dim3 grid((unsigned) S, (unsigned) A.H, (unsigned) ((Vt + LS_VT - 1) / LS_VT));
     const size_t row_f = ((size_t) (mode == 0 ? 3 * A.D : 2 * A.D) + LS_VT + ((mode == 1 || mode == 3 || mode == 4) ? 2 : 0) + 4) & ~(size_t) 3;
@@ -575,7 +608,7 @@ static int lin_scan(int mode, ls_args & A, int S, cudaStream_t st) {
                                     pib_launch(lin_scan_kernel<RPT, MODE, FULL>, dim3(grid), dim3(16 * LS_VT), (size_t) smem, st, A); } while (0)
 #define LS_PICK(MODE) do { if (A.D == 64) LS_GO(4, MODE, true); else if (A.D == 128) LS_GO(8, MODE, true); else if (A.D <= 32) LS_GO(2, MODE, false); \
                            else if (A.D <= 64) LS_GO(4, MODE, false); else if (A.D <= 128) LS_GO(8, MODE, false); else LS_GO(16, MODE, false); } while (0)
-    if (mode == 0) LS_PICK(0); else if (mode == 1) LS_PICK(1); else if (mode == 2) LS_PICK(2); else if (mode == 3) LS_PICK(3); else LS_PICK(4);
+    if (mode == 0) LS_PICK(0); else if (mode == 1) LS_PICK(1); else if (mode == 2) LS_PICK(2); else if (mode == 3) LS_PICK(3); else if (A.D <= 256) LS_PICK(4); else LS_GO(32, 4, false);
 #undef LS_PICK
 #undef LS_GO
     CKL();
@@ -766,9 +799,10 @@ int pib_mamba2_scan(const float * xbc, int ldc, float * dg, const pib_hlayer & L
 // matrix memory: rows proj[t] hold q (H*D) at q_off, k (H*D) at k_off, v (H*V) at v_off; dg[t] = [e^(i - m) (H) | decay (H) | log decay (H) | e^-m (H)]
 // (pib_attn_mem_prep); the matrices are [H][D][V + 1], out [T][H][V + 1] = [S^T q | n . q].  Parts as for Mamba-2.
 int pib_memory_scan(const float * proj, int ldp, int q_off, int k_off, int v_off, float * dg, const pib_hlayer & L, const pib_hbatch & b, float * state, size_t state_stride, float * out,
-                    cudaStream_t st, float * split_buf, int parts, int per) {
+                    cudaStream_t st, float * split_buf, int parts, int per, const int32_t * skip) {
     const int H = L.heads2;
     ls_args A;
+    A.skip = skip;
     A.a = proj + q_off; A.lda = ldp; A.a_hs = L.dim2; A.k = proj + k_off; A.ldk = ldp; A.k_hs = L.dim2; A.w = dg; A.ldw = 4 * H; A.v = proj + v_off; A.ldv = ldp; A.u = nullptr;
     A.H = H; A.G = H; A.D = L.dim2; A.V = L.vdim2; A.seg_start = b.seg_start; A.seg_len = b.seg_len; A.seg_slot = b.seg_slot;
     A.state = state; A.state_stride = state_stride; A.state_off = L.state_off; A.out = out;

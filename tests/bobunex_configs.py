@@ -43,6 +43,16 @@ def memory_only():
     return model(48, 100, [(left(1, 1, 4, 4, 4, 0, 0), right(6, 24, 8), None), (left(1, 1, 4, 4, 4, 1, 2), right(3, 33, 25, cap=2.0), 40)], taps=2)
 
 
+def memory_wide():
+    """memories whose long portions run as matmuls in served mode, beside a small attention"""
+    return model(64, 110, [(left(1, 1, 8, 8, 5, 1, 4), right(3, 24, 20), 48), (left(1, 1, 8, 8, 5, 0, 0), right(2, 64, 33, cap=8.0), None)])
+
+
+def deep_memory():
+    """one memory with more rows than the other recurrences take, rows not a multiple of anything"""
+    return model(40, 60, [(left(1, 1, 8, 8, 4, 1, 0), right(1, 301, 12), 24), (left(1, 1, 8, 8, 4, 1, 0), right(2, 264, 20), None)], taps=5)
+
+
 def ones():
     """values that happen to be 1 or equal: one head, one state, one tap, window 1, nothing kept, nothing rotated, factors of 1"""
     return model(32, 40, [(left(1, 1, 1, 1, 1, 0, 0, scale=1.0, softcap=1.0), right(1, 1, 1, cap=1.0), 1),
@@ -88,4 +98,4 @@ def drawn(seed):
     return model(pick([24, 40, 53, 96, 136]), int(r.integers(30, 400)), layers, taps=int(r.integers(1, 7)), eps=pick([1e-6, 1e-5, 1e-3]), embed_scale=float(pick([1.0, 0.5, 7.5])))
 
 
-CONFIGS = {f.__name__: f for f in (mixed_small, attention_only, memory_only, ones, far_keys, wide_heads, medium)}
+CONFIGS = {f.__name__: f for f in (mixed_small, attention_only, memory_only, memory_wide, deep_memory, ones, far_keys, wide_heads, medium)}

@@ -62,7 +62,7 @@ def spotlight(cfg, W, special_token, fi=3, fj=5):
 
 
 # ---- each mechanism alone, float32 and bfloat16 -------------------------------------------------------------------------------------------
-@pytest.mark.parametrize("name", ["attention_only", "memory_only", "ones", "mixed_small", "far_keys", "wide_heads"])
+@pytest.mark.parametrize("name", ["attention_only", "memory_only", "deep_memory", "ones", "mixed_small", "far_keys", "wide_heads"])
 @pytest.mark.parametrize("float32", [True, False])
 def test_whole_prompt_matches_oracle(tmp_path, name, float32):
     cfg = CONFIGS[name]()
@@ -138,7 +138,7 @@ def test_every_tensor_shows(tmp_path):
 
 
 # ---- prefill against token-by-token decoding, and portions down to two tokens ------------------------------------------------------------
-@pytest.mark.parametrize("name", ["mixed_small", "attention_only", "memory_only", "ones"])
+@pytest.mark.parametrize("name", ["mixed_small", "attention_only", "memory_only", "deep_memory", "ones"])
 def test_cuts_do_not_matter(tmp_path, name):
     cfg = CONFIGS[name]()
     W = O.random_weights(cfg, 12)
@@ -278,6 +278,33 @@ def test_long_prompt_carries_the_memory(tmp_path, name):
     assert close16(row_err(s.feed(0, toks, []), ref))
     assert close16(row_err(s.feed(1, toks, [300, 650] + list(range(651, 700))), ref))
     assert close16(row_err(s.feed(2, toks, range(100, 700, 100)), ref))
+    s.close()
+
+
+def test_memory_as_matmuls_against_the_walk(tmp_path):
+    """served mode: a 2200-token prompt takes the matmul form of the recurrence (chunks of 128, blocks of 2048 tokens), portions of 100 tokens
+    walk token by token; both against the oracle and against each other, lengths around a chunk's edge, and two long segments in one batch"""
+    cfg = CONFIGS["memory_wide"]()
+    W = O.random_weights(cfg, 41)
+    for i, jl in enumerate(cfg["layers"]):
+        W["l%d.mix.right.f.b" % i] = O.bf16_round(np.linspace(0.0, 8.0, jl["mixer"]["right"]["heads"]))
+    toks, other = tokens(cfg, 2200, 15), tokens(cfg, 300, 16)
+    ref, ref_o = oracle_logits(cfg, W, toks), oracle_logits(cfg, W, other)
+    s = Served(tmp_path, cfg, W, float32=False, n_ctx=7000)
+    whole = s.feed(0, toks, [])
+    small = s.feed(1, toks, range(100, 2200, 100))
+    for e in (row_err(whole, ref), row_err(small, ref), row_err(whole, small)):
+        assert close16(e)
+    assert np.median(row_err(whole, small)) < 0.5 * TOL16
+    s.end(0)
+    s.end(1)
+    assert close16(row_err(s.feed(2, toks[:900], [128, 257, 400, 527, 530, 531, 787]), ref[:900]))        # 128, 129, 143, 127, 3, 1, 256 and 113 tokens
+    s.end(2)
+    a = s.step([(3, toks[:300]), (4, other[:5]), (5, other[:1]), (6, other[:140])])
+    b = s.step([(5, other[1:]), (4, other[5:]), (6, other[140:141]), (3, toks[300:520])])
+    assert close16(row_err(np.concatenate([a[3], b[3]]), ref[:520]))
+    assert close16(row_err(np.concatenate([a[4], b[4]]), ref_o)) and close16(row_err(np.concatenate([a[5], b[5]]), ref_o))
+    assert close16(row_err(np.concatenate([a[6], b[6]]), ref_o[:141]))
     s.close()
 
 
