@@ -153,10 +153,10 @@ int pib_gated_norm(float * x, const pib_sublayer_out & o, const float * w, float
 }
 
 // ---- attention beside a matrix memory: what follows the projections -----------------------------------------------------------------------
-// Tokens (attn_rows_kernel; in batches of single tokens blocks of attn_mem_prep_kernel): one block each.  proj[t] = [q (nq = H*D) | k (nk = G*D) | v (nv = G*V) | ...]: q / rms(q) q_norm and k / rms(k) k_norm (one root mean
+// The last T blocks: one token each.  proj[t] = [q (nq = H*D) | k (nk = G*D) | v (nv = G*V) | ...]: q / rms(q) q_norm and k / rms(k) k_norm (one root mean
 // square over ALL rows of q, one over all of k), then the first rot_dims coordinates of every D-wide row turn (pairs (i, i + rot_dims / 2)); q[t] gets
 // the query rows, the token's cell [k | v].
-// Gates (attn_mem_prep_kernel): a block takes a few heads of one segment.  i = cap tanh((proj[i_off + h] + i_bias) / cap), f = log sigmoid(cap tanh((proj[f_off + h] +
+// The blocks in front of them: the memory's gates of a few heads of one segment.  i = cap tanh((proj[i_off + h] + i_bias) / cap), f = log sigmoid(cap tanh((proj[f_off + h] +
 // f_bias) / cap)); the running maximum m' = max(f + m, i) starts from the slot's and is left there.  It composes like a pair (F, M): m -> max(F + m, M),
 // (F1, M1) then (F2, M2) = (F1 + F2, max(M1 + F2, M2)), so a warp takes 32 K tokens per trip: K in a row per lane, an inclusive scan over the lanes (and, with
 // several warps per head, over the warps).
@@ -217,21 +217,21 @@ __device__ __forceinline__ void amp_token(const amp_args & A, int t, float2 * re
     }
     for (int e = threadIdx.x * VEC; e < A.nv; e += blockDim.x * VEC) gf_store<VEC>(row + A.nk + e, gf_load<VEC>(p + nqk + e));
 }
-// K == 1: tokens and gates of a batch of single tokens; K == 8: the gates alone
+// K == 1: batches of single tokens; K == 4: any batch
 template <int K, int VEC>
-__global__ void __launch_bounds__(K == 1 ? 1024 : 256) attn_mem_prep_kernel(amp_args A) {
+__global__ void __launch_bounds__(K == 1 ? 1024 : 256, K == 1 ? 1 : 4) attn_mem_prep_kernel(amp_args A) {
     pib_pdl_wait();
     pib_pdl_trigger();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    if (K == 1 && (int) blockIdx.x >= A.gate_blocks) {
+    if ((int) blockIdx.x >= A.gate_blocks) {
         __shared__ float2 red[32];
         amp_token<VEC>(A, blockIdx.x - A.gate_blocks, red);
         return;
     }
-    // K == 1 (single tokens): a block takes 8 heads of one segment, a warp per head.  K == 8: a block takes two heads, four warps each on neighbouring runs of
-    // 256 tokens; logits come in, and factors leave, through shared memory with neighbouring lanes on neighbouring heads
-    static_assert(K == 1 || K == 8, "tokens per lane");
-    constexpr int WPH = K == 1 ? 1 : 4, HPB = 8 / WPH, RUN = 32 * K, TT = WPH * RUN, PITCH = TT + TT / 8 + 1;      // token t sits at t + t / 8: a lane's 8 tokens start 9 words behind its neighbour's
+    // K == 1 (single tokens): a block takes 8 heads of one segment, a warp per head.  K == 4: a block takes two heads, four warps each on neighbouring runs of
+    // 128 tokens; logits come in, and factors leave, through shared memory with neighbouring lanes on neighbouring heads
+    static_assert(K == 1 || K == 4, "tokens per lane");
+    constexpr int WPH = K == 1 ? 1 : 4, HPB = 8 / WPH, RUN = 32 * K, TT = WPH * RUN, PITCH = TT + TT / K + 1;      // token t sits at t + t / K: a lane's K tokens start K + 1 words behind its neighbour's
     __shared__ float buf[K == 1 ? 1 : 4 * HPB * PITCH];
     __shared__ float2 agg[8];
     if (warp >= 8) return;                                       // (only K == 1 has more threads, and no barrier below)
@@ -257,13 +257,13 @@ __global__ void __launch_bounds__(K == 1 ? 1024 : 256) attn_mem_prep_kernel(amp_
     for (int t0 = 0; t0 < n; t0 += TT) {
         float gi[K], gf[K];
         const int  base = part * RUN + lane * K;                 // this lane's first token of the tile
-        const int  pos  = hw * PITCH + base + base / 8;
+        const int  pos  = hw * PITCH + base + base / K;
         if (K > 1) {
             __syncthreads();                                     // the trip before has left the buffer
 #pragma unroll
             for (int k = 0; k < NS; k++) {
                 const int t = tl + STEP * k;
-                buf[hl * PITCH + t + t / 8] = pi[k]; buf[(HPB + hl) * PITCH + t + t / 8] = pf[k];
+                buf[hl * PITCH + t + t / K] = pi[k]; buf[(HPB + hl) * PITCH + t + t / K] = pf[k];
             }
             __syncthreads();
         }
@@ -319,19 +319,12 @@ __global__ void __launch_bounds__(K == 1 ? 1024 : 256) attn_mem_prep_kernel(amp_
                 if (t0 + t < n && h0 + hl < H) {
                     float * d = A.dg + (size_t) (s0 + t0 + t) * 4 * H + h0 + hl;
 #pragma unroll
-                    for (int j = 0; j < 4; j++) d[j * H] = buf[(HPB * j + hl) * PITCH + t + t / 8];
+                    for (int j = 0; j < 4; j++) d[j * H] = buf[(HPB * j + hl) * PITCH + t + t / K];
                 }
             }
         }
     }
     if (lane == 0 && part == 0 && h < H) *mslot = m0;
-}
-template <int VEC>
-__global__ void __launch_bounds__(256) attn_rows_kernel(amp_args A) {
-    pib_pdl_wait();
-    pib_pdl_trigger();
-    __shared__ float2 red[32];
-    amp_token<VEC>(A, blockIdx.x, red);
 }
 int pib_attn_mem_prep(const float * proj, int ldp, int i_off, int f_off, const pib_hlayer & L, float eps, const pib_hbatch & b, const float2 * rope, float * q, float * cache,
                       int cache_row, float * state, size_t state_stride, float * dg, cudaStream_t st) {
@@ -345,10 +338,9 @@ int pib_attn_mem_prep(const float * proj, int ldp, int i_off, int f_off, const p
         if (vec) pib_launch(attn_mem_prep_kernel<1, 4>, grid, threads, (size_t) 0, st, A);
         else     pib_launch(attn_mem_prep_kernel<1, 1>, grid, threads, (size_t) 0, st, A);
     } else {
-        pib_launch(attn_mem_prep_kernel<8, 1>, dim3((unsigned) (b.S * groups)), dim3(256), (size_t) 0, st, A);
-        CKL();
-        if (vec) pib_launch(attn_rows_kernel<4>, dim3((unsigned) b.T), dim3(256), (size_t) 0, st, A);
-        else     pib_launch(attn_rows_kernel<1>, dim3((unsigned) b.T), dim3(256), (size_t) 0, st, A);
+        const dim3 grid((unsigned) (b.T + b.S * groups));
+        if (vec) pib_launch(attn_mem_prep_kernel<4, 4>, grid, dim3(256), (size_t) 0, st, A);
+        else     pib_launch(attn_mem_prep_kernel<4, 1>, grid, dim3(256), (size_t) 0, st, A);
     }
     CKL();
     return PIB_OK;

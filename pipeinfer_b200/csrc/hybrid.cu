@@ -491,7 +491,6 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
         float * cache = x->cache[L.cache_id];
         if ((rc = with_gate(HK_AMPROJ, mmfl(L.qkv), mmby(L.qkv), mm_of(L.qkv, hin, W, x->proj, ldp, PIB_EPI_NONE))) != PIB_OK) return rc;
         RC(HK_AMPREP, 0, 4.0 * Td * (2.0 * q2 + 6.0 * H2), pib_attn_mem_prep(x->proj, ldp, gi, gf, L, eps, B, x->rope[L.rope_id], x->q, cache, row, x->state, hy->state_floats, x->cq, st));
-        nk += T > B.S;
         if ((rc = kv_attend(L, cache, row, x->lat)) != PIB_OK) return rc;
         // long segments in served mode: chunks as matmuls; the others token by token (one long segment alone: in parts)
         const bool mm_ok = !exact && pib_chunk_scan_fits(D2, V2) && chunk_scan_enabled();
