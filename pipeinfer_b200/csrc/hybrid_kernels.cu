@@ -159,7 +159,7 @@ __global__ void __launch_bounds__(256) canon_tail_kernel(const float * __restric
     pib_pdl_trigger();
     const int sg = blockIdx.x, s0 = seg_start[sg], s1 = s0 + seg_len[sg];
     float * tail = state + (size_t) seg_slot[sg] * state_stride + tail_off;
-    for (int c = threadIdx.x; c < W; c += blockDim.x) {
+    for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < W; c += blockDim.x * gridDim.y) {
         float v[CANON_MAX_TAPS];
 #pragma unroll
         for (int k = 0; k < CANON_MAX_TAPS; k++) {
@@ -190,7 +190,7 @@ int pib_chan_conv(const float * u, int ldu, const float * w, int taps, const pib
 #undef CANON_GO
     else pib_launch(canon_kernel, dim3((unsigned) b.T, ny), dim3(256), (size_t) (0), st, u, ldu, w, taps, b.seg, b.seg_start, b.seg_slot, state, state_stride, tail_off, C, out, ldo, flags, bias);
     CKL();
-    if (taps > 1 && b.T > b.S) { pib_launch(canon_tail_kernel, dim3(b.S), dim3(256), (size_t) (0), st, u, ldu, taps, b.seg_start, b.seg_len, b.seg_slot, state, state_stride, tail_off, C); CKL(); }
+    if (taps > 1 && b.T > b.S) { pib_launch(canon_tail_kernel, dim3((unsigned) b.S, (unsigned) std::min(16, (C + 255) / 256)), dim3(256), (size_t) (0), st, u, ldu, taps, b.seg_start, b.seg_len, b.seg_slot, state, state_stride, tail_off, C); CKL(); }
     return PIB_OK;
 }
 // h = x + conv(x) over the model's width, in front of a mixer

@@ -70,6 +70,23 @@ def test_paired_gated_epilogue(M, F, K):
     np.testing.assert_allclose(got32, ref_of(X.astype(np.float32).astype(np.float64)), rtol=1e-5, atol=3e-6 * np.sqrt(K))
 
 
+@pytest.mark.parametrize("M,F,K", [(1, 40, 64), (3, 33, 72), (16, 200, 128), (17, 70, 64), (130, 150, 96), (300, 64, 200), (5, 7, 11)])
+def test_paired_gelu_epilogue(M, F, K):
+    """rows (gate i, up i) interleaved; output i is gelu(gate) * up with gelu = 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3)))"""
+    rng = np.random.default_rng(M + F)
+    Wg, Wu = bf16_round(rng.standard_normal((F, K))), bf16_round(rng.standard_normal((F, K)))
+    W = np.stack([Wg, Wu], 1).reshape(2 * F, K)
+    X = rng.standard_normal((M, K)) * 0.2
+
+    def ref_of(x):
+        z = x @ Wg.T
+        return 0.5 * z * (1.0 + np.tanh(np.sqrt(2.0 / np.pi) * (z + 0.044715 * z ** 3))) * (x @ Wu.T)
+    got = mm(W, X, M, 2 * F, K, ldy=F, epi=4).reshape(M, F)
+    np.testing.assert_allclose(got, ref_of(bf16_round(X)), rtol=1e-3, atol=1e-3 * np.sqrt(K))
+    got32 = mm(W, X, M, 2 * F, K, ldy=F, epi=4, exact=True, f32=True).reshape(M, F)
+    np.testing.assert_allclose(got32, ref_of(X.astype(np.float32).astype(np.float64)), rtol=1e-4, atol=1e-5 * np.sqrt(K))
+
+
 @pytest.mark.parametrize("T,H,D,R", [(5, 3, 24, 56), (40, 6, 72, 104), (200, 4, 128, 256), (130, 2, 16, 40)])
 def test_one_problem_per_head(T, H, D, R):
     """Y[t][h][r] = sum_d X[t][h][d] * W[h][r][d], X rows carry other columns between the heads' parts (the rotated query part)"""
