@@ -37,7 +37,7 @@ def rms_norm(x, w, eps):
 
 
 def input_conv(h, w, st, key):
-    """h + causal per-channel convolution of h; w [width, taps], the last column on the current token, zeros before the sequence's start"""
+    """h + causal per-channel convolution of h; w [width, taps], the last column on the current token; a fresh sequence has a tail of zeros"""
     taps = w.shape[1]
     ext = np.concatenate([st.get(key, np.zeros((taps - 1, h.shape[1]))), h], 0)
     out = h.copy()
@@ -130,7 +130,8 @@ def window_attention(h, W, pre, mx, eps, st, pos):
 
 # ---- matrix-memory branch ---------------------------------------------------------------------------------------------------------------
 def memory_scan(q, k, v, i, f, st):
-    """per head: m' = max(f + m, i); S <- e^(f + m - m') S + e^(i - m') k v^T, n likewise with k alone; o = S^T q / (max(|n . q|, e^-m') + 1e-6).
+    """per head: m' = max(f + m, i); S <- e^(f + m - m') S + e^(i - m') k v^T and, as if v were 1, n <- e^(f + m - m') n + e^(i - m') k;
+    o = S^T q / (max(|n . q|, e^-m') + 1e-6).
     q, k [T, H, D], v [T, H, V], i, f [T, H] (logarithms of the gates); S, n, m start at zero."""
     T, H, D = q.shape
     V = v.shape[2]
@@ -162,7 +163,7 @@ def matrix_memory(h, W, pre, mx, eps, st):
 
 
 def two_branches(h, W, pre, mx, eps, st, pos):
-    """half the sum of the two branches' outputs, each RMS-normed over the width"""
+    """the mean of attention and memory, after a norm over the width of either"""
     a = window_attention(h, W, pre + "left.", mx["left"], eps, st, pos)
     b = matrix_memory(h, W, pre + "right.", mx["right"], eps, st)
     return 0.5 * (rms_norm(a, W[pre + "left.out"], eps) + rms_norm(b, W[pre + "right.out"], eps))
@@ -188,7 +189,7 @@ def layer(x, cfg, W, il, st, pos):
 
 
 def forward(cfg, W, seq, tokens, trace=None):
-    """logits [T, vocab] of the next `tokens` of the sequence; trace (a list) receives the residual stream after every layer"""
+    """logits [T, vocab] of the next `tokens` of the sequence; trace (a list) receives x as each layer leaves it"""
     T = len(tokens)
     pos = list(range(seq.n, seq.n + T))
     x = W["embed"][np.asarray(tokens)] * cfg["embedding"]["scale"]
