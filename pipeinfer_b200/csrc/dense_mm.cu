@@ -31,7 +31,9 @@ struct mm_dev {
     int M, N, K;
     const int32_t * zrange;
     float e0, e1;
+    float * Y2; int64_t ld2; int n2; const int32_t * rows2;      // outputs n >= n2: Y2[rows2[m] * ld2 + n - n2]
 };
+__device__ __forceinline__ float * mm_out(const mm_dev & a, float * Y, int m, int n) { return n >= a.n2 ? a.Y2 + (size_t) a.rows2[m] * a.ld2 + (n - a.n2) : Y + (size_t) m * a.ldy + n; }
 
 template <typename WT, bool ROUND, int EPI>
 __global__ void __launch_bounds__(256) mm_tile_kernel(mm_dev a) {
@@ -108,7 +110,7 @@ __global__ void __launch_bounds__(256) mm_tile_kernel(mm_dev a) {
         for (int j = 0; j < 4; j++) {
             const int n = n0 + tx * 4 + j;
             if (n >= a.N) continue;
-            Y[(size_t) m * a.ldy + n] = pib_epilogue<EPI, ROUND>(acc[i][j], a.e0, a.e1);
+            *mm_out(a, Y, m, n) = pib_epilogue<EPI, ROUND>(acc[i][j], a.e0, a.e1);
         }
     }
 }
@@ -183,7 +185,7 @@ __device__ __forceinline__ void mv_rows_body(const mm_dev & a, bool xvec, int z,
 #pragma unroll
     for (int b = 0; b < B; b++) {
         if (lane == 0 && row0 + b < row1)
-            Y[(size_t) (row0 + b) * a.ldy + n] = pib_epi_pairs(EPI) ? pib_glu_pair<EPI, ROUND>(res[0][b], res[NR - 1][b], a.e0) : pib_epilogue<EPI, ROUND>(res[0][b], a.e0, a.e1);
+            *mm_out(a, Y, row0 + b, n) = pib_epi_pairs(EPI) ? pib_glu_pair<EPI, ROUND>(res[0][b], res[NR - 1][b], a.e0) : pib_epilogue<EPI, ROUND>(res[0][b], a.e0, a.e1);
     }
 }
 
@@ -279,13 +281,14 @@ int pib_dense_mm_tc(const pib_mm & a, cudaStream_t st);     // dense_mma.cu: bfl
 int pib_dense_mm(const pib_mm & a, cudaStream_t st) {
     if (a.M <= 0 || a.N <= 0 || a.K <= 0 || a.Z <= 0) return PIB_OK;
     if (a.exact && a.wtype != PIB_TYPE_F32) { pib_set_error("dense matmul: exact mode needs float32 weights"); return PIB_ERR_ARG; }
+    if (a.Y2 && (a.Z != 1 || a.zrange || pib_epi_pairs(a.epi) || !a.rows2)) { pib_set_error("dense matmul: a second destination takes one plain problem and a row list"); return PIB_ERR_ARG; }
     if (a.wtype == PIB_TYPE_BF16 && !a.exact) {
         const int rc = pib_dense_mm_tc(a, st);
         if (rc != PIB_ERR_UNSUPP) return rc;
     }
     if (a.x_bf16) { pib_set_error("dense matmul: bfloat16 activations need the tensor-core path (more than 16 rows, strides multiples of 8)"); return PIB_ERR_UNSUPP; }
-    mm_dev d = { a.W, a.ldw, a.wz, a.X, a.ldx, a.xz, a.xrows, a.xdiv < 1 ? 1 : a.xdiv, a.Y, a.ldy, a.yz, a.M, a.N, a.K, a.zrange, a.e0, a.e1 };
-    if (a.wtype == PIB_TYPE_F32 && a.exact && a.N <= 32 && a.M > MV_MAXB && a.Z == 1 && !a.xrows && !a.zrange && a.epi == PIB_EPI_NONE) {
+    mm_dev d = { a.W, a.ldw, a.wz, a.X, a.ldx, a.xz, a.xrows, a.xdiv < 1 ? 1 : a.xdiv, a.Y, a.ldy, a.yz, a.M, a.N, a.K, a.zrange, a.e0, a.e1, a.Y2, a.ld2, a.Y2 ? a.n2 : 0x7fffffff, a.rows2 };
+    if (a.wtype == PIB_TYPE_F32 && a.exact && !a.Y2 && a.N <= 32 && a.M > MV_MAXB && a.Z == 1 && !a.xrows && !a.zrange && a.epi == PIB_EPI_NONE) {
         dim3 grid((unsigned) ((a.M + 7) / 8));
         if (a.N <= 8)       pib_launch(mm_few_cols_kernel<8>, dim3(grid), dim3(256), (size_t) 0, st, d);
         else if (a.N <= 16) pib_launch(mm_few_cols_kernel<16>, dim3(grid), dim3(256), (size_t) 0, st, d);
@@ -297,6 +300,7 @@ int pib_dense_mm(const pib_mm & a, cudaStream_t st) {
 #define MM_GO(WT, ROUND) (a.epi == PIB_EPI_RELU2 ? launch_mm<WT, ROUND, PIB_EPI_RELU2>(a, d, st) : a.epi == PIB_EPI_XIELU ? launch_mm<WT, ROUND, PIB_EPI_XIELU>(a, d, st) : \
                           a.epi == PIB_EPI_GLU_PAIR ? launch_mm<WT, ROUND, PIB_EPI_GLU_PAIR>(a, d, st) : \
                           a.epi == PIB_EPI_GEGLU_PAIR ? launch_mm<WT, ROUND, PIB_EPI_GEGLU_PAIR>(a, d, st) : \
+                          a.epi == PIB_EPI_SWIGLU_PAIR ? launch_mm<WT, ROUND, PIB_EPI_SWIGLU_PAIR>(a, d, st) : \
                                                     launch_mm<WT, ROUND, PIB_EPI_NONE>(a, d, st))
     if (a.wtype == PIB_TYPE_BF16) return MM_GO(__nv_bfloat16, true);
     if (a.wtype == PIB_TYPE_F32) return a.exact ? MM_GO(float, false) : MM_GO(float, true);
@@ -318,13 +322,13 @@ static void launch_pair(const mm_dev & a, const mm_dev & b, bool xva, bool xvb, 
 }
 int pib_dense_mm_pair(const pib_mm & a, const pib_mm & b, cudaStream_t st) {
     const int V = a.wtype == PIB_TYPE_BF16 ? 8 : 4;
-    auto plain = [&](const pib_mm & m) { return m.Z == 1 && !m.xrows && !m.zrange && !m.x_bf16 && m.ldw % V == 0 && ((uintptr_t) m.W & 15) == 0; };
+    auto plain = [&](const pib_mm & m) { return m.Z == 1 && !m.xrows && !m.zrange && !m.x_bf16 && !m.Y2 && m.ldw % V == 0 && ((uintptr_t) m.W & 15) == 0; };
     if (a.M < 1 || a.M > MV_MAXB || a.M != b.M || a.wtype != b.wtype || a.exact != b.exact || !plain(a) || !plain(b) || a.epi != PIB_EPI_NONE ||
         (b.epi != PIB_EPI_NONE && b.epi != PIB_EPI_GEGLU_PAIR) || (pib_epi_pairs(b.epi) && (b.N & 1)) || (a.exact && a.wtype != PIB_TYPE_F32)) {
         const int rc = pib_dense_mm(a, st);
         return rc != PIB_OK ? rc : pib_dense_mm(b, st);
     }
-    auto dev = [](const pib_mm & m) { return mm_dev{ m.W, m.ldw, m.wz, m.X, m.ldx, m.xz, nullptr, 1, m.Y, m.ldy, m.yz, m.M, m.N, m.K, nullptr, m.e0, m.e1 }; };
+    auto dev = [](const pib_mm & m) { return mm_dev{ m.W, m.ldw, m.wz, m.X, m.ldx, m.xz, nullptr, 1, m.Y, m.ldy, m.yz, m.M, m.N, m.K, nullptr, m.e0, m.e1, nullptr, 0, 0x7fffffff, nullptr }; };
     auto xvec = [](const pib_mm & m) { return m.ldx % 4 == 0 && ((uintptr_t) m.X & 15) == 0; };
 #define PAIR_GO(WT, ROUND) do { if (b.epi == PIB_EPI_NONE) launch_pair<WT, ROUND, PIB_EPI_NONE>(dev(a), dev(b), xvec(a), xvec(b), st); \
                                 else launch_pair<WT, ROUND, PIB_EPI_GEGLU_PAIR>(dev(a), dev(b), xvec(a), xvec(b), st); } while (0)

@@ -89,7 +89,7 @@ template <int NB> struct dt_cfg {
 template <int NB, int EPI>
 __global__ void __launch_bounds__(DT_THREADS)
 dense_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ CUtensorMap xmap, int M, int N, int K, const int32_t * __restrict__ zrange,
-                int x_has_z, float * __restrict__ Y, int64_t ldy, int64_t yz, int * __restrict__ err, float e0, float e1) {
+                int x_has_z, float * __restrict__ Y, int64_t ldy, int64_t yz, int * __restrict__ err, float e0, float e1, float * __restrict__ Y2, int64_t ld2, int n2, const int32_t * __restrict__ rows2) {
     pib_pdl_wait();
     pib_pdl_trigger();
     const int z = blockIdx.z;
@@ -178,12 +178,12 @@ dense_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_constant_
                         if (!(lane & 1) && orow + 1 < N && m < row1) Yz[(size_t) m * ldy + (orow >> 1)] = pib_glu_pair<EPI, true>(mine, other, e0);
                     }
                 } else if (orow < N) {
+                    const bool second = orow >= n2;
+                    float *    base   = second ? Y2 + (orow - n2) : Yz + orow;
 #pragma unroll
                     for (int j = 0; j < 32; j++) {
                         const int m = m0 + c0 + j;
-                        if (m < row1) {
-                            Yz[(size_t) m * ldy + orow] = pib_epilogue<EPI, true>(__uint_as_float(v[j]), e0, e1);
-                        }
+                        if (m < row1) base[second ? (size_t) rows2[m] * ld2 : (size_t) m * ldy] = pib_epilogue<EPI, true>(__uint_as_float(v[j]), e0, e1);
                     }
                 }
             }
@@ -258,14 +258,21 @@ static int dt_launch(const pib_mm & a, const CUtensorMap & wmap, const CUtensorM
         PIB_CHECK(cudaFuncSetAttribute(dense_tc_kernel<NB, PIB_EPI_XIELU>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int) C::SMEM));
         PIB_CHECK(cudaFuncSetAttribute(dense_tc_kernel<NB, PIB_EPI_GLU_PAIR>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int) C::SMEM));
         PIB_CHECK(cudaFuncSetAttribute(dense_tc_kernel<NB, PIB_EPI_GEGLU_PAIR>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int) C::SMEM));
+        PIB_CHECK(cudaFuncSetAttribute(dense_tc_kernel<NB, PIB_EPI_SWIGLU_PAIR>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int) C::SMEM));
         configured = true;
     }
     dim3 grid((unsigned) ((a.N + DT_BM - 1) / DT_BM), (unsigned) ((a.M + NB - 1) / NB), (unsigned) a.Z);
-    if (a.epi == PIB_EPI_RELU2)      pib_launch(dense_tc_kernel<NB, PIB_EPI_RELU2>, dim3(grid), dim3(DT_THREADS), (size_t) (C::SMEM), st, wmap, xmap, a.M, a.N, a.K, a.zrange, x_has_z, a.Y, a.ldy, a.yz, err, a.e0, a.e1);
-    else if (a.epi == PIB_EPI_XIELU) pib_launch(dense_tc_kernel<NB, PIB_EPI_XIELU>, dim3(grid), dim3(DT_THREADS), (size_t) (C::SMEM), st, wmap, xmap, a.M, a.N, a.K, a.zrange, x_has_z, a.Y, a.ldy, a.yz, err, a.e0, a.e1);
-    else if (a.epi == PIB_EPI_GLU_PAIR) pib_launch(dense_tc_kernel<NB, PIB_EPI_GLU_PAIR>, dim3(grid), dim3(DT_THREADS), (size_t) (C::SMEM), st, wmap, xmap, a.M, a.N, a.K, a.zrange, x_has_z, a.Y, a.ldy, a.yz, err, a.e0, a.e1);
-    else if (a.epi == PIB_EPI_GEGLU_PAIR) pib_launch(dense_tc_kernel<NB, PIB_EPI_GEGLU_PAIR>, dim3(grid), dim3(DT_THREADS), (size_t) (C::SMEM), st, wmap, xmap, a.M, a.N, a.K, a.zrange, x_has_z, a.Y, a.ldy, a.yz, err, a.e0, a.e1);
-    else                             pib_launch(dense_tc_kernel<NB, PIB_EPI_NONE>, dim3(grid), dim3(DT_THREADS), (size_t) (C::SMEM), st, wmap, xmap, a.M, a.N, a.K, a.zrange, x_has_z, a.Y, a.ldy, a.yz, err, a.e0, a.e1);
+#define DT_GO(EPI) pib_launch(dense_tc_kernel<NB, EPI>, dim3(grid), dim3(DT_THREADS), (size_t) (C::SMEM), st, wmap, xmap, a.M, a.N, a.K, a.zrange, x_has_z, a.Y, a.ldy, a.yz, err, a.e0, a.e1, \
+                              a.Y2, a.ld2, a.Y2 ? a.n2 : 0x7fffffff, a.rows2)
+    switch (a.epi) {
+        case PIB_EPI_RELU2:       DT_GO(PIB_EPI_RELU2); break;
+        case PIB_EPI_XIELU:       DT_GO(PIB_EPI_XIELU); break;
+        case PIB_EPI_GLU_PAIR:    DT_GO(PIB_EPI_GLU_PAIR); break;
+        case PIB_EPI_GEGLU_PAIR:  DT_GO(PIB_EPI_GEGLU_PAIR); break;
+        case PIB_EPI_SWIGLU_PAIR: DT_GO(PIB_EPI_SWIGLU_PAIR); break;
+        default:                  DT_GO(PIB_EPI_NONE); break;
+    }
+#undef DT_GO
     PIB_CHECK(cudaGetLastError());
     return PIB_OK;
 }

@@ -58,13 +58,15 @@ static const char * const HK_NAMES[] = { "cellmap", "embed_ln", "canon_conv", "m
                                          "mm_dual_proj", "dual_prep", "decay_scan", "dual_gate", "mm_dual_o",
                                          "hyper_norm", "mm_mamba2_in", "mamba2_conv", "mamba2_prep", "mamba2_scan", "gated_group_norm", "mm_mamba2_o", "qkv_rope", "diff_combine",
                                          "mm_gate_up",
-                                         "gated_norm", "input_conv", "mm_res_gate", "mm_attn_mem_proj", "attn_mem_prep", "memory_scan", "attn_mem_gate", "mm_attn_mem_o", "mm_gate_pair", "memory_scan_mm" };
+                                         "gated_norm", "input_conv", "mm_res_gate", "mm_attn_mem_proj", "attn_mem_prep", "memory_scan", "attn_mem_gate", "mm_attn_mem_o", "mm_gate_pair", "memory_scan_mm",
+                                         "sandwich_norm", "moe_route_sort" };
 enum { HK_CELLMAP, HK_EMBED, HK_CANON, HK_DQKV, HK_LPREP, HK_UQ, HK_ABSORB, HK_LATTN, HK_UV, HK_AO, HK_QFV, HK_GATES, HK_SCAN, HK_HO, HK_LNRES, HK_UP, HK_POLY, HK_DOWN,
        HK_ROUTER, HK_ROUTE, HK_SORT, HK_EUP, HK_EDOWN, HK_SUP, HK_SDOWN, HK_COMBINE, HK_FINAL, HK_HEAD, HK_SAMPLE, HK_LATTN_MM,
        HK_EMBSCALE, HK_NORM2, HK_QKV, HK_QKVCONV, HK_APREP, HK_KVATTN, HK_KVATTN_MM, HK_SHIFT, HK_RKVG, HK_DECAY, HK_DECAYACT, HK_WKVSCAN, HK_DPREP, HK_DSCAN, HK_GHNORM, HK_GLU,
        HK_PSUM, HK_EMBPAIR, HK_PRENORM, HK_CONCAT, HK_LOOPIN, HK_SSMIN, HK_SSMCONV, HK_SSMX, HK_SSMDT, HK_SSMSCAN, HK_SSMO, HK_DUALPROJ, HK_DUALPREP, HK_DECAYSCAN, HK_DUALGATE,
        HK_DUALO, HK_HYPER, HK_M2IN, HK_M2CONV, HK_M2PREP, HK_M2SCAN, HK_GGNORM, HK_M2O, HK_QKVROPE, HK_DIFFCOMB, HK_GATEUP,
-       HK_GNORM, HK_INCONV, HK_RGATE, HK_AMPROJ, HK_AMPREP, HK_MEMSCAN, HK_AMGATE, HK_AMO, HK_GATE_PAIR, HK_MEMSCAN_MM, HK_COUNT };
+       HK_GNORM, HK_INCONV, HK_RGATE, HK_AMPROJ, HK_AMPREP, HK_MEMSCAN, HK_AMGATE, HK_AMO, HK_GATE_PAIR, HK_MEMSCAN_MM,
+       HK_SANDWICH, HK_ROUTE_SORT, HK_COUNT };
 const char * pib_hybrid_kind_name(int k) { return k >= 0 && k < HK_COUNT ? HK_NAMES[k] : "?"; }
 
 // fetch and clear the records; returns the count (the stream is synchronised)
@@ -327,7 +329,7 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
         return PIB_OK;
     };
     // the attention of cached key / value heads over `q`: per-token kernel, or the matmul form for long portions in served mode
-    auto kv_attend = [&](const pib_hlayer & L, float * cache, int row, float * out) -> int {
+    auto kv_attend = [&](const pib_hlayer & L, const pib_kv_query & q, float * cache, int row, float * out) -> int {
         const int H = L.heads * L.maps, G = L.kv_heads * L.maps, D = L.dim, V = L.vdim;      // query rows and key heads: one per map
         const double keys = key_pairs(L.window, L.mask, L.keep);
         const bool mm_ok = !exact && D % 8 == 0 && D >= 16 && V >= 16 && attn_mm_enabled();
@@ -335,7 +337,7 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
         for (const pib_hseg & g : segs) { if (mm_ok && g.len >= MM_ATTN_MIN_LEN) any_mm = true; else any_simt = true; }
         if (any_simt)
             RC(HK_KVATTN, 2.0 * keys * H * (D + V), 4.0 * keys * G * (D + V) + 4.0 * Td * H * (D + V),
-               pib_kv_attention(x->q, L, B, cache, row, x->cellmap, (int) c->n_ctx, out, any_mm ? B.mmflag : nullptr, st));
+               pib_kv_attention(q, L, B, cache, row, x->cellmap, (int) c->n_ctx, out, any_mm ? B.mmflag : nullptr, st));
         for (const pib_hseg & g : segs) {
             if (!mm_ok || g.len < MM_ATTN_MIN_LEN) continue;
             const int nb = (g.len + MM_ATTN_BLOCK - 1) / MM_ATTN_BLOCK, per = (g.len + nb - 1) / nb;      // blocks of equal size: none is left with a handful of rows
@@ -346,7 +348,7 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
                 const int NK = n_front + p0 + nq - j0;
                 if ((rc = grow_attn_mm(c, (size_t) G * std::max(D, V), (size_t) 3 * G * D + V, nq * H, nq * H, NK)) != PIB_OK) return rc;
                 RC(HK_KVATTN_MM, 2.0 * nq * H * (double) NK * (D + 2.0 * V), 2.0 * NK * G * (D + 2.0 * V) + 8.0 * nq * H * (D + V) + 8.0 * nq * H * (double) NK,
-                   pib_kv_attention_mm(x->q, L, B, cache, row, x->cellmap + (size_t) g.slot * c->n_ctx, g.start + o, nq, j0, n_front, NK, x->am_kb, x->am_vt, x->am_q, x->am_s,
+                   pib_kv_attention_mm(q, L, B, cache, row, x->cellmap + (size_t) g.slot * c->n_ctx, g.start + o, nq, j0, n_front, NK, x->am_kb, x->am_vt, x->am_q, x->am_s,
                                        x->am_p, out, st));
                 nk += 5;
             }
@@ -365,7 +367,18 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
             src = x->cv;
         }
         RC(HK_APREP, 0, 8.0 * Td * C, pib_swa_prep(src, C, L, eps, B, x->q, cache, row, x->vfirst, st));
-        if ((rc = kv_attend(L, cache, row, x->att)) != PIB_OK) return rc;
+        if ((rc = kv_attend(L, { x->q, L.heads * L.dim }, cache, row, x->att)) != PIB_OK) return rc;
+        RC(HK_AO, mmfl(L.wo), mmby(L.wo), mm(L.wo, x->att, H * V, x->y, W, PIB_EPI_NONE));
+        return PIB_OK;
+    };
+    // plain attention over cached key / value heads: one matmul whose keys and values land in their cells, attention with distance biases and the output gate, output
+    auto mixer_kv = [&](const pib_hlayer & L, const float * hin) -> int {
+        const int H = L.heads, D = L.dim, V = L.vdim, nq = H * D, ng = L.out_gate ? H * V : 0, ldp = (nq + ng + 3) & ~3, row = hy->cache_row[L.cache_id];
+        float * cache = x->cache[L.cache_id];
+        pib_mm a = mm_of(L.qkv, hin, W, x->proj, ldp, PIB_EPI_NONE);
+        if (L.kv_from < 0) { a.Y2 = cache; a.ld2 = row; a.n2 = nq + ng; a.rows2 = B.cell; }
+        RC(HK_QKV, mmfl(L.qkv), mmby(L.qkv), pib_dense_mm(a, st));
+        if ((rc = kv_attend(L, { x->proj, ldp, L.out_gate ? x->proj + nq : nullptr, ldp }, cache, row, x->att)) != PIB_OK) return rc;
         RC(HK_AO, mmfl(L.wo), mmby(L.wo), mm(L.wo, x->att, H * V, x->y, W, PIB_EPI_NONE));
         return PIB_OK;
     };
@@ -443,7 +456,7 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
         float * cache = x->cache[L.cache_id];
         RC(HK_DUALPROJ, mmfl(L.qkv), mmby(L.qkv), mm(L.qkv, hin, W, x->proj, ldp, PIB_EPI_NONE));
         RC(HK_DUALPREP, 0, 8.0 * Td * ldp, pib_dual_prep(x->proj, ldp, L, eps, B, x->rope[L.rope_id], x->q, cache, row, st));
-        if ((rc = kv_attend(L, cache, row, x->lat)) != PIB_OK) return rc;
+        if ((rc = kv_attend(L, { x->q, L.heads * L.maps * L.dim }, cache, row, x->lat)) != PIB_OK) return rc;
         int parts = 0, per = 0;
         if ((rc = split_plan(H2, D2, V2, parts, per)) != PIB_OK) return rc;
         RC(HK_DECAYSCAN, 5.0 * Td * H2 * D2 * V2, 4.0 * Td * H2 * (2.0 * D2 + 2.0 * V2),
@@ -476,7 +489,7 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
         float * cache = x->cache[L.cache_id];
         RC(HK_QKV, mmfl(L.qkv), mmby(L.qkv), mm(L.qkv, hin, W, x->proj, ldp, PIB_EPI_NONE));
         RC(HK_QKVROPE, 0, 8.0 * Td * N, pib_qkv_rope(x->proj, ldp, L, B, x->rope[L.rope_id], x->q, cache, row, st));
-        if ((rc = kv_attend(L, cache, row, x->lat)) != PIB_OK) return rc;
+        if ((rc = kv_attend(L, { x->q, L.heads * L.maps * L.dim }, cache, row, x->lat)) != PIB_OK) return rc;
         RC(HK_DIFFCOMB, 0, 4.0 * Td * H * V * (L.maps + 1.0), pib_diff_combine(x->lat, L, eps, T, x->att, st));
         RC(HK_AO, mmfl(L.wo), mmby(L.wo), mm(L.wo, x->att, H * V, x->y, W, PIB_EPI_NONE));
         return PIB_OK;
@@ -491,7 +504,7 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
         float * cache = x->cache[L.cache_id];
         if ((rc = with_gate(HK_AMPROJ, mmfl(L.qkv), mmby(L.qkv), mm_of(L.qkv, hin, W, x->proj, ldp, PIB_EPI_NONE))) != PIB_OK) return rc;
         RC(HK_AMPREP, 0, 4.0 * Td * (2.0 * q2 + 6.0 * H2), pib_attn_mem_prep(x->proj, ldp, gi, gf, L, eps, B, x->rope[L.rope_id], x->q, cache, row, x->state, hy->state_floats, x->cq, st));
-        if ((rc = kv_attend(L, cache, row, x->lat)) != PIB_OK) return rc;
+        if ((rc = kv_attend(L, { x->q, L.heads * L.maps * L.dim }, cache, row, x->lat)) != PIB_OK) return rc;
         // long segments in served mode: chunks as matmuls; the others token by token (one long segment alone: in parts)
         const bool mm_ok = !exact && pib_chunk_scan_fits(D2, V2) && chunk_scan_enabled();
         double tok_mm = 0;
@@ -537,35 +550,46 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
             case PIB_MIXER_MAMBA2: return mixer_mamba2(L, hin);
             case PIB_MIXER_DIFF:   return mixer_diff(L, hin);
             case PIB_MIXER_ATTN_MEM: return mixer_attn_mem(L, hin);
+            case PIB_MIXER_KV:     return mixer_kv(L, hin);
         }
         pib_set_error("decode: mixer %d", L.mixer);
         return PIB_ERR_UNSUPP;
     };
     // routed experts + shared expert of `min` [T][W]: x->edn holds the experts' outputs per (token, expert) pair in sorted order, x->ysh the
     // shared expert's; the caller combines them.  relu^2 experts: up rows only, the weights multiply the outputs (moe_combine); clamped gated
-    // experts: rows gate | up, the router's weight multiplies the expert's input, i.e. both products before the clamp (glu_clamp)
+    // experts: rows gate | up, the router's weight multiplies the expert's input, i.e. both products before the clamp (glu_clamp); silu-gated
+    // experts: gate and up rows interleaved, gate and product ride on the matmul's way out, the weights multiply the outputs.  The router may have
+    // outputs that are no experts (identity): their pairs sort behind all others and no matmul sees them
     auto run_experts = [&](const pib_hlayer & L, const float * min, int * ld_shared) -> int {
-        const int E = L.n_experts, top = L.top, P = T * top, glu = L.expert == PIB_EXPERT_GLU_CLAMP, NU = (glu ? 2 : 1) * L.ff_e;
-        const double touched = P >= E ? 1.0 : (double) P / E;          // weights of experts without a row are not read
+        const int  n_exp = L.n_experts, E = n_exp + L.identity, top = L.top, P = T * top;
+        const bool clamp = L.expert == PIB_EXPERT_GLU_CLAMP, paired = L.expert == PIB_EXPERT_SWIGLU;
+        const int  NU = (clamp || paired ? 2 : 1) * L.ff_e, ldu = paired ? L.ff_e : NU, epi = clamp ? PIB_EPI_NONE : paired ? PIB_EPI_SWIGLU_PAIR : PIB_EPI_RELU2;
+        const double Pe = (double) P * n_exp / E;                      // pairs of experts, if the router spreads them evenly
+        const double touched = Pe >= n_exp ? 1.0 : Pe / n_exp;         // weights of experts without a row are not read
+        const pib_router R = { E, top, L.route, L.groups, L.keep_groups, L.route_scale, L.correction };
         RC(HK_ROUTER, mmfl(L.router), mmby(L.router), mm(L.router, min, W, x->rlog, E, PIB_EPI_NONE));
-        RC(HK_ROUTE, 0, 4.0 * Td * E, pib_moe_route(x->rlog, T, E, top, L.route, x->ids, x->wts, st));
-        RC(HK_SORT, 0, 4.0 * P * (E + 3.0), pib_moe_sort(x->ids, P, E, x->counts, x->offs, x->perm, x->inv, st)); nk++;
+        if (pib_moe_route_sort_fits(T, R)) {
+            RC(HK_ROUTE_SORT, 0, 4.0 * Td * E + 16.0 * P, pib_moe_route_sort(x->rlog, T, R, x->ids, x->wts, x->offs, x->perm, x->inv, st));
+        } else {
+            RC(HK_ROUTE, 0, 4.0 * Td * E, pib_moe_route(x->rlog, T, R, x->ids, x->wts, st));
+            RC(HK_SORT, 0, 4.0 * P * (E + 3.0), pib_moe_sort(x->ids, P, E, x->counts, x->offs, x->perm, x->inv, st)); nk++;
+        }
         {   // up-projection of every (token, expert) pair, pairs grouped by expert
             pib_mm a;
             a.W = L.e_up->base; a.wtype = L.e_up->type; a.ldw = W; a.wz = (int64_t) NU * W; a.X = min; a.ldx = W; a.xrows = x->perm; a.xdiv = top;
-            a.Y = x->eup; a.ldy = NU; a.M = P; a.N = NU; a.K = W; a.Z = E; a.zrange = x->offs; a.epi = glu ? PIB_EPI_NONE : PIB_EPI_RELU2; a.exact = exact;
-            RC(HK_EUP, 2.0 * P * NU * Wd, wbytes(L.e_up) * touched + 4.0 * P * (Wd + NU), pib_dense_mm(a, st));
-            if (glu) RC(HK_GLU, 0, 12.0 * P * L.ff_e, pib_glu_clamp(x->eup, NU, L.ff_e, L.limit_e, x->wts, x->perm, P, st));
+            a.Y = x->eup; a.ldy = ldu; a.M = P; a.N = NU; a.K = W; a.Z = n_exp; a.zrange = x->offs; a.epi = epi; a.exact = exact;
+            RC(HK_EUP, 2.0 * Pe * NU * Wd, wbytes(L.e_up) * touched + 4.0 * Pe * (Wd + ldu), pib_dense_mm(a, st));
+            if (clamp) RC(HK_GLU, 0, 12.0 * P * L.ff_e, pib_glu_clamp(x->eup, NU, L.ff_e, L.limit_e, x->wts, x->perm, P, st));
             pib_mm b;
-            b.W = L.e_down->base; b.wtype = L.e_down->type; b.ldw = L.ff_e; b.wz = (int64_t) W * L.ff_e; b.X = x->eup; b.ldx = NU;
-            b.Y = x->edn; b.ldy = W; b.M = P; b.N = W; b.K = L.ff_e; b.Z = E; b.zrange = x->offs; b.exact = exact;
-            RC(HK_EDOWN, 2.0 * P * L.ff_e * Wd, wbytes(L.e_down) * touched + 4.0 * P * (Wd + L.ff_e), pib_dense_mm(b, st));
+            b.W = L.e_down->base; b.wtype = L.e_down->type; b.ldw = L.ff_e; b.wz = (int64_t) W * L.ff_e; b.X = x->eup; b.ldx = ldu;
+            b.Y = x->edn; b.ldy = W; b.M = P; b.N = W; b.K = L.ff_e; b.Z = n_exp; b.zrange = x->offs; b.exact = exact;
+            RC(HK_EDOWN, 2.0 * Pe * L.ff_e * Wd, wbytes(L.e_down) * touched + 4.0 * Pe * (Wd + L.ff_e), pib_dense_mm(b, st));
         }
         if (L.s_up) {
-            const int NS = (int) L.s_up->N, ld = (NS + 3) & ~3;
+            const int ld = ((paired ? L.ff_s : (int) L.s_up->N) + 3) & ~3;
             *ld_shared = ld;
-            RC(HK_SUP, mmfl(L.s_up), mmby(L.s_up), mm(L.s_up, min, W, x->proj, ld, glu ? PIB_EPI_NONE : PIB_EPI_RELU2));
-            if (glu) RC(HK_GLU, 0, 12.0 * Td * L.ff_s, pib_glu_clamp(x->proj, ld, L.ff_s, L.limit_s, nullptr, nullptr, T, st));
+            RC(HK_SUP, mmfl(L.s_up), wbytes(L.s_up) + 4.0 * Td * (Wd + ld), mm(L.s_up, min, W, x->proj, ld, epi));
+            if (clamp) RC(HK_GLU, 0, 12.0 * Td * L.ff_s, pib_glu_clamp(x->proj, ld, L.ff_s, L.limit_s, nullptr, nullptr, T, st));
             pib_mm d;
             d.W = L.s_down->base; d.wtype = L.s_down->type; d.ldw = L.ff_s; d.X = x->proj; d.ldx = ld; d.Y = x->ysh; d.ldy = W; d.M = T; d.N = W; d.K = L.ff_s;
             d.exact = exact || L.s_down->type == PIB_TYPE_F32;
@@ -576,7 +600,7 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
 
     RC(HK_CELLMAP, 0, 16.0 * Td, pib_cellmap_set(x->cellmap, (int) c->n_ctx, B, st));
     if (hy->form == PIB_FORM_HYPER)        RC(HK_EMBSCALE, 0, (2.0 + 4.0 * hy->streams) * Td * Wd, pib_embed_scale(m->tok_embd, B.tok, hy->embd_scale, T, W, x->x, st, hy->streams));
-    else if (hy->form == PIB_FORM_PARALLEL || hy->form == PIB_FORM_GATED) RC(HK_EMBSCALE, 0, 6.0 * Td * Wd, pib_embed_scale(m->tok_embd, B.tok, hy->embd_scale, T, W, x->x, st));
+    else if (hy->form == PIB_FORM_PARALLEL || hy->form == PIB_FORM_GATED || hy->form == PIB_FORM_SANDWICH) RC(HK_EMBSCALE, 0, 6.0 * Td * Wd, pib_embed_scale(m->tok_embd, B.tok, hy->embd_scale, T, W, x->x, st));
     else if (hy->form == PIB_FORM_PRENORM) RC(HK_EMBPAIR, 0, (hy->loops ? 10.0 : 6.0) * Td * Wd, pib_embed_pair(m->tok_embd, B.tok, T, W, x->x, hy->loops ? x->cat : nullptr, st));
     else                                   RC(HK_EMBED, 0, 6.0 * Td * Wd, pib_embed_ln(m->tok_embd, B.tok, hy->embd_norm, eps, T, W, x->x, st));
     // pre-norm form: the stream is (have_x ? cur : 0) + pend_y + pend_b; the sum is formed by the next norm's kernel, which leaves it in the
@@ -606,10 +630,31 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
         }
         return PIB_OK;
     };
+    // sandwich frame: what the sublayer before left is normed, scaled and added by the kernel that norms the stream for the next one
+    pib_sublayer_y leftn;
+    auto sandwich = [&](const float * w, const float * b) -> int {
+        RC(HK_SANDWICH, 0, 4.0 * Td * Wd * ((leftn.y ? 3.0 : leftn.top ? 2.0 : 1.0) + leftn.top + (w ? 1.0 : 0.0)), pib_sandwich_norm(x->x, leftn, w, b, eps, T, W, w ? x->h : nullptr, st));
+        leftn = pib_sublayer_y();
+        return PIB_OK;
+    };
     for (int il = 0; il < m->n_layer; il++) {
         const pib_hlayer & L = hy->layers[il];
         int lds = 0;
-        if (hy->form == PIB_FORM_GATED) {
+        if (hy->form == PIB_FORM_SANDWICH) {
+            if ((rc = sandwich(L.norm1, L.norm1_b)) != PIB_OK) return rc;
+            if ((rc = run_mixer(L, x->h)) != PIB_OK) return rc;
+            leftn.y = x->y; leftn.w = L.post1; leftn.b = L.post1_b;
+            if (L.mlp != PIB_MLP_NONE && (rc = sandwich(L.norm2, L.norm2_b)) != PIB_OK) return rc;
+            if (L.mlp == PIB_MLP_RELU2) {
+                RC(HK_UP, mmfl(L.up), mmby(L.up), mm(L.up, x->h, W, x->proj, L.ff, PIB_EPI_RELU2));
+                RC(HK_DOWN, mmfl(L.down), mmby(L.down), mm(L.down, x->proj, L.ff, x->y, W, PIB_EPI_NONE));
+                leftn.y = x->y;
+            } else if (L.mlp == PIB_MLP_MOE && L.expert == PIB_EXPERT_SWIGLU) {
+                if ((rc = run_experts(L, x->h, &lds)) != PIB_OK) return rc;
+                leftn.y = L.s_up ? x->ysh : nullptr; leftn.edn = x->edn; leftn.wts = x->wts; leftn.ids = x->ids; leftn.inv = x->inv; leftn.hin = x->h; leftn.top = L.top; leftn.n_real = L.n_experts;
+            } else if (L.mlp != PIB_MLP_NONE) { pib_set_error("decode: feed-forward %d in a sandwich layer", L.mlp); return PIB_ERR_UNSUPP; }
+            if (L.mlp != PIB_MLP_NONE) { leftn.w = L.post2; leftn.b = L.post2_b; }
+        } else if (hy->form == PIB_FORM_GATED) {
             if ((rc = gated(L.norm1, L.canon, L.tail_off)) != PIB_OK) return rc;
             gate_w = L.rg1;
             if (L.mixer != PIB_MIXER_ATTN_MEM) { RC(HK_RGATE, mmfl(L.rg1), mmby(L.rg1), mm(L.rg1, x->h, W, x->rg, W, PIB_EPI_NONE)); gate_w = nullptr; }      // the other mixers launch their matmuls alone
@@ -680,6 +725,7 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
                 RC(HK_LNRES, 0, 12.0 * Td * Wd, pib_layer_norm(x->y, L.norm2, eps, T, W, x->x, 1, st));
             }
         }
+        if (getenv("PIB_HYBRID_DUMP") && hy->form == PIB_FORM_SANDWICH) { if ((rc = sandwich(nullptr, nullptr)) != PIB_OK) return rc; }
         if (getenv("PIB_HYBRID_DUMP") && hy->form == PIB_FORM_GATED && left.ya) { if ((rc = gated(nullptr, nullptr, 0)) != PIB_OK) return rc; }
         if (getenv("PIB_HYBRID_DUMP") && hy->form == PIB_FORM_HYPER) {   // debugging: the sum of the streams after every layer, one file per layer and decode
             if (pend_y) { RC(HK_HYPER, 0, 0, pib_hyper_norm(x->x, hy->streams, pend_y, pend_b, nullptr, nullptr, nullptr, eps, T, W, nullptr, st)); pend_y = pend_b = nullptr; }
@@ -702,7 +748,8 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
             if (FILE * f = fopen(path, "wb")) { fwrite(hb.data(), 4, hb.size(), f); fclose(f); }
         }
     }
-    if (hy->form == PIB_FORM_GATED)         { if ((rc = gated(m->output_norm, nullptr, 0)) != PIB_OK) return rc; }
+    if (hy->form == PIB_FORM_SANDWICH)      { if ((rc = sandwich(m->output_norm, hy->final_b)) != PIB_OK) return rc; }
+    else if (hy->form == PIB_FORM_GATED)    { if ((rc = gated(m->output_norm, nullptr, 0)) != PIB_OK) return rc; }
     else if (hy->form == PIB_FORM_HYPER)    RC(HK_FINAL, 0, (4.0 * hy->streams + 8.0) * Td * Wd, pib_hyper_norm(x->x, hy->streams, pend_y, pend_b, nullptr, m->output_norm, hy->final_b, eps, T, W, x->h, st));
     else if (hy->form == PIB_FORM_PRENORM)  { if ((rc = prenorm(hy->final_g, nullptr, 0, false)) != PIB_OK) return rc; }
     else if (hy->form == PIB_FORM_PARALLEL) RC(HK_FINAL, 0, 8.0 * Td * Wd, pib_rms_norm2(x->x, m->output_norm, nullptr, eps, hy->logit_scale, T, W, x->h, nullptr, st));

@@ -23,7 +23,13 @@
 //   one more mixer: windowed softmax attention that also keeps the sequence's first tokens (one RMS norm over all query rows and one over
 //                  all key rows, capped scores, a sink of score 0, a gate per head) beside a matrix memory with exponential gates (mLSTM);
 //                  each branch has an output matrix of its own, their outputs are RMS-normed over the width and averaged
-// Designs built from these parts: "Rapisun", "Fabivik", "Lulenex", "Putazen", "Bobunex".  The parts take their sizes and constants as parameters so that another
+//   plain attention: queries, keys and values straight from one projection, which writes the cache cells itself; scores with a distance bias --
+//                  a slope per head (ALiBi), or a learned number per head and distance bucket (T5) --, a learned sink or kept first tokens, an
+//                  optional sigmoid gate on every value of the heads' outputs; a layer may read another layer's cells (kv_from)
+//   and a frame for it: a LayerNorm before and one after every sublayer, the result scaled per channel and by one number (sandwich)
+//   more mixtures: softmax scores without renormalisation, chosen by score + correction inside the best groups of neighbours, with identity
+//                  outputs that pass the input on; silu-gated experts.  A dense squared-relu feed-forward
+// Designs built from these parts: "Rapisun", "Fabivik", "Lulenex", "Putazen", "Bobunex", "Gusedra".  The parts take their sizes and constants as parameters so that another
 // layer-list design can name them too.
 //
 // What such a model adds to the runtime, beside what llama / falcon graphs use:
@@ -38,28 +44,29 @@
 #include "engine.cuh"
 
 enum { PIB_MIXER_LATENT = 1, PIB_MIXER_HGRN2 = 2, PIB_MIXER_SWA = 3, PIB_MIXER_WKV = 4, PIB_MIXER_DELTA = 5, PIB_MIXER_SSM = 6, PIB_MIXER_DUAL = 7,
-       PIB_MIXER_MAMBA2 = 8, PIB_MIXER_DIFF = 9, PIB_MIXER_ATTN_MEM = 10 };
-enum { PIB_MLP_NONE = 0, PIB_MLP_POLYNORM = 1, PIB_MLP_MOE = 2, PIB_MLP_XIELU = 3, PIB_MLP_GLU = 4, PIB_MLP_GEGLU = 5 };
+       PIB_MIXER_MAMBA2 = 8, PIB_MIXER_DIFF = 9, PIB_MIXER_ATTN_MEM = 10, PIB_MIXER_KV = 11 };
+enum { PIB_MLP_NONE = 0, PIB_MLP_POLYNORM = 1, PIB_MLP_MOE = 2, PIB_MLP_XIELU = 3, PIB_MLP_GLU = 4, PIB_MLP_GEGLU = 5, PIB_MLP_RELU2 = 6 };
 // which earlier positions j a token at p may read: the last `window` ones (p - window < j <= p), or those of its own chunk (j / window == p / window)
 enum { PIB_MASK_WINDOW = 0, PIB_MASK_CHUNK = 1 };
 // what a matmul does to an output on its way out: nothing; max(y, 0)^2; xIELU (y > 0: e0 y^2 + y/2, else e1 (exp(y) - 1 - y) + y/2)
 //   PIB_EPI_GLU_PAIR: outputs come in pairs (2 i: gate g, 2 i + 1: linear part u; the weight rows are stored interleaved); output i of a row with pitch ldy is
 //   a sigmoid(1.702 a) (b + 1), a = min(g, e0), b = clamp(u, -e0, e0).  N counts the weight rows (twice the outputs).
-//   PIB_EPI_GEGLU_PAIR: pairs as above; output i is gelu(g) u, gelu in its tanh form.
-enum { PIB_EPI_NONE = 0, PIB_EPI_RELU2 = 1, PIB_EPI_XIELU = 2, PIB_EPI_GLU_PAIR = 3, PIB_EPI_GEGLU_PAIR = 4 };
+//   PIB_EPI_GEGLU_PAIR: pairs as above; output i is gelu(g) u, gelu in its tanh form.   PIB_EPI_SWIGLU_PAIR: g sigmoid(g) u.
+enum { PIB_EPI_NONE = 0, PIB_EPI_RELU2 = 1, PIB_EPI_XIELU = 2, PIB_EPI_GLU_PAIR = 3, PIB_EPI_GEGLU_PAIR = 4, PIB_EPI_SWIGLU_PAIR = 5 };
 // layer forms: x += LN(mixer(conv(x))), x += LN(ff(x))   |   x += mixer(N1(x)) + ff(N2(x)), N = RMS norm with weight (1 + w)
 //              x += mixer(shift(N(x))), x += ff(N(x)), N = RMS norm times one number, shift(h)_t = h_t + (h_{t-1} - h_t) * mu
 //              hyper-connections over S streams X_s: u = sum_s in_s X_s, y = sublayer(LN(u)) (LayerNorm with weight and bias),
 //              X_t <- sum_s mix[s][t] X_s + out_t y, for the mixer and then for the feed-forward; the model's output reads sum_s X_s
 //              gated: h = N(x), x += sublayer(h + conv(h)) * sigmoid(R h + r), for the mixer and then for the feed-forward
-enum { PIB_FORM_POSTNORM = 0, PIB_FORM_PARALLEL = 1, PIB_FORM_PRENORM = 2, PIB_FORM_HYPER = 3, PIB_FORM_GATED = 4 };
+//              sandwich: x += m ls * LN'(sublayer(LN(x))), both LayerNorms with weight and bias, m one number, ls per channel
+enum { PIB_FORM_POSTNORM = 0, PIB_FORM_PARALLEL = 1, PIB_FORM_PRENORM = 2, PIB_FORM_HYPER = 3, PIB_FORM_GATED = 4, PIB_FORM_SANDWICH = 5 };
 // how a rotation pairs coordinates: (i, i + dims / 2) or (2 i, 2 i + 1)
 enum { PIB_PAIR_HALF = 0, PIB_PAIR_ADJACENT = 1 };
 // how a rotation's frequencies are scaled (see pib_hybrid::Rope)
 enum { PIB_ROPE_PLAIN = 0, PIB_ROPE_YARN = 1, PIB_ROPE_BANDS = 2 };
 // mixture of experts: how the router's logits become weights, where a weight multiplies, what an expert computes
-enum { PIB_ROUTE_SOFTMAX_RENORM = 0, PIB_ROUTE_SIGMOID = 1 };
-enum { PIB_EXPERT_RELU2 = 0, PIB_EXPERT_GLU_CLAMP = 1 };
+enum { PIB_ROUTE_SOFTMAX_RENORM = 0, PIB_ROUTE_SIGMOID = 1, PIB_ROUTE_SOFTMAX_GROUPS = 2 };
+enum { PIB_EXPERT_RELU2 = 0, PIB_EXPERT_GLU_CLAMP = 1, PIB_EXPERT_SWIGLU = 2 };
 
 struct pib_hlayer {
     int     mixer = 0, mlp = 0;
@@ -148,6 +155,13 @@ struct pib_hlayer {
     float * i_bias = nullptr;                         // [heads2]  (forget gates: f_bias)
     float * out_a = nullptr, * out_b = nullptr;       // [width]: weights of the branches' output norms
     size_t  max_off = 0;                              // floats into a slot's state: m [heads2]   (state_off: the matrices)
+    // ---- plain attention (PIB_MIXER_KV): qkv rows q (heads*dim) | output gates (heads*vdim, with out_gate) | k (kv_heads*dim) | v (kv_heads*vdim), the last two
+    // absent with kv_from; any attention over cached key / value heads can name the distance biases ----
+    float * slopes = nullptr;                         // [heads]: score - slope * distance
+    float * rel = nullptr;                            // [heads][n_rel]: score + rel[head][min(distance, n_rel - 1)]
+    int     n_rel = 0, out_gate = 0;
+    // ---- sandwich frame: weights and biases of the norms behind the sublayers, times the layer scale and the residual multiplier ----
+    float * post1 = nullptr, * post1_b = nullptr, * post2 = nullptr, * post2_b = nullptr;
     // ---- feed-forward ----
     int   ff = 0;
     pib_weight * up = nullptr, * down = nullptr;
@@ -159,6 +173,11 @@ struct pib_hlayer {
     int   route = PIB_ROUTE_SOFTMAX_RENORM, expert = PIB_EXPERT_RELU2;
     float limit_e = 0.f, limit_s = 0.f;               // clamped gated experts: e_up / s_up hold rows gate | up (s_up one more row: the shared expert's gate logit)
     int   s_gate = 0;
+    // PIB_ROUTE_SOFTMAX_GROUPS: the router has n_experts + identity outputs in `groups` equal groups of neighbours, of which the `keep_groups` with the
+    // largest choice score (score + correction) take part; the chosen ones' softmax scores times route_scale are the weights
+    int   identity = 0, groups = 1, keep_groups = 1;
+    float route_scale = 1.f;
+    float * correction = nullptr;
 };
 
 struct pib_hybrid {
@@ -222,6 +241,8 @@ struct pib_mm {
     int             epi = PIB_EPI_NONE;
     float           e0 = 0.f, e1 = 0.f;                  // the epilogue's constants (xIELU: softplus(p), 1/2 + softplus(q))
     int             exact = 0;                           // 1: operands stay fp32 (no bfloat16 rounding of X); W must be float32
+    // outputs n >= n2 of row m go to Y2[rows2[m] * ld2 + n - n2] (keys and values straight into their cache cells); Z 1, no paired epilogue
+    float *         Y2 = nullptr; int64_t ld2 = 0; int n2 = 0x7fffffff; const int32_t * rows2 = nullptr;
     int             x_bf16 = 0;                          // 1: X already holds bfloat16 rows (ldx in elements, a multiple of 8): tensor-core path only, no staging copy
 };
 #ifdef __CUDACC__
@@ -234,12 +255,13 @@ template <int EPI, bool FAST> __device__ __forceinline__ float pib_epilogue(floa
     }
     return v;
 }
-__host__ __device__ constexpr bool pib_epi_pairs(int epi) { return epi == PIB_EPI_GLU_PAIR || epi == PIB_EPI_GEGLU_PAIR; }
+__host__ __device__ constexpr bool pib_epi_pairs(int epi) { return epi == PIB_EPI_GLU_PAIR || epi == PIB_EPI_GEGLU_PAIR || epi == PIB_EPI_SWIGLU_PAIR; }
 template <int EPI, bool FAST> __device__ __forceinline__ float pib_glu_pair(float g, float u, float limit) {
     if (EPI == PIB_EPI_GEGLU_PAIR) {      // 0.5 g (1 + tanh z) = g sigmoid(2 z)
         const float z = 0.7978845608028654f * fmaf(0.044715f * g * g, g, g);
         return (FAST ? g / (1.0f + __expf(-2.0f * z)) : 0.5f * g * (1.0f + tanhf(z))) * u;
     }
+    if (EPI == PIB_EPI_SWIGLU_PAIR) return g / (1.0f + (FAST ? __expf(-g) : expf(-g))) * u;
     const float a = fminf(g, limit), b = fminf(fmaxf(u, -limit), limit);
     return a / (1.0f + (FAST ? __expf(-1.702f * a) : expf(-1.702f * a))) * (b + 1.0f);
 }
@@ -272,12 +294,16 @@ int pib_latent_attention(const float * q, int ldq, const float * qlat, const pib
 int pib_latent_attention_mm(const float * q, int ldq, const float * qlat, const pib_hlayer & L, const pib_hbatch & b, const float2 * rope, const float * cache, int cache_row,
                             const int32_t * map, int t0, int nq, int j0, int NK, void * Kb, void * Vt, float * Qc, float * S, void * P, float * ctx, cudaStream_t st);
 int pib_window_softmax(float * S, void * P, int NKp, int NK, int j0, int window, const int32_t * pos, int t0, int n_rows, int rows_per_z, int rep, const float * sink,
-                       cudaStream_t st, int mask = PIB_MASK_WINDOW, int keep = 0, int n_front = 0, float softcap = 0.f);
+                       cudaStream_t st, int mask = PIB_MASK_WINDOW, int keep = 0, int n_front = 0, float softcap = 0.f, const float * slopes = nullptr, const float * rel = nullptr,
+                       int n_rel = 0);
 int pib_hgrn2_gates(float * qfv, int ld, const float * f_bias, const float * lower, int T, int HD, cudaStream_t st);
 int pib_hgrn2_scan(const float * qfv, int ld, const pib_hlayer & L, const pib_hbatch & b, float * state, size_t state_stride, const float * onorm, float eps,
                    float * out, cudaStream_t st);
 int pib_polynorm(float * z, int T, int F, const float * act4, float eps, cudaStream_t st);
-int pib_moe_route(const float * logits, int T, int E, int top, int mode, int32_t * ids, float * wts, cudaStream_t st);
+struct pib_router { int E = 0, top = 0, mode = PIB_ROUTE_SOFTMAX_RENORM, groups = 1, keep_groups = 1; float scale = 1.f; const float * correction = nullptr; };   // E: outputs, identity ones included
+int pib_moe_route(const float * logits, int T, const pib_router & r, int32_t * ids, float * wts, cudaStream_t st);
+bool pib_moe_route_sort_fits(int T, const pib_router & r);
+int pib_moe_route_sort(const float * logits, int T, const pib_router & r, int32_t * ids, float * wts, int32_t * offs, int32_t * perm, int32_t * inv, cudaStream_t st);   // both steps of a small batch in one launch
 int pib_moe_sort(const int32_t * ids, int n_pairs, int E, int32_t * counts, int32_t * offs, int32_t * perm, int32_t * inv, cudaStream_t st);
 int pib_moe_combine(const float * shared, const float * edn, const float * wts, const int32_t * inv, int T, int top, int W, float * y, cudaStream_t st);
 int pib_cellmap_set(int32_t * cellmap, int n_ctx, const pib_hbatch & b, cudaStream_t st);
@@ -286,9 +312,12 @@ int pib_cellmap_set(int32_t * cellmap, int n_ctx, const pib_hbatch & b, cudaStre
 int pib_embed_scale(const pib_weight * embd, const int32_t * tok, float scale, int T, int W, float * x, cudaStream_t st, int copies = 1);
 int pib_rms_norm2(const float * x, const float * w1, const float * w2, float eps, float out_scale, int T, int W, float * h1, float * h2, cudaStream_t st);
 int pib_swa_prep(const float * cv, int ldc, const pib_hlayer & L, float eps, const pib_hbatch & b, float * q, float * cache, int cache_row, float * vfirst, cudaStream_t st);
-int pib_kv_attention(const float * q, const pib_hlayer & L, const pib_hbatch & b, const float * cache, int cache_row, const int32_t * cellmap, int n_ctx, float * out,
+struct pib_kv_query {                // query rows [heads * maps][dim] of token t at q + t * ldq; gate (optional): the heads' outputs are multiplied by sigmoid(gate[t * ldg + i])
+    const float * q; int ldq; const float * gate = nullptr; int ldg = 0;
+};
+int pib_kv_attention(const pib_kv_query & q, const pib_hlayer & L, const pib_hbatch & b, const float * cache, int cache_row, const int32_t * cellmap, int n_ctx, float * out,
                      const int32_t * skip, cudaStream_t st);
-int pib_kv_attention_mm(const float * q, const pib_hlayer & L, const pib_hbatch & b, const float * cache, int cache_row, const int32_t * map, int t0, int nq, int j0, int n_front, int NK,
+int pib_kv_attention_mm(const pib_kv_query & q, const pib_hlayer & L, const pib_hbatch & b, const float * cache, int cache_row, const int32_t * map, int t0, int nq, int j0, int n_front, int NK,
                         void * Kb, void * Vt, float * Qc, float * S, void * P, float * out, cudaStream_t st);
 int pib_token_shift(const float * h, const float * mu, int n_mix, const pib_hbatch & b, float * state, size_t state_stride, size_t shift_off, int W, float * mixes, cudaStream_t st);
 int pib_rows_act(float * z, int ld, int n, int T, int op, const float * bias, cudaStream_t st);           // op 0: tanh; 1: exp(-exp(z + bias))
@@ -333,6 +362,14 @@ int pib_attn_mem_gate(const float * a, const float * mem, const float * dg, cons
                       int ldo, int mem_off, cudaStream_t st);
 int pib_memory_scan(const float * proj, int ldp, int q_off, int k_off, int v_off, float * dg, const pib_hlayer & L, const pib_hbatch & b, float * state, size_t state_stride, float * out,
                     cudaStream_t st, float * split_buf = nullptr, int parts = 0, int per = 0, const int32_t * skip = nullptr);   // mixer_kernels.cu
+// sandwich_kernels.cu
+struct pib_sublayer_y {              // a sublayer's output: y, plus (top > 0) the routed experts: sum_k w_k edn[inv_k], or w_k hin for ids >= n_real (identity outputs)
+    const float * y = nullptr, * edn = nullptr, * wts = nullptr, * hin = nullptr;
+    const int32_t * ids = nullptr, * inv = nullptr;
+    int top = 0, n_real = 0;
+    const float * w = nullptr, * b = nullptr;       // the norm behind it (times layer scale and residual multiplier)
+};
+int pib_sandwich_norm(float * x, const pib_sublayer_y & o, const float * w, const float * b, float eps, int T, int W, float * h, cudaStream_t st);
 // chunk_scan.cu: n tokens of one segment (batch rows t0 ..) of a recurrence with one decay per head and token, as matmuls (served mode)
 struct pib_chunk_scan {
     const float * q = nullptr, * k = nullptr, * v = nullptr; int ldq = 0, ldk = 0, ldv = 0;   // rows [G][D], [G][D], [H][V] per token

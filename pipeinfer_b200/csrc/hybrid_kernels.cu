@@ -395,12 +395,20 @@ __global__ void __launch_bounds__(128) lat_qcat_kernel(const float * __restrict_
     for (int i = threadIdx.x; i < rot_dim; i += blockDim.x) out[R + i] = rot_coord(qr, i, rot_dims, pairs, cs) * scale;
 }
 // one score row per (token, head), in place: keys outside [p - window + 1, p] (chunk mask: outside [p - p % window, p]) and the pad get weight 0, the sink (optional) one share of
-// the denominator.  The first `keep` positions are read from everywhere: columns [0, n_front) are positions 0 .. n_front - 1 (n_front is 0 or keep), the columns
+// the denominator.  Distance biases (optional) join the scores behind the cap.  The first `keep` positions are read from everywhere: columns [0, n_front) are positions 0 .. n_front - 1 (n_front is 0 or keep), the columns
 // behind them positions j0, j0 + 1, ... (n_front 0: then j0 is 0 or nothing is kept).  softcap > 0: a score becomes softcap tanh(score / softcap) first.  Rows come in groups of rows_per_z (one group per problem of the score matmul), inside a group `rep` heads per token:
 // token t0 + (row % rows_per_z) / rep, head (row / rows_per_z) * rep + (row % rows_per_z) % rep.
+// what the distance of column j's position from p adds to a score of head h: -slopes[h] distance, rel[h][min(distance, n_rel - 1)]
+__device__ __forceinline__ float dist_bias(int p, int j, int j0, int n_front, const float * __restrict__ slopes, const float * __restrict__ rel, int n_rel, int h) {
+    const int d = p - (j < n_front ? j : j0 + j - n_front);
+    float v = 0.f;
+    if (slopes) v -= slopes[h] * (float) d;
+    if (rel) v += rel[(size_t) h * n_rel + min(d, n_rel - 1)];
+    return v;
+}
 __global__ void __launch_bounds__(256) lat_softmax_kernel(float * __restrict__ S, __nv_bfloat16 * __restrict__ P, int NKp, int NK, int j0, int window,
                                                           const int32_t * __restrict__ pos, int t0, int rows_per_z, int rep, const float * __restrict__ sink, int mask, int keep, int n_front,
-                                                          float softcap) {
+                                                          float softcap, const float * __restrict__ slopes, const float * __restrict__ rel, int n_rel) {
     pib_pdl_wait();
     pib_pdl_trigger();
     __shared__ float red[32];
@@ -414,7 +422,9 @@ __global__ void __launch_bounds__(256) lat_softmax_kernel(float * __restrict__ S
     for (int e = threadIdx.x; e < ka + hi - lo + 1; e += blockDim.x) {
         const int j = e < ka ? e : lo + e - ka;
         float v = s[j];
-        if (softcap > 0.f) { v = softcap * tanhf(v / softcap); s[j] = v; }
+        if (softcap > 0.f) v = softcap * tanhf(v / softcap);
+        v += dist_bias(p, j, j0, n_front, slopes, rel, n_rel, h);
+        s[j] = v;
         m = fmaxf(m, v);
     }
     m = warp_max(m);
@@ -441,7 +451,8 @@ __global__ void __launch_bounds__(256) lat_softmax_kernel(float * __restrict__ S
 // (only where a key is seen) and its weights leave in one pass
 template <int NR>
 __global__ void __launch_bounds__(256) row_softmax_kernel(const float * __restrict__ S, __nv_bfloat16 * __restrict__ P, int NKp, int j0, int window, const int32_t * __restrict__ pos, int t0,
-                                                          int rows_per_z, int rep, const float * __restrict__ sink, int mask, int keep, int n_front, float softcap) {
+                                                          int rows_per_z, int rep, const float * __restrict__ sink, int mask, int keep, int n_front, float softcap,
+                                                          const float * __restrict__ slopes, const float * __restrict__ rel, int n_rel) {
     pib_pdl_wait();
     pib_pdl_trigger();
     __shared__ float red[32];
@@ -461,6 +472,10 @@ __global__ void __launch_bounds__(256) row_softmax_kernel(const float * __restri
             const float2 x = *reinterpret_cast<const float2 *>(s + j);
             if (a) v[i].x = softcap > 0.f ? softcap * tanhf(x.x * icap) : x.x;
             if (b) v[i].y = softcap > 0.f ? softcap * tanhf(x.y * icap) : x.y;
+            if (slopes || rel) {
+                if (a) v[i].x += dist_bias(p, j, j0, n_front, slopes, rel, n_rel, h);
+                if (b) v[i].y += dist_bias(p, j + 1, j0, n_front, slopes, rel, n_rel, h);
+            }
             m = fmaxf(m, fmaxf(v[i].x, v[i].y));
         }
     }
@@ -484,11 +499,11 @@ __global__ void __launch_bounds__(256) row_softmax_kernel(const float * __restri
     }
 }
 int pib_window_softmax(float * S, void * P, int NKp, int NK, int j0, int window, const int32_t * pos, int t0, int n_rows, int rows_per_z, int rep, const float * sink,
-                       cudaStream_t st, int mask, int keep, int n_front, float softcap) {
-#define SM_GO(NR) pib_launch(row_softmax_kernel<NR>, dim3(n_rows), dim3(256), (size_t) 0, st, (const float *) S, (__nv_bfloat16 *) P, NKp, j0, window, pos, t0, rows_per_z, rep, sink, mask, keep, n_front, softcap)
+                       cudaStream_t st, int mask, int keep, int n_front, float softcap, const float * slopes, const float * rel, int n_rel) {
+#define SM_GO(NR) pib_launch(row_softmax_kernel<NR>, dim3(n_rows), dim3(256), (size_t) 0, st, (const float *) S, (__nv_bfloat16 *) P, NKp, j0, window, pos, t0, rows_per_z, rep, sink, mask, keep, n_front, softcap, slopes, rel, n_rel)
     if (NKp <= 512) SM_GO(1); else if (NKp <= 1024) SM_GO(2); else if (NKp <= 2048) SM_GO(4); else if (NKp <= 4096) SM_GO(8);
 #undef SM_GO
-    else pib_launch(lat_softmax_kernel, dim3(n_rows), dim3(256), (size_t) (0), st, S, (__nv_bfloat16 *) P, NKp, NK, j0, window, pos, t0, rows_per_z, rep, sink, mask, keep, n_front, softcap);
+    else pib_launch(lat_softmax_kernel, dim3(n_rows), dim3(256), (size_t) (0), st, S, (__nv_bfloat16 *) P, NKp, NK, j0, window, pos, t0, rows_per_z, rep, sink, mask, keep, n_front, softcap, slopes, rel, n_rel);
     CKL();
     return PIB_OK;
 }
@@ -669,48 +684,119 @@ int pib_polynorm(float * z, int T, int F, const float * act4, float eps, cudaStr
 }
 
 // ---- mixture of experts ------------------------------------------------------------------------------------------------------------
-// one warp per token: the `top` largest logits (ties: the lower index).  mode PIB_ROUTE_SOFTMAX_RENORM: scores = softmax over the E
-// logits, weights = score / (sum of the chosen + 1e-20); PIB_ROUTE_SIGMOID: weights = sigmoid(logit) of the chosen, as they are (the
-// order of the logits is the order of their sigmoids)
+// One warp per token: the `top` outputs of the router with the largest choice value (ties: the lower index).
+//   PIB_ROUTE_SOFTMAX_RENORM:  scores = softmax over the E logits, weights = score / (sum of the chosen + 1e-20); chosen by the logits
+//   PIB_ROUTE_SIGMOID:         weights = sigmoid(logit) of the chosen, as they are (the order of the logits is the order of their sigmoids)
+//   PIB_ROUTE_SOFTMAX_GROUPS:  scores = softmax over the E logits; the choice values are score + correction; the outputs form equal groups of neighbours, a group
+//                              stands for its largest choice value, and only members of the keep_groups best groups are chosen; weights = score * scale
+// cv: the warp's scratch in shared memory, E + groups floats.  Output k of the token goes to ids[k], wts[k].
 #define MOE_MAX_TOP 16
-__global__ void moe_route_kernel(const float * __restrict__ logits, int T, int E, int top, int mode, int32_t * __restrict__ ids, float * __restrict__ wts) {
-    pib_pdl_wait();
-    pib_pdl_trigger();
-    const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-    if (t >= T) return;
-    const float * z = logits + (size_t) t * E;
+__device__ __forceinline__ void moe_route_token(const float * __restrict__ z, const pib_router & R, float * cv, int lane, int32_t * ids, float * wts) {
+    const int E = R.E;
     float mx = -INFINITY;
     for (int i = lane; i < E; i += 32) mx = fmaxf(mx, z[i]);
     mx = warp_max(mx);
     float sum = 0.f;
     for (int i = lane; i < E; i += 32) sum += expf(z[i] - mx);
     sum = warp_sum(sum);
+    const bool grouped = R.mode == PIB_ROUTE_SOFTMAX_GROUPS;
+    for (int i = lane; i < E; i += 32) cv[i] = grouped ? expf(z[i] - mx) / sum + (R.correction ? R.correction[i] : 0.f) : z[i];
+    if (grouped && R.keep_groups < R.groups) {
+        float *   gv  = cv + E;
+        const int per = E / R.groups;
+        __syncwarp();
+        for (int g = lane; g < R.groups; g += 32) {
+            float best = -INFINITY;
+            for (int i = g * per; i < (g + 1) * per; i++) best = fmaxf(best, cv[i]);
+            gv[g] = best;
+        }
+        __syncwarp();
+        for (int i = lane; i < E; i += 32) {
+            const int g = i / per;
+            int better = 0;
+            for (int o = 0; o < R.groups; o++) better += gv[o] > gv[g] || (gv[o] == gv[g] && o < g);
+            if (better >= R.keep_groups) cv[i] = -INFINITY;
+        }
+    }
+    float tot = 0.f, score[MOE_MAX_TOP];
     int   chosen[MOE_MAX_TOP];
-    float score[MOE_MAX_TOP], tot = 0.f;
-    for (int k = 0; k < top; k++) {
+    for (int k = 0; k < R.top; k++) {
         float bv = -INFINITY;
         int   bi = 0x7fffffff;
-        for (int i = lane; i < E; i += 32) {
-            bool taken = false;
-            for (int j = 0; j < k; j++) taken |= chosen[j] == i;
-            const float v = z[i];
-            if (!taken && (v > bv || (v == bv && i < bi))) { bv = v; bi = i; }
-        }
+        for (int i = lane; i < E; i += 32) { const float v = cv[i]; if (v > bv || (v == bv && v > -INFINITY && i < bi)) { bv = v; bi = i; } }      // a lane reads back only what it wrote
         for (int o = 16; o > 0; o >>= 1) {
             const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
             const int   oi = __shfl_xor_sync(0xffffffffu, bi, o);
             if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
         }
+        if (bi >= E) bi = k;                                // nothing comparable is left (logits that are no numbers): stay inside the arrays
+        if ((bi & 31) == lane) cv[bi] = -INFINITY;
         chosen[k] = bi;
-        score[k]  = mode == PIB_ROUTE_SIGMOID ? 1.0f / (1.0f + expf(-bv)) : expf(bv - mx) / sum;
+        score[k]  = R.mode == PIB_ROUTE_SIGMOID ? 1.0f / (1.0f + expf(-z[bi])) : expf(z[bi] - mx) / sum;
         tot += score[k];
     }
     if (lane == 0)
-        for (int k = 0; k < top; k++) { ids[(size_t) t * top + k] = chosen[k]; wts[(size_t) t * top + k] = mode == PIB_ROUTE_SIGMOID ? score[k] : score[k] / (tot + 1e-20f); }
+        for (int k = 0; k < R.top; k++) {
+            ids[k] = chosen[k];
+            wts[k] = R.mode == PIB_ROUTE_SIGMOID ? score[k] : grouped ? score[k] * R.scale : score[k] / (tot + 1e-20f);
+        }
 }
-int pib_moe_route(const float * logits, int T, int E, int top, int mode, int32_t * ids, float * wts, cudaStream_t st) {
-    if (top > MOE_MAX_TOP || top > E) { pib_set_error("router: top %d of %d experts (max %d)", top, E, MOE_MAX_TOP); return PIB_ERR_UNSUPP; }
-    pib_launch(moe_route_kernel, dim3((T + 7) / 8), dim3(256), (size_t) (0), st, logits, T, E, top, mode, ids, wts);
+__global__ void __launch_bounds__(128) moe_route_kernel(const float * __restrict__ logits, int T, pib_router R, int32_t * __restrict__ ids, float * __restrict__ wts) {
+    pib_pdl_wait();
+    pib_pdl_trigger();
+    extern __shared__ float route_sm[];
+    const int warp = threadIdx.x >> 5, t = blockIdx.x * (blockDim.x >> 5) + warp;
+    if (t >= T) return;
+    moe_route_token(logits + (size_t) t * R.E, R, route_sm + (size_t) warp * (R.E + R.groups), threadIdx.x & 31, ids + (size_t) t * R.top, wts + (size_t) t * R.top);
+}
+static int moe_router_check(const pib_router & R) {
+    if (R.top < 1 || R.top > MOE_MAX_TOP || R.top > R.E) { pib_set_error("router: top %d of %d experts (max %d)", R.top, R.E, MOE_MAX_TOP); return PIB_ERR_UNSUPP; }
+    if (R.groups < 1 || R.E % R.groups || R.keep_groups < 1 || R.keep_groups > R.groups || R.top > R.keep_groups * (R.E / R.groups)) {
+        pib_set_error("router: %d outputs in %d groups of which %d take part, top %d", R.E, R.groups, R.keep_groups, R.top); return PIB_ERR_UNSUPP;
+    }
+    if (4 * (R.E + R.groups) * 4 > 48 * 1024) { pib_set_error("router: %d outputs", R.E); return PIB_ERR_UNSUPP; }
+    return PIB_OK;
+}
+int pib_moe_route(const float * logits, int T, const pib_router & R, int32_t * ids, float * wts, cudaStream_t st) {
+    const int rc = moe_router_check(R);
+    if (rc != PIB_OK) return rc;
+    pib_launch(moe_route_kernel, dim3((T + 3) / 4), dim3(128), (size_t) 16 * (R.E + R.groups), st, logits, T, R, ids, wts);
+    CKL();
+    return PIB_OK;
+}
+
+// routing and sorting of a small batch in one block: a warp per token in turn, then a thread per router output counts and places its pairs (in pair order, as
+// the kernels below do)
+#define MOE_SMALL_T 16
+#define MOE_SMALL_PAIRS 256
+__global__ void __launch_bounds__(512) moe_route_sort_kernel(const float * __restrict__ logits, int T, pib_router R, int32_t * __restrict__ ids, float * __restrict__ wts,
+                                                             int32_t * __restrict__ offs, int32_t * __restrict__ perm, int32_t * __restrict__ inv) {
+    pib_pdl_wait();
+    pib_pdl_trigger();
+    extern __shared__ float route_sm[];
+    __shared__ int32_t sid[MOE_SMALL_PAIRS], cnt[512];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, P = T * R.top;
+    if (warp < T) moe_route_token(logits + (size_t) warp * R.E, R, route_sm + (size_t) warp * (R.E + R.groups), lane, sid + warp * R.top, wts + (size_t) warp * R.top);
+    __syncthreads();
+    for (int i = threadIdx.x; i < P; i += blockDim.x) ids[i] = sid[i];
+    const int e = threadIdx.x;
+    int n = 0;
+    for (int i = 0; i < P; i++) n += sid[i] == e;
+    cnt[e] = n;
+    __syncthreads();
+    if (e >= R.E) return;
+    int o = 0;
+    for (int i = 0; i < e; i++) o += cnt[i];
+    offs[e] = o;
+    if (e == R.E - 1) offs[R.E] = o + n;
+    if (n > 0) for (int i = 0; i < P; i++) if (sid[i] == e) { perm[o] = i; inv[i] = o; o++; }
+}
+bool pib_moe_route_sort_fits(int T, const pib_router & R) { return T <= MOE_SMALL_T && T * R.top <= MOE_SMALL_PAIRS && R.E <= 512 && (size_t) T * (R.E + R.groups) * 4 <= 40 * 1024; }
+int pib_moe_route_sort(const float * logits, int T, const pib_router & R, int32_t * ids, float * wts, int32_t * offs, int32_t * perm, int32_t * inv, cudaStream_t st) {
+    const int rc = moe_router_check(R);
+    if (rc != PIB_OK) return rc;
+    const int threads = ((R.E > 32 * T ? R.E : 32 * T) + 31) & ~31;
+    pib_launch(moe_route_sort_kernel, dim3(1), dim3(threads), (size_t) T * (R.E + R.groups) * 4, st, logits, T, R, ids, wts, offs, perm, inv);
     CKL();
     return PIB_OK;
 }

@@ -2,7 +2,8 @@
 //
 //   embedding rows times a constant; RMS norm with a weight stored around zero, two norms of the same row in one pass
 //   windowed softmax attention over cached key / value heads: per-head RMS norm of queries and keys, value mixing with the values an
-//       earlier layer computed for the same token, grouped queries, an optional sink logit
+//       earlier layer computed for the same token, grouped queries, an optional sink logit, optional distance biases (a slope per head, or a
+//       table per head over distances) and an optional sigmoid gate on every output value
 //   RWKV-style time mixing: the five token-shift mixes, the per-channel decay, and the recurrence
 //       o_t = (S + diag(u) k_t v_t^T)^T r_t,  S <- diag(w_t) S + k_t v_t^T
 //   the gated delta rule: S <- g_t S,  e_t = beta_t (v_t - S^T k_t),  S <- S + k_t e_t^T,  o_t = S^T q_t
@@ -107,46 +108,79 @@ int pib_swa_prep(const float * cv, int ldc, const pib_hlayer & L, float eps, con
 }
 
 // grid (token, head group); a block holds HPB query heads x KS key shares, one warp each.  A warp walks its share of the window
-// [max(0, p - window + 1), p] (chunk mask: of the token's chunk [p - p % window, p]) and the kept first positions [0, keep) through the slot's position -> cell table, keeps a running maximum / denominator / weighted sum of value
+// [max(0, p - window + 1), p] (chunk mask: of the token's chunk [p - p % window, p]) and the kept first positions [0, keep) through the slot's position -> cell table, UK
+// keys per trip (their rows are in flight together and their sums cross the lanes side by side), keeps a running maximum / denominator / weighted sum of value
 // rows, and the shares of a head are merged in shared memory.  A sink (optional) is one more logit without a row: the running state of
-// share 0 starts at (max = sink, denominator = 1).  softcap > 0: a score becomes softcap tanh(score / softcap).
-template <int RPL>
-__global__ void __launch_bounds__(512) kv_attn_kernel(const float * __restrict__ q, int H, int G, int maps, int D, int V, float scale, int window, int mask, int keep, float softcap, const float * __restrict__ sink,
-                                                      const int32_t * __restrict__ pos, const int32_t * __restrict__ slot, const float * __restrict__ cache, int cache_row,
-                                                      const int32_t * __restrict__ cellmap, int n_ctx, int HPB, int KS, float * __restrict__ out,
-                                                      const int32_t * __restrict__ skip) {
+// share 0 starts at (max = sink, denominator = 1).  softcap > 0: a score becomes softcap tanh(score / softcap).  Distance biases (optional) join the score
+// behind the cap: -slopes[h] (p - j), or rel[h][min(p - j, n_rel - 1)].  gate (optional): every output value is multiplied by sigmoid(gate).
+struct kva_args {
+    pib_kv_query q;
+    int H, G, maps, D, V;
+    float scale; int window, mask, keep; float softcap;
+    const float * sink, * slopes, * rel; int n_rel;
+    const int32_t * pos, * slot;
+    const float * cache; int cache_row;
+    const int32_t * cellmap; int n_ctx, HPB, KS;
+    float * out;
+    const int32_t * skip;
+};
+template <int RPL, int UK>
+__global__ void __launch_bounds__(512) kv_attn_kernel(kva_args A) {
     pib_pdl_wait();
     pib_pdl_trigger();
     extern __shared__ float sm[];                 // [HPB * KS][V + 2] partial states
-    const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    if (skip && skip[t]) return;                  // this token's segment goes through the matmul form
-    const int hl = warp / KS, ks = warp % KS, h = blockIdx.y * HPB + hl;
-    const int p = pos[t], lo = mask == PIB_MASK_CHUNK ? p - p % window : max(0, p - window + 1);
+    const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, H = A.H, D = A.D, V = A.V, KS = A.KS;
+    if (A.skip && A.skip[t]) return;              // this token's segment goes through the matmul form
+    const int hl = warp / KS, ks = warp % KS, h = blockIdx.y * A.HPB + hl;
+    const int p = A.pos[t], lo = A.mask == PIB_MASK_CHUNK ? p - p % A.window : max(0, p - A.window + 1);
     const bool live = h < H;
     float qv[RPL], acc[RPL];
     float m = -INFINITY, l = 0.f;
     if (live) {
         // H counts query rows: `maps` rows per head, next to each other; row h reads map h % maps of its key / value head's keys and that head's values
-        const int g = h / maps / (H / (G * maps)), mp = h % maps;
-        const float * qp = q + ((size_t) t * H + h) * D;
+        const int g = h / A.maps / (H / (A.G * A.maps)), mp = h % A.maps;
+        const float * qp = A.q.q + (size_t) t * A.q.ldq + (size_t) h * D;
 #pragma unroll
-        for (int i = 0; i < RPL; i++) { const int r = i * 32 + lane; qv[i] = r < D ? qp[r] * scale : 0.f; acc[i] = 0.f; }
-        if (ks == 0 && sink) { m = sink[h]; l = 1.f; }
-        const int32_t * map = cellmap + (size_t) slot[t] * n_ctx;
-        const size_t ko = (size_t) (g * maps + mp) * D, vo = (size_t) G * maps * D + (size_t) g * V;
-        const int nf = min(keep, lo), n_keys = nf + p - lo + 1;          // kept positions in front of the window, then the window
-        for (int e = ks; e < n_keys; e += KS) {
-            const int     j   = e < nf ? e : lo + e - nf;
-            const float * row = cache + (size_t) map[j] * cache_row;
-            float s = 0.f, c[RPL];
+        for (int i = 0; i < RPL; i++) { const int r = i * 32 + lane; qv[i] = r < D ? qp[r] * A.scale : 0.f; acc[i] = 0.f; }
+        if (ks == 0 && A.sink) { m = A.sink[h]; l = 1.f; }
+        const int32_t * map = A.cellmap + (size_t) A.slot[t] * A.n_ctx;
+        const float *   rel = A.rel ? A.rel + (size_t) h * A.n_rel : nullptr;
+        const float     slope = A.slopes ? A.slopes[h] : 0.f;
+        const size_t ko = (size_t) (g * A.maps + mp) * D, vo = (size_t) A.G * A.maps * D + (size_t) g * V;
+        const int nf = min(A.keep, lo), n_keys = nf + p - lo + 1;        // kept positions in front of the window, then the window
+        for (int e0 = ks; e0 < n_keys; e0 += KS * UK) {
+            float s[UK], c[UK][RPL];
+            int   dist[UK];
 #pragma unroll
-            for (int i = 0; i < RPL; i++) { const int r = i * 32 + lane; if (r < D) s = fmaf(qv[i], row[ko + r], s); c[i] = r < V ? row[vo + r] : 0.f; }
-            s = warp_sum(s);
-            if (softcap > 0.f) s = softcap * tanhf(s / softcap);
-            const float mn = fmaxf(m, s), a = expf(m - mn), w = expf(s - mn);         // m == -inf only before the first key: a = 0
-            l = l * a + w;
+            for (int u = 0; u < UK; u++) {
+                const int e = min(e0 + u * KS, n_keys - 1), j = e < nf ? e : lo + e - nf;      // a trip past the end reads the last key again; its score is dropped below
+                dist[u] = p - j;
+                const float * row = A.cache + (size_t) map[j] * A.cache_row;
+                s[u] = 0.f;
 #pragma unroll
-            for (int i = 0; i < RPL; i++) acc[i] = fmaf(acc[i], a, w * c[i]);
+                for (int i = 0; i < RPL; i++) { const int r = i * 32 + lane; if (r < D) s[u] = fmaf(qv[i], row[ko + r], s[u]); c[u][i] = r < V ? row[vo + r] : 0.f; }
+            }
+            float mn = m;
+#pragma unroll
+            for (int u = 0; u < UK; u++) {
+                s[u] = warp_sum(s[u]);
+                if (A.softcap > 0.f) s[u] = A.softcap * tanhf(s[u] / A.softcap);
+                if (A.slopes) s[u] -= slope * (float) dist[u];
+                if (rel) s[u] += rel[min(dist[u], A.n_rel - 1)];
+                if (UK > 1 && e0 + u * KS >= n_keys) s[u] = -INFINITY;
+                mn = fmaxf(mn, s[u]);
+            }
+            const float a = expf(m - mn);                                              // m == -inf only before the first key: a = 0
+            l *= a;
+#pragma unroll
+            for (int i = 0; i < RPL; i++) acc[i] *= a;
+#pragma unroll
+            for (int u = 0; u < UK; u++) {
+                const float w = expf(s[u] - mn);
+                l += w;
+#pragma unroll
+                for (int i = 0; i < RPL; i++) acc[i] = fmaf(w, c[u][i], acc[i]);
+            }
             m = mn;
         }
         float * part = sm + (size_t) warp * (V + 2);
@@ -172,13 +206,14 @@ __global__ void __launch_bounds__(512) kv_attn_kernel(const float * __restrict__
             for (int i = 0; i < RPL; i++) { const int r = i * 32 + lane; if (r < V) o[i] = fmaf(pk[r], f, o[i]); }
         }
         const float inv = 1.0f / Lsum;
-        float * op = out + ((size_t) t * H + h) * V;
+        float * op = A.out + ((size_t) t * H + h) * V;
+        const float * gp = A.q.gate ? A.q.gate + (size_t) t * A.q.ldg + (size_t) h * V : nullptr;
 #pragma unroll
-        for (int i = 0; i < RPL; i++) { const int r = i * 32 + lane; if (r < V) op[r] = o[i] * inv; }
+        for (int i = 0; i < RPL; i++) { const int r = i * 32 + lane; if (r < V) op[r] = o[i] * inv * (gp ? mk_sigmoid(gp[r]) : 1.0f); }
     }
 }
 
-int pib_kv_attention(const float * q, const pib_hlayer & L, const pib_hbatch & b, const float * cache, int cache_row, const int32_t * cellmap, int n_ctx, float * out,
+int pib_kv_attention(const pib_kv_query & q, const pib_hlayer & L, const pib_hbatch & b, const float * cache, int cache_row, const int32_t * cellmap, int n_ctx, float * out,
                      const int32_t * skip, cudaStream_t st) {
     const int H = L.heads * L.maps, V = L.vdim, R = L.dim > L.vdim ? L.dim : L.vdim;
     const int HPB = (long long) b.T * H <= 1024 ? 1 : (H < 4 ? H : 4);
@@ -187,12 +222,13 @@ int pib_kv_attention(const float * q, const pib_hlayer & L, const pib_hbatch & b
     const size_t smem = (size_t) HPB * KS * (V + 2) * 4;
     dim3 grid((unsigned) b.T, (unsigned) ((H + HPB - 1) / HPB));
     const int threads = HPB * KS * 32;
-#define KA_GO(RPL) do {                                                                                                              \
-        if (smem > 48 * 1024) cudaFuncSetAttribute(kv_attn_kernel<RPL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int) smem);   \
-        pib_launch(kv_attn_kernel<RPL>, dim3(grid), dim3(threads), (size_t) smem, st, q, H, L.kv_heads, L.maps, L.dim, V, L.scale, L.window, L.mask, L.keep, L.softcap, (const float *) L.sink, b.pos, b.slot, cache, \
-                   cache_row, cellmap, n_ctx, HPB, KS, out, skip);                                                                  \
+    const kva_args A = { q, H, L.kv_heads, L.maps, L.dim, V, L.scale, L.window, L.mask, L.keep, L.softcap, L.sink, L.slopes, L.rel, L.n_rel, b.pos, b.slot, cache, cache_row, cellmap, n_ctx,
+                         HPB, KS, out, skip };
+#define KA_GO(RPL, UK) do {                                                                                                              \
+        if (smem > 48 * 1024) cudaFuncSetAttribute(kv_attn_kernel<RPL, UK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int) smem);   \
+        pib_launch(kv_attn_kernel<RPL, UK>, dim3(grid), dim3(threads), (size_t) smem, st, A);                                           \
     } while (0)
-    if (R <= 32) KA_GO(1); else if (R <= 64) KA_GO(2); else if (R <= 128) KA_GO(4); else if (R <= 256) KA_GO(8); else if (R <= 512) KA_GO(16);
+    if (R <= 32) KA_GO(1, 4); else if (R <= 64) KA_GO(2, 4); else if (R <= 128) KA_GO(4, 4); else if (R <= 256) KA_GO(8, 2); else if (R <= 512) KA_GO(16, 1);
     else { pib_set_error("attention: head size %d (max 512)", R); return PIB_ERR_UNSUPP; }
 #undef KA_GO
     CKL();
@@ -258,12 +294,12 @@ __device__ __forceinline__ size_t kv_problem_row(int h, int maps, int rep, int n
     return (size_t) z * nq * rep + (size_t) ti * rep + hq % rep;
 }
 // Qc[z][ti * rep + hr] = [hi | lo | hi] of scale * q[t0 + ti][h]
-__global__ void __launch_bounds__(256) kv_query_rows_kernel(const float * __restrict__ q, __nv_bfloat16 * __restrict__ Qc, int H, int maps, int rep, int nq, int D, int t0, float scale) {
+__global__ void __launch_bounds__(256) kv_query_rows_kernel(const float * __restrict__ q, int ldq, __nv_bfloat16 * __restrict__ Qc, int H, int maps, int rep, int nq, int D, int t0, float scale) {
     pib_pdl_wait();
     pib_pdl_trigger();
     const int ti = blockIdx.x;
     for (int h = threadIdx.x >> 5; h < H; h += blockDim.x >> 5) {           // a warp per query row
-        const float * src = q + ((size_t) (t0 + ti) * H + h) * D;
+        const float * src = q + (size_t) (t0 + ti) * ldq + (size_t) h * D;
         __nv_bfloat16 * dst = Qc + kv_problem_row(h, maps, rep, nq, ti) * 3 * D;
         for (int i = threadIdx.x & 31; i < D; i += 32) {
             __nv_bfloat16 hi, lo;
@@ -272,36 +308,38 @@ __global__ void __launch_bounds__(256) kv_query_rows_kernel(const float * __rest
         }
     }
 }
-// out[t0 + ti][h][V] = O[z][ti * rep + hr][V]
-__global__ void __launch_bounds__(256) kv_token_order_kernel(const float * __restrict__ O, float * __restrict__ out, int H, int maps, int rep, int nq, int V, int t0) {
+// out[t0 + ti][h][V] = O[z][ti * rep + hr][V], times the sigmoid of the gate where there is one
+__global__ void __launch_bounds__(256) kv_token_order_kernel(const float * __restrict__ O, float * __restrict__ out, const float * __restrict__ gate, int ldg, int H, int maps, int rep, int nq,
+                                                             int V, int t0) {
     pib_pdl_wait();
     pib_pdl_trigger();
     const int ti = blockIdx.x;
     for (int h = threadIdx.x >> 5; h < H; h += blockDim.x >> 5) {
         const float * src = O + kv_problem_row(h, maps, rep, nq, ti) * V;
         float * dst = out + ((size_t) (t0 + ti) * H + h) * V;
-        for (int i = threadIdx.x & 31; i < V; i += 32) dst[i] = src[i];
+        const float * gp = gate ? gate + (size_t) (t0 + ti) * ldg + (size_t) h * V : nullptr;
+        for (int i = threadIdx.x & 31; i < V; i += 32) dst[i] = gp ? src[i] * mk_sigmoid(gp[i]) : src[i];
     }
 }
-int pib_kv_attention_mm(const float * q, const pib_hlayer & L, const pib_hbatch & b, const float * cache, int cache_row, const int32_t * map, int t0, int nq, int j0, int n_front, int NK,
+int pib_kv_attention_mm(const pib_kv_query & q, const pib_hlayer & L, const pib_hbatch & b, const float * cache, int cache_row, const int32_t * map, int t0, int nq, int j0, int n_front, int NK,
                         void * Kb, void * Vt, float * Qc, float * S, void * P, float * out, cudaStream_t st) {
     const int maps = L.maps, H = L.heads * maps, G = L.kv_heads, GK = G * maps, D = L.dim, V = L.vdim, rep = L.heads / G, NKp = (NK + 7) & ~7, M = nq * rep;
     if (maps > 1 && L.sink) { pib_set_error("attention: a sink with several maps per head"); return PIB_ERR_UNSUPP; }
     pib_launch(kv_gather_kernel, dim3((unsigned) ((NKp + 31) / 32), (unsigned) GK, 2), dim3(256), (size_t) 0, st, cache, cache_row, map, j0, n_front, NK, NKp, G, maps, D, V, (__nv_bfloat16 *) Kb, (__nv_bfloat16 *) Vt);
     CKL();
-    pib_launch(kv_query_rows_kernel, dim3((unsigned) nq), dim3(256), (size_t) 0, st, q, (__nv_bfloat16 *) Qc, H, maps, rep, nq, D, t0, L.scale);
+    pib_launch(kv_query_rows_kernel, dim3((unsigned) nq), dim3(256), (size_t) 0, st, q.q, q.ldq, (__nv_bfloat16 *) Qc, H, maps, rep, nq, D, t0, L.scale);
     CKL();
     pib_mm a;
     a.W = Kb; a.wtype = PIB_TYPE_BF16; a.ldw = 3 * D; a.wz = (int64_t) NKp * 3 * D; a.X = Qc; a.ldx = 3 * D; a.xz = (int64_t) M * 3 * D; a.x_bf16 = 1;
     a.Y = S; a.ldy = NKp; a.yz = (int64_t) M * NKp; a.M = M; a.N = NK; a.K = 3 * D; a.Z = GK;
     int rc = pib_dense_mm(a, st);
     if (rc != PIB_OK) return rc;
-    if ((rc = pib_window_softmax(S, P, NKp, NK, j0, L.window, b.pos, t0, GK * M, M, rep, L.sink, st, L.mask, L.keep, n_front, L.softcap)) != PIB_OK) return rc;
+    if ((rc = pib_window_softmax(S, P, NKp, NK, j0, L.window, b.pos, t0, GK * M, M, rep, L.sink, st, L.mask, L.keep, n_front, L.softcap, L.slopes, L.rel, L.n_rel)) != PIB_OK) return rc;
     pib_mm v;
     v.W = Vt; v.wtype = PIB_TYPE_BF16; v.ldw = 2 * NKp; v.wz = (int64_t) V * 2 * NKp; v.X = (const float *) P; v.ldx = 2 * NKp; v.xz = (int64_t) M * 2 * NKp; v.x_bf16 = 1;
     v.Y = Qc; v.ldy = V; v.yz = (int64_t) M * V; v.M = M; v.N = V; v.K = 2 * NKp; v.Z = GK;              // the query rows are used up: the outputs take their place
     if ((rc = pib_dense_mm(v, st)) != PIB_OK) return rc;
-    pib_launch(kv_token_order_kernel, dim3((unsigned) nq), dim3(256), (size_t) 0, st, (const float *) Qc, out, H, maps, rep, nq, V, t0);
+    pib_launch(kv_token_order_kernel, dim3((unsigned) nq), dim3(256), (size_t) 0, st, (const float *) Qc, out, q.gate, q.ldg, H, maps, rep, nq, V, t0);
     CKL();
     return PIB_OK;
 }

@@ -183,13 +183,14 @@ struct TensorSource {
         for (char ch : name) h = (h ^ (uint8_t) ch) * 0x100000001B3ull;
         auto next = [&]() { h ^= h << 13; h ^= h >> 7; h ^= h << 17; return (float) ((h >> 11) & 0xFFFFFF) / 16777216.0f; };     // [0, 1)
         const int64_t last = shape.size() ? *(shape.end() - 1) : 1;
-        const bool norm = ends(name, "norm") || ends(name, "norm1") || ends(name, "norm2");
+        const bool norm = ends(name, "norm") || ends(name, "norm1") || ends(name, "norm2") || ends(name, "norm1b") || ends(name, "norm2b") || ends(name, ".ls1") || ends(name, ".ls2");
+        const bool norm_bias = ends(name, "norm.b") || ends(name, "norm1.b") || ends(name, "norm2.b") || ends(name, "norm1b.b") || ends(name, "norm2b.b");
         const bool around_zero = norms_around_zero && (ends(name, "norm1") || ends(name, "norm2") || name == "final.norm");
         const float amp = 1.5f * sqrtf(3.0f / (float) last);
         for (size_t i = 0; i < out.size(); i++) {
             const float u = next() * 2.f - 1.f;
             float v;
-            if (around_zero) v = 0.2f * u;
+            if (around_zero || norm_bias || ends(name, ".correction")) v = 0.2f * u;
             else if (norm) v = 1.0f + 0.2f * u;
             else if (name.find(".mu.") != std::string::npos) v = 0.5f + 0.5f * u;
             else if (name.find(".hc") != std::string::npos)                // hyper-connections: read about evenly, write with weights near 1, mix near the identity
@@ -231,13 +232,20 @@ static pib_weight * upload_mat(const std::vector<float> & v, int64_t N, int64_t 
 }
 
 // gate row i and up row i next to each other: the matmul's paired epilogue forms the activation on the way out
-static pib_weight * upload_gate_up(TensorSource & src, const std::string & pre, int ff, int W, int dtype, pib_model * m) {
-    std::vector<float> v, all((size_t) 2 * ff * W);
+static bool append_gate_up(TensorSource & src, const std::string & pre, int ff, int W, std::vector<float> & all) {
+    const size_t at = all.size();
+    std::vector<float> v;
+    all.resize(at + (size_t) 2 * ff * W);
     const char * names[2] = { "gate", "up" };
     for (int k = 0; k < 2; k++) {
-        if (!src.get(pre + names[k], { (int64_t) ff, (int64_t) W }, v)) return nullptr;
-        for (int64_t i = 0; i < ff; i++) memcpy(&all[(size_t) (2 * i + k) * W], &v[(size_t) i * W], (size_t) W * 4);
+        if (!src.get(pre + names[k], { (int64_t) ff, (int64_t) W }, v)) return false;
+        for (int64_t i = 0; i < ff; i++) memcpy(&all[at + (size_t) (2 * i + k) * W], &v[(size_t) i * W], (size_t) W * 4);
     }
+    return true;
+}
+static pib_weight * upload_gate_up(TensorSource & src, const std::string & pre, int ff, int W, int dtype, pib_model * m) {
+    std::vector<float> all;
+    if (!append_gate_up(src, pre, ff, W, all)) return nullptr;
     return upload_mat(all, 2 * (int64_t) ff, W, dtype, m);
 }
 
@@ -1056,10 +1064,173 @@ static pib_model * build_bobunex(const Json & cfg, TensorSource & src, int dtype
     return mp.release();
 }
 
+// ---- the Gusedra builder ----------------------------------------------------------------------------------------------------------
+// Sandwich layers (LayerNorms with weight and bias before and after every sublayer, layer scales, one residual multiplier); mixers "attention" (scores fall by a
+// slope per head and token of distance, a sliding window, a learned sink; a layer may read an earlier layer's cells: kv_from) and "attention_2" (a learned number
+// per distance bucket and head, a sliding window that keeps the first tokens, a sigmoid gate on every output value); feed-forwards: dense squared relu, or a
+// mixture of silu-gated experts with grouped choice, corrections and identity outputs beside a shared expert.  Sizes the configuration leaves out come from the
+// tensors' shapes.  Tensor names: '<layer>.norm1|norm1b|norm2|norm2b' (+ '.b'), '<layer>.ls1|ls2', '<layer>.mix.q|k|v|o|sink|rel|g',
+// '<layer>.mlp.up|down|router|correction|e<i>.*|shared.*', 'final.norm' (+ '.b'), 'embed', 'head'.
+static pib_model * build_gusedra(const Json & cfg, TensorSource & src, int dtype) {
+    std::unique_ptr<pib_model, void (*)(pib_model *)> mp(new pib_model(), pib_model_free);
+    pib_model * m = mp.get();
+    pib_hybrid * hy = new pib_hybrid();
+    m->hy = hy;
+    m->arch = 2; m->name = "Gusedra";
+    bool ok = true;
+    const int W = (int) jnum(&cfg, "width", 0, &ok), V = (int) jnum(&cfg, "vocab", 0, &ok);
+    const Json * layers = cfg.get("layers");
+    if (!ok || W <= 0 || V <= 0 || !layers || layers->kind != Json::ARR || layers->arr.empty()) { pib_set_error("model: config.json needs width, vocab and layers"); return nullptr; }
+    hy->dtype = dtype;
+    hy->form = PIB_FORM_SANDWICH;
+    hy->eps = (float) jnum(cfg.get("norm"), "eps", 1e-5);
+    hy->taps = 0;
+    const double mult = jnum(&cfg, "residual_mult", 1.0);
+    m->n_embd = W; m->n_vocab = V; m->n_layer = (int) layers->arr.size(); m->layer_begin = 0; m->layer_end = m->n_layer;
+    m->wtype = dtype; m->n_ctx_train = 1 << 20; m->n_head = 1; m->n_head_kv = 1; m->tok_bos = -1; m->tok_eos = -1;
+    std::vector<float> v;
+#define GET(name, ...) do { if (!src.get((name), { __VA_ARGS__ }, v)) return nullptr; } while (0)
+#define VEC(dst, name, n) do { GET(name, (int64_t) (n)); if (!((dst) = upload_f32v(v))) return nullptr; } while (0)
+#define MAT(dst, name, N, K) do { GET(name, (int64_t) (N), (int64_t) (K)); if (!((dst) = upload_mat(v, (N), (K), dtype, m))) return nullptr; } while (0)
+#define APPEND(all, name, N, K) do { GET(name, (int64_t) (N), (int64_t) (K)); (all).insert((all).end(), v.begin(), v.end()); } while (0)
+    MAT(m->tok_embd, "embed", V, W);
+    VEC(m->output_norm, "final.norm", W);
+    VEC(hy->final_b, "final.norm.b", W);
+    MAT(m->output, "head", V, W);
+    hy->layers.resize(m->n_layer);
+    auto widen = [](int & a, int64_t b) { if (b > a) a = (int) b; };
+    // the norm behind a sublayer with the layer scale and the residual multiplier in its weight and bias
+    auto post_norm = [&](const std::string & norm, const std::string & ls, float *& w, float *& b) -> bool {
+        std::vector<float> scale, u;
+        if (!src.get(ls, { (int64_t) W }, scale)) return false;
+        for (int k = 0; k < 2; k++) {
+            if (!src.get(k ? norm + ".b" : norm, { (int64_t) W }, u)) return false;
+            for (int i = 0; i < W; i++) u[(size_t) i] = (float) (mult * (double) scale[(size_t) i] * (double) u[(size_t) i]);
+            if (!((k ? b : w) = upload_f32v(u))) return false;
+        }
+        return true;
+    };
+    for (int il = 0; il < m->n_layer; il++) {
+        const Json & jl = layers->arr[il];
+        pib_hlayer & L = hy->layers[il];
+        const std::string p = "l" + std::to_string(il) + ".", px = p + "mix.", pm = p + "mlp.";
+        const Json * ty = jl.get("type"), * mx = jl.get("mixer"), * ml = jl.get("mlp");
+        if (!ty || ty->kind != Json::STR || !mx) { pib_set_error("model: layer %d needs type and mixer", il); return nullptr; }
+        const bool buckets = ty->str == "attention_2";
+        if (!buckets && ty->str != "attention") { pib_set_error("model: layer %d: unknown mixer '%s'", il, ty->str.c_str()); return nullptr; }
+        VEC(L.norm1, p + "norm1", W);
+        VEC(L.norm1_b, p + "norm1.b", W);
+        if (!post_norm(p + "norm1b", p + "ls1", L.post1, L.post1_b)) return nullptr;
+        // ---- attention ----
+        L.mixer = PIB_MIXER_KV;
+        const Json * kf = mx->get("kv_from"), * mk = mx->get("mask");
+        L.kv_from = kf && kf->kind == Json::NUM ? (int) kf->num : -1;
+        if (L.kv_from >= 0 && (L.kv_from >= il || hy->layers[L.kv_from].kv_from >= 0)) { pib_set_error("model: layer %d: kv_from %d is not an earlier layer with keys of its own", il, L.kv_from); return nullptr; }
+        const pib_hlayer * F = L.kv_from >= 0 ? &hy->layers[L.kv_from] : nullptr;
+        L.heads = (int) jnum(mx, "heads", (double) (buckets ? src.dim(px + "rel", 1, 0) : src.dim(px + "sink", 0, 0)));
+        L.dim = (int) jnum(mx, "dim", L.heads > 0 ? (double) (src.dim(px + "q", 0, 0) / L.heads) : 0.0);
+        L.vdim = (int) jnum(mx, "vdim", L.heads > 0 ? (double) (src.dim(px + "o", 1, 0) / L.heads) : 0.0);
+        L.kv_heads = (int) jnum(mx, "kv_heads", F ? (double) F->kv_heads : L.dim > 0 ? (double) (src.dim(px + "k", 0, (int64_t) L.heads * L.dim) / L.dim) : 0.0);
+        if (L.heads <= 0 || L.dim <= 0 || L.vdim <= 0 || L.kv_heads <= 0 || L.heads % L.kv_heads) { pib_set_error("model: layer %d: heads / kv_heads / dim / vdim", il); return nullptr; }
+        if (F && (F->kv_heads != L.kv_heads || F->dim != L.dim || F->vdim != L.vdim)) { pib_set_error("model: layer %d: its keys or values have another shape than those of layer %d", il, L.kv_from); return nullptr; }
+        L.scale = (float) jnum(mx, "scale", 1.0 / sqrt((double) L.dim));
+        L.window = mk && !mk->is_null() ? (int) jnum(mk, "size", 0) : 0;
+        if (L.window <= 0) L.window = 1 << 30;                              // no mask: every earlier token is seen
+        L.keep = mk && !mk->is_null() ? std::max(0, (int) jnum(mk, "keep_first", 0)) : 0;
+        if (L.window == 1 << 30) L.keep = 0;
+        L.out_gate = buckets ? 1 : 0;
+        const int64_t H = L.heads, G = L.kv_heads, D = L.dim, Vd = L.vdim, n_own = H * D + (buckets ? H * Vd : 0);
+        std::vector<float> all;
+        APPEND(all, px + "q", H * D, W);
+        if (buckets) APPEND(all, px + "g", H * Vd, W);
+        if (!F) { APPEND(all, px + "k", G * D, W); APPEND(all, px + "v", G * Vd, W); }
+        if (!(L.qkv = upload_mat(all, (int64_t) all.size() / W, W, dtype, m))) return nullptr;
+        MAT(L.wo, px + "o", W, H * Vd);
+        if (buckets) {
+            // one row per head over distances: the bucket of a distance n is n below half the buckets, then a half that widens geometrically up to bias_max.  The last
+            // row of the table repeats for all distances from the first one in the last bucket on
+            const int64_t Bk = src.dim(px + "rel", 0, 32);
+            const double  half = (double) (Bk / 2), most = jnum(mx, "bias_max", 128.0);
+            GET(px + "rel", Bk, H);
+            std::vector<int64_t> of;
+            for (int64_t n = 0; ; n++) {
+                int64_t b = n;
+                if (n >= Bk / 2) {
+                    double e = most > half && half > 0 ? log((double) n / half) / log(most / half) * (double) (Bk - Bk / 2) : (double) Bk;
+                    if (fabs(e - round(e)) < 1e-9) e = round(e);                // a border that is met exactly
+                    b = e >= (double) (Bk - 1 - Bk / 2) ? Bk - 1 : Bk / 2 + (int64_t) floor(e);
+                }
+                of.push_back(b);
+                if (b == Bk - 1) break;
+                if (n > (1 << 24)) { pib_set_error("model: layer %d: bias_max %g", il, most); return nullptr; }
+            }
+            L.n_rel = (int) of.size();
+            std::vector<float> tab((size_t) H * of.size());
+            for (int64_t h = 0; h < H; h++) for (size_t n = 0; n < of.size(); n++) tab[(size_t) h * of.size() + n] = v[(size_t) (of[n] * H + h)];
+            if (!(L.rel = upload_f32v(tab))) return nullptr;
+        } else {
+            std::vector<float> sl((size_t) H);
+            for (int64_t h = 0; h < H; h++) sl[(size_t) h] = (float) exp2(-8.0 * (double) (h + 1) / (double) H);
+            if (!(L.slopes = upload_f32v(sl))) return nullptr;
+            VEC(L.sink, px + "sink", H);
+        }
+        if (F) L.cache_id = F->cache_id;
+        else { L.cache_id = hy->n_cache++; hy->cache_row.push_back((int) (G * (D + Vd))); }
+        widen(hy->w_proj, (n_own + 3) & ~(int64_t) 3); widen(hy->w_att, H * Vd);
+        // ---- the feed-forward ----
+        if (!ml || ml->is_null()) continue;
+        VEC(L.norm2, p + "norm2", W);
+        VEC(L.norm2_b, p + "norm2.b", W);
+        if (!post_norm(p + "norm2b", p + "ls2", L.post2, L.post2_b)) return nullptr;
+        const Json * kind = ml->get("kind");
+        if (kind && kind->str == "dense") {
+            L.mlp = PIB_MLP_RELU2; L.ff = (int) jnum(ml, "ff", (double) src.dim(pm + "up", 0, 0));
+            if (L.ff <= 0) { pib_set_error("model: layer %d: mlp.ff", il); return nullptr; }
+            MAT(L.up, pm + "up", L.ff, W);
+            MAT(L.down, pm + "down", W, L.ff);
+            widen(hy->w_proj, (int64_t) L.ff);
+        } else if (kind && kind->str == "moe") {
+            L.mlp = PIB_MLP_MOE; L.route = PIB_ROUTE_SOFTMAX_GROUPS; L.expert = PIB_EXPERT_SWIGLU;
+            const Json * ro = ml->get("router"), * gr = ro ? ro->get("groups") : nullptr, * sh = ml->get("shared");
+            L.n_experts = (int) jnum(ro, "experts", 0); L.identity = (int) jnum(ro, "identity", 0); L.top = (int) jnum(ro, "top", 0); L.route_scale = (float) jnum(ro, "scale", 1.0);
+            L.groups = gr && !gr->is_null() ? (int) jnum(gr, "count", 1) : 1; L.keep_groups = gr && !gr->is_null() ? (int) jnum(gr, "keep", L.groups) : 1;
+            L.ff_e = (int) jnum(ml->get("expert"), "ff", (double) src.dim(pm + "e0.up", 0, 0));
+            L.ff_s = sh && !sh->is_null() ? (int) jnum(sh, "ff", (double) src.dim(pm + "shared.up", 0, 0)) : 0;
+            const int E = L.n_experts + L.identity;
+            if (L.n_experts <= 0 || L.identity < 0 || L.top <= 0 || L.top > E || L.ff_e <= 0) { pib_set_error("model: layer %d: router.experts / router.identity / router.top / expert.ff", il); return nullptr; }
+            if (L.groups < 1 || E % L.groups || L.keep_groups < 1 || L.keep_groups > L.groups || L.top > L.keep_groups * (E / L.groups)) {
+                pib_set_error("model: layer %d: %d router outputs in %d groups of which %d are kept, top %d", il, E, L.groups, L.keep_groups, L.top); return nullptr;
+            }
+            std::vector<float> ups, downs;
+            for (int e = 0; e < L.n_experts; e++) {
+                const std::string pe = pm + "e" + std::to_string(e) + ".";
+                if (!append_gate_up(src, pe, L.ff_e, W, ups)) return nullptr;
+                APPEND(downs, pe + "down", W, L.ff_e);
+            }
+            if (!(L.e_up = upload_mat(ups, (int64_t) L.n_experts * 2 * L.ff_e, W, dtype, m)) || !(L.e_down = upload_mat(downs, (int64_t) L.n_experts * W, L.ff_e, dtype, m))) return nullptr;
+            GET(pm + "router", (int64_t) E, (int64_t) W);
+            if (!(L.router = upload_mat(v, E, W, PIB_TYPE_F32, m))) return nullptr;                     // the router is always 32-bit
+            if (src.has(pm + "correction")) VEC(L.correction, pm + "correction", E);
+            if (L.ff_s > 0) {
+                if (!(L.s_up = upload_gate_up(src, pm + "shared.", L.ff_s, W, dtype, m))) return nullptr;
+                MAT(L.s_down, pm + "shared.down", W, L.ff_s);
+                widen(hy->w_proj, (L.ff_s + 3) & ~3);
+            }
+            widen(hy->w_pairs, L.top); widen(hy->w_eup, (int64_t) L.top * L.ff_e); widen(hy->w_router, E);
+        } else { pib_set_error("model: layer %d: unknown mlp kind", il); return nullptr; }
+    }
+    hy->state_floats = 4;
+#undef GET
+#undef VEC
+#undef MAT
+#undef APPEND
+    return mp.release();
+}
+
 // ---- registry: config.json "architecture" -> builder ---------------------------------------------------------------------------------
 struct DirArch { const char * name; pib_model * (*build)(const Json &, TensorSource &, int); };
 static const DirArch DIR_ARCHS[] = { { "Rapisun", build_rapisun }, { "Fabivik", build_fabivik }, { "Lulenex", build_lulenex }, { "Putazen", build_putazen },
-                                     { "Bobunex", build_bobunex } };
+                                     { "Bobunex", build_bobunex }, { "Gusedra", build_gusedra } };
 
 static pib_model * build_from_config(const Json & cfg, TensorSource & src, int dtype) {
     const Json * a = cfg.get("architecture");
@@ -1096,7 +1267,8 @@ void pib_hybrid_model_free(pib_model * m) {
     for (pib_hlayer & L : hy->layers) {
         if (L.weights_of >= 0) continue;                  // a later walk of the same layer: the tensors are the first walk's
         for (float * f : { L.norm1, L.norm2, L.canon, L.dq_norm, L.dkv_norm, L.sink, L.f_bias, L.lower, L.onorm, L.conv, L.q_norm, L.k_norm, L.mu, L.w0, L.bonus, L.a_log,
-                           L.dt_bias, L.shift, L.conv_b, L.ssm_a, L.ssm_d, L.proj_bias, L.o_bias, L.decay, L.hc1, L.hc2, L.norm1_b, L.norm2_b, L.rg1_b, L.rg2_b, L.canon2, L.i_bias, L.out_a, L.out_b }) if (f) cudaFree(f);
+                           L.dt_bias, L.shift, L.conv_b, L.ssm_a, L.ssm_d, L.proj_bias, L.o_bias, L.decay, L.hc1, L.hc2, L.norm1_b, L.norm2_b, L.rg1_b, L.rg2_b, L.canon2, L.i_bias, L.out_a, L.out_b, L.slopes, L.rel, L.post1,
+                           L.post1_b, L.post2, L.post2_b, L.correction }) if (f) cudaFree(f);
         for (pib_weight * w : { L.dqkv, L.uq, L.ukT, L.uv, L.wo, L.qfv, L.up, L.down, L.e_up, L.e_down, L.router, L.s_up, L.s_down, L.qkv, L.rkvg, L.w1, L.w2, L.ssm_in, L.ssm_x,
                                 L.ssm_dt, L.rg1, L.rg2, L.wo2 }) if (w) pib_weight_free(w);
     }
