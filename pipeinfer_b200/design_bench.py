@@ -1,10 +1,11 @@
-"""`bench.py --design rapisun | fabivik | lulenex | putazen | bobunex`: prefill and decode throughput of a layer-list design at sizes that resemble a real
+"""`bench.py --design rapisun | fabivik | lulenex | putazen | bobunex | gusedra`: prefill and decode throughput of a layer-list design at sizes that resemble a real
 model's layers (random weights drawn in the loader from a seed), beside the closest existing model of the library at equal width / depth /
 vocabulary -- for Rapisun the llama architecture in Q4_K (prompts on its tcgen05 GEMM, decoding on its tensor-core GEMVs), for Fabivik
 the Rapisun design (the other layer-list model: same runtime, same dense matmuls), for Lulenex the Fabivik design (attention over cached
 key / value heads and recurrences on the same kernels), for Putazen the Lulenex design (a state-space scan beside attention over cached
 key / value heads, a dense feed-forward in every layer, a layer walked twice), for Bobunex the Lulenex design too (softmax attention beside a
-linear recurrence in one mixer) -- plus the share and the roofline fraction of every kind of launch.  Everything goes through llama_decode on host batches; times are medians of CUDA-side
+linear recurrence in one mixer), for Gusedra the Fabivik design (windowed attention over cached key / value heads, mixtures of gated experts with a shared
+expert) -- plus the share and the roofline fraction of every kind of launch.  Everything goes through llama_decode on host batches; times are medians of CUDA-side
 work as seen by the caller (llama_decode returns after the run's event), the per-kind numbers come from CUDA events around each
 launch (llama_pib_profile_layer).  One JSON line on stdout."""
 import ctypes as C
@@ -90,11 +91,25 @@ def bobunex_config(width, vocab, blocks, heads, window, ff, **_):
             "layers": [{"type": "parallel", "mixer": two, "mlp": {"kind": "dense", "ff": ff}}] * (4 * blocks)}
 
 
+def gusedra_config(width, vocab, blocks, heads, window, ff, experts, top, ff_e, ff_s, **_):
+    """one block = [slopes + sink, dense; buckets + kept tokens, MoE; slopes over the first one's cells, MoE; buckets, MoE]; a fifth of the router's outputs pass their
+    input on, half of its two groups take part"""
+    dim, ident = 128, experts // 4
+    moe = {"kind": "moe", "router": {"experts": experts, "top": top, "scale": 1.5, "identity": ident, "groups": {"count": 2, "keep": 1}}, "expert": {"ff": ff_e}, "shared": {"ff": ff_s}}
+    att = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": dim, "vdim": dim, "mask": {"size": window}, "scale": 1.0 / math.sqrt(dim)}
+    rel = dict(att, mask={"size": window, "keep_first": 4}, bias_max=window)
+    layers = []
+    for b in range(blocks):
+        layers += [{"type": "attention", "mixer": att, "mlp": {"kind": "dense", "ff": ff}}, {"type": "attention_2", "mixer": rel, "mlp": moe},
+                   {"type": "attention", "mixer": dict(att, kv_from=4 * b), "mlp": moe}, {"type": "attention_2", "mixer": rel, "mlp": moe}]
+    return {"architecture": "Gusedra", "width": width, "vocab": vocab, "norm": {"eps": 1e-5}, "residual_mult": 0.5, "layers": layers}
+
+
 # design -> (its name, its configuration, the comparator's key)
 DESIGNS = {"rapisun": ("Rapisun", design_config, "llama_q4k"), "fabivik": ("Fabivik", fabivik_config, "rapisun"), "lulenex": ("Lulenex", lulenex_config, "fabivik"),
-           "putazen": ("Putazen", putazen_config, "lulenex"), "bobunex": ("Bobunex", bobunex_config, "lulenex")}
+           "putazen": ("Putazen", putazen_config, "lulenex"), "bobunex": ("Bobunex", bobunex_config, "lulenex"), "gusedra": ("Gusedra", gusedra_config, "fabivik")}
 COMPARATORS = {"llama_q4k": "llama architecture, Q4_K", "rapisun": "Rapisun (layer-list design of this library), same width / depth / vocabulary / experts",
-               "fabivik": "Fabivik (layer-list design of this library), same width / layer runs / vocabulary",
+               "fabivik": "Fabivik (layer-list design of this library), same width / layer runs / vocabulary (and experts where the design has them)",
                "lulenex": "Lulenex (layer-list design of this library), same width / layer runs / vocabulary / feed-forward width"}
 
 SIZES = {

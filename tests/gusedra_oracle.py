@@ -7,6 +7,7 @@ token-by-token decoding.
 Notation: x the residual stream [T, width], N a LayerNorm with weight and bias.  A sublayer f adds  m * ls * N'(f(N(x)))  to x, with one
 number m for the model and one vector ls per sublayer.
 """
+import functools
 import math
 
 import numpy as np
@@ -50,6 +51,7 @@ def slope(h, H):
     return 2.0 ** (-8.0 * (h + 1) / H)
 
 
+@functools.lru_cache(maxsize=None)
 def bucket(n, B, D):
     """distances below B/2 one by one, then B/2 buckets whose widths grow geometrically up to distance D, the last one open"""
     half = B // 2

@@ -87,6 +87,43 @@ def test_paired_gelu_epilogue(M, F, K):
     np.testing.assert_allclose(got32, ref_of(X.astype(np.float32).astype(np.float64)), rtol=1e-4, atol=1e-5 * np.sqrt(K))
 
 
+@pytest.mark.parametrize("M,F,K", [(1, 40, 64), (3, 33, 72), (16, 200, 128), (17, 70, 64), (130, 150, 96), (300, 64, 200), (5, 7, 11)])
+def test_paired_silu_epilogue(M, F, K):
+    """rows (gate i, up i) interleaved; output i is gate / (1 + exp(-gate)) * up"""
+    rng = np.random.default_rng(M + F)
+    Wg, Wu = bf16_round(rng.standard_normal((F, K))), bf16_round(rng.standard_normal((F, K)))
+    W = np.stack([Wg, Wu], 1).reshape(2 * F, K)
+    X = rng.standard_normal((M, K)) * 0.2
+
+    def ref_of(x):
+        z = x @ Wg.T
+        return z / (1.0 + np.exp(-z)) * (x @ Wu.T)
+    got = mm(W, X, M, 2 * F, K, ldy=F, epi=5).reshape(M, F)
+    np.testing.assert_allclose(got, ref_of(bf16_round(X)), rtol=1e-3, atol=1e-3 * np.sqrt(K))
+    got32 = mm(W, X, M, 2 * F, K, ldy=F, epi=5, exact=True, f32=True).reshape(M, F)
+    np.testing.assert_allclose(got32, ref_of(X.astype(np.float32).astype(np.float64)), rtol=1e-4, atol=1e-5 * np.sqrt(K))
+
+
+@pytest.mark.parametrize("T,E,top,K,F", [(4, 6, 3, 88, 40), (2, 5, 2, 64, 24), (70, 5, 2, 64, 24), (400, 12, 2, 200, 44), (300, 3, 3, 128, 65), (90, 4, 2, 50, 9)])
+def test_grouped_paired_silu_epilogue(T, E, top, K, F):
+    """experts' gate and up rows interleaved, pairs sorted by expert; the last expert's pairs lie behind the range of every problem and are left alone"""
+    rng = np.random.default_rng(T + E)
+    Wg, Wu = bf16_round(rng.standard_normal((E - 1, F, K))), bf16_round(rng.standard_normal((E - 1, F, K)))
+    W = np.stack([Wg, Wu], 2).reshape(E - 1, 2 * F, K)
+    X = rng.standard_normal((T, K)) * 0.2
+    ids = np.stack([rng.permutation(E)[:top] for _ in range(T)]).reshape(-1)
+    perm = np.argsort(ids, kind="stable").astype(np.int32)
+    offs = np.concatenate([[0], np.cumsum(np.bincount(ids, minlength=E))]).astype(np.int32)
+    got = mm(W, X, T * top, 2 * F, K, Z=E - 1, ldw=K, wz=2 * F * K, xrows=perm, xdiv=top, ldy=F, zrange=offs[:E], epi=5, y_elems=T * top * F).reshape(T * top, F)
+    for i, p in enumerate(perm):
+        if ids[p] == E - 1:
+            assert np.isnan(got[i]).all()
+            continue
+        x = bf16_round(X[p // top])
+        z = x @ Wg[ids[p]].T
+        np.testing.assert_allclose(got[i], z / (1.0 + np.exp(-z)) * (x @ Wu[ids[p]].T), rtol=1e-3, atol=1e-3 * np.sqrt(K))
+
+
 @pytest.mark.parametrize("T,H,D,R", [(5, 3, 24, 56), (40, 6, 72, 104), (200, 4, 128, 256), (130, 2, 16, 40)])
 def test_one_problem_per_head(T, H, D, R):
     """Y[t][h][r] = sum_d X[t][h][d] * W[h][r][d], X rows carry other columns between the heads' parts (the rotated query part)"""
