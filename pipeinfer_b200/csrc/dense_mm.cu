@@ -9,8 +9,8 @@
 // through an index list.
 //
 // Kernels: mm_tile_kernel (any shape; 64 x 64 x 16 tiles, 4 x 4 outputs per thread), for up to MV_MAXB rows mv_rows_kernel
-// (one warp per weight row, 16-byte weight loads: the weights are read once at the speed of memory), and for up to 32 float32 outputs
-// over many rows mm_few_cols_kernel (a warp per row: a router's logits, where 64-wide output tiles would leave most of the machine idle).
+// (one warp per weight row, 16-byte weight loads: the weights are read once at the speed of memory), and for up to 128 float32 outputs
+// over many rows mm_few_cols_kernel (a warp per four rows: a router's logits, where 64-wide output tiles would leave most of the machine idle).
 #include "hybrid.cuh"
 
 #include <cuda_bf16.h>
@@ -31,6 +31,7 @@ struct mm_dev {
     int M, N, K;
     const int32_t * zrange;
     float e0, e1;
+    const int32_t * zlist;
     float * Y2; int64_t ld2; int n2; const int32_t * rows2;      // outputs n >= n2: Y2[rows2[m] * ld2 + n - n2]
 };
 __device__ __forceinline__ float * mm_out(const mm_dev & a, float * Y, int m, int n) { return n >= a.n2 ? a.Y2 + (size_t) a.rows2[m] * a.ld2 + (n - a.n2) : Y + (size_t) m * a.ldy + n; }
@@ -193,24 +194,48 @@ __device__ __forceinline__ void mv_rows_body(const mm_dev & a, bool xvec, int z,
 // step has one or two of the batch's pairs -- and takes the instance that fits its own count, so that it stays bound by its weights' bytes
 // and not by B times the arithmetic.  Every row's sum is formed in the same order whichever instance runs.
 template <typename WT, bool ROUND, int EPI, int B>
+__device__ __forceinline__ void mv_rows_fit(const mm_dev & a, bool xvec, int z, int n, int lane, int row0, int row1) {
+    const int cnt = row1 - row0;
+    if (B > 1 && cnt == 1)               mv_rows_body<WT, ROUND, EPI, 1>(a, xvec, z, n, lane, row0, row1);
+    else if (B > 2 && cnt <= 2)          mv_rows_body<WT, ROUND, EPI, 2>(a, xvec, z, n, lane, row0, row1);
+    else if (B > 4 && cnt <= 4)          mv_rows_body<WT, ROUND, EPI, (B > 4 ? 4 : B)>(a, xvec, z, n, lane, row0, row1);
+    else if (B > 8 && cnt <= 8)          mv_rows_body<WT, ROUND, EPI, (B > 8 ? 8 : B)>(a, xvec, z, n, lane, row0, row1);
+    else                                 mv_rows_body<WT, ROUND, EPI, B>(a, xvec, z, n, lane, row0, row1);
+}
+// the problem of grid place iz: the iz-th one that has rows (zlist), or iz itself; false when there is nothing to do
+__device__ __forceinline__ bool mv_problem(const mm_dev & a, int iz, int B, int & z, int & row0, int & row1) {
+    z = iz; row0 = 0; row1 = a.M;
+    if (a.zlist) { if (iz >= a.zlist[0]) return false; z = a.zlist[1 + iz]; }
+    if (a.zrange) { row0 = a.zrange[z]; row1 = a.zrange[z + 1]; }
+    if (row1 - row0 > B) row1 = row0 + B;            // the host only picks these kernels when every z has at most B rows
+    return row0 < row1;
+}
+template <typename WT, bool ROUND, int EPI, int B>
 __global__ void __launch_bounds__(256) mv_rows_kernel(mm_dev a, bool xvec) {
     pib_pdl_wait();
     pib_pdl_trigger();
-    const int z = blockIdx.z;
-    int row0 = 0, row1 = a.M;
-    if (a.zrange) { row0 = a.zrange[z]; row1 = a.zrange[z + 1]; }
-    if (row1 - row0 > B) row1 = row0 + B;            // the host only picks this kernel when every z has at most B rows
-    if (row0 >= row1) return;
+    int z, row0, row1;
+    if (!mv_problem(a, blockIdx.z, B, z, row0, row1)) return;
     const int lane = threadIdx.x & 31, n = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     if (n >= (pib_epi_pairs(EPI) ? a.N / 2 : a.N)) return;
-    const int cnt = row1 - row0;
-    if (B > 1 && a.zrange && cnt < B) {
-        if (cnt == 1)                { mv_rows_body<WT, ROUND, EPI, 1>(a, xvec, z, n, lane, row0, row1); return; }
-        if (B > 2 && cnt <= 2)       { mv_rows_body<WT, ROUND, EPI, 2>(a, xvec, z, n, lane, row0, row1); return; }
-        if (B > 4 && cnt <= 4)       { mv_rows_body<WT, ROUND, EPI, (B > 4 ? 4 : B)>(a, xvec, z, n, lane, row0, row1); return; }
-        if (B > 8 && cnt <= 8)       { mv_rows_body<WT, ROUND, EPI, (B > 8 ? 8 : B)>(a, xvec, z, n, lane, row0, row1); return; }
+    if (a.zrange) mv_rows_fit<WT, ROUND, EPI, B>(a, xvec, z, n, lane, row0, row1);
+    else          mv_rows_body<WT, ROUND, EPI, B>(a, xvec, z, n, lane, row0, row1);
+}
+// a grouped problem and a plain one in one launch: blocks [0, za * blocks_a) walk the weight rows of a's problems with rows, the others b's
+template <typename WT, bool ROUND, int EPI, int B>
+__global__ void __launch_bounds__(256) mv_experts_kernel(mm_dev a, mm_dev b, bool xva, bool xvb, int blocks_a, int za) {
+    pib_pdl_wait();
+    pib_pdl_trigger();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, per = blockDim.x >> 5, blk = blockIdx.x - blocks_a * za;
+    int z, row0, row1;
+    if (blk < 0) {
+        const int n = ((int) blockIdx.x % blocks_a) * per + warp;
+        if (!mv_problem(a, blockIdx.x / blocks_a, B, z, row0, row1) || n >= (pib_epi_pairs(EPI) ? a.N / 2 : a.N)) return;
+        mv_rows_fit<WT, ROUND, EPI, B>(a, xva, z, n, lane, row0, row1);
+    } else {
+        const int n = blk * per + warp;
+        if (n < (pib_epi_pairs(EPI) ? b.N / 2 : b.N)) mv_rows_fit<WT, ROUND, EPI, B>(b, xvb, 0, n, lane, 0, b.M);
     }
-    mv_rows_body<WT, ROUND, EPI, B>(a, xvec, z, n, lane, row0, row1);
 }
 
 // two independent few-row matmuls in one launch (decode steps: a launch costs as much as a small matrix): blocks [0, blocks_a) walk a's weight rows,
@@ -229,29 +254,62 @@ __global__ void __launch_bounds__(256) mv_pair_kernel(mm_dev a, mm_dev b, bool x
     }
 }
 
-// ---- few outputs, many rows (a router's logits over a prompt): one warp per row m, lanes stride over k, NB accumulators per lane ----
-// float32 weights and activations, no rounding; the weight matrix (N x K floats) stays in L1 / L2 while every warp walks it.
-template <int NB>
-__global__ void __launch_bounds__(256) mm_few_cols_kernel(mm_dev a) {
+// ---- few outputs, many rows (a router's logits over a prompt): a warp takes FC_ROWS rows of X and NB outputs, lanes stride over k in 16-byte pieces ----
+// float32 weights and activations, no rounding.  A weight piece is used for FC_ROWS rows, so the matrix crosses L1 once per that many rows; grid.y walks the
+// outputs in runs of NB.
+#define FC_ROWS 4
+template <int NB, bool VEC>
+__global__ void __launch_bounds__(128) mm_few_cols_kernel(mm_dev a) {
     pib_pdl_wait();
     pib_pdl_trigger();
-    const int lane = threadIdx.x & 31, m = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-    if (m >= a.M) return;
-    const float * W = reinterpret_cast<const float *>(a.W);
-    const float * x = a.X + (size_t) m * a.ldx;
-    float acc[NB];
+    const int lane = threadIdx.x & 31, m0 = (blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5)) * FC_ROWS, n0 = blockIdx.y * NB;
+    if (m0 >= a.M) return;
+    const float * W = reinterpret_cast<const float *>(a.W) + (size_t) n0 * a.ldw;
+    const int nn = min(NB, a.N - n0);
+    const float * x[FC_ROWS];
 #pragma unroll
-    for (int n = 0; n < NB; n++) acc[n] = 0.f;
-    for (int k = lane; k < a.K; k += 32) {
-        const float xv = x[k];
+    for (int r = 0; r < FC_ROWS; r++) x[r] = a.X + (size_t) min(m0 + r, a.M - 1) * a.ldx;
+    float acc[FC_ROWS][NB];
 #pragma unroll
-        for (int n = 0; n < NB; n++) if (n < a.N) acc[n] = fmaf(xv, W[(size_t) n * a.ldw + k], acc[n]);
+    for (int r = 0; r < FC_ROWS; r++)
+#pragma unroll
+        for (int n = 0; n < NB; n++) acc[r][n] = 0.f;
+    if (VEC) {
+        for (int k = lane * 4; k < a.K; k += 128) {
+            float4 xv[FC_ROWS];
+#pragma unroll
+            for (int r = 0; r < FC_ROWS; r++) xv[r] = *reinterpret_cast<const float4 *>(x[r] + k);
+#pragma unroll
+            for (int n = 0; n < NB; n++) {
+                if (n < nn) {
+                    const float4 w = *reinterpret_cast<const float4 *>(W + (size_t) n * a.ldw + k);
+#pragma unroll
+                    for (int r = 0; r < FC_ROWS; r++) acc[r][n] = fmaf(xv[r].w, w.w, fmaf(xv[r].z, w.z, fmaf(xv[r].y, w.y, fmaf(xv[r].x, w.x, acc[r][n]))));
+                }
+            }
+        }
+    } else {
+        for (int k = lane; k < a.K; k += 32) {
+            float xv[FC_ROWS];
+#pragma unroll
+            for (int r = 0; r < FC_ROWS; r++) xv[r] = x[r][k];
+#pragma unroll
+            for (int n = 0; n < NB; n++) {
+                if (n < nn) {
+                    const float w = W[(size_t) n * a.ldw + k];
+#pragma unroll
+                    for (int r = 0; r < FC_ROWS; r++) acc[r][n] = fmaf(xv[r], w, acc[r][n]);
+                }
+            }
+        }
     }
 #pragma unroll
-    for (int n = 0; n < NB; n++) {
-        const float v = warp_sum(acc[n]);
-        if (lane == 0 && n < a.N) a.Y[(size_t) m * a.ldy + n] = v;
-    }
+    for (int r = 0; r < FC_ROWS; r++)
+#pragma unroll
+        for (int n = 0; n < NB; n++) {
+            const float v = warp_sum(acc[r][n]);
+            if (lane == 0 && n < nn && m0 + r < a.M) a.Y[(size_t) (m0 + r) * a.ldy + n0 + n] = v;
+        }
 }
 
 template <typename WT, bool ROUND, int EPI>
@@ -261,7 +319,7 @@ static int launch_mm(const pib_mm & a, const mm_dev & d, cudaStream_t st) {
     const bool vec_ok = a.ldw % V == 0 && a.wz % V == 0 && ((uintptr_t) a.W & 15) == 0;
     // few rows in all (with zrange: no problem z can own more than the total): a warp per weight row; problems without rows leave at once
     if (a.M <= MV_MAXB && vec_ok) {
-        dim3 grid((unsigned) (((pib_epi_pairs(EPI) ? a.N / 2 : a.N) + 7) / 8), 1, (unsigned) a.Z);
+        dim3 grid((unsigned) (((pib_epi_pairs(EPI) ? a.N / 2 : a.N) + 7) / 8), 1, (unsigned) (a.zlist && a.M < a.Z ? a.M : a.Z));
         const bool xvec = a.ldx % 4 == 0 && a.xz % 4 == 0 && ((uintptr_t) a.X & 15) == 0;
         if (a.M == 1)      pib_launch(mv_rows_kernel<WT, ROUND, EPI, 1>, dim3(grid), dim3(256), (size_t) (0), st, d, xvec);
         else if (a.M == 2) pib_launch(mv_rows_kernel<WT, ROUND, EPI, 2>, dim3(grid), dim3(256), (size_t) (0), st, d, xvec);
@@ -287,12 +345,14 @@ int pib_dense_mm(const pib_mm & a, cudaStream_t st) {
         if (rc != PIB_ERR_UNSUPP) return rc;
     }
     if (a.x_bf16) { pib_set_error("dense matmul: bfloat16 activations need the tensor-core path (more than 16 rows, strides multiples of 8)"); return PIB_ERR_UNSUPP; }
-    mm_dev d = { a.W, a.ldw, a.wz, a.X, a.ldx, a.xz, a.xrows, a.xdiv < 1 ? 1 : a.xdiv, a.Y, a.ldy, a.yz, a.M, a.N, a.K, a.zrange, a.e0, a.e1, a.Y2, a.ld2, a.Y2 ? a.n2 : 0x7fffffff, a.rows2 };
-    if (a.wtype == PIB_TYPE_F32 && a.exact && !a.Y2 && a.N <= 32 && a.M > MV_MAXB && a.Z == 1 && !a.xrows && !a.zrange && a.epi == PIB_EPI_NONE) {
-        dim3 grid((unsigned) ((a.M + 7) / 8));
-        if (a.N <= 8)       pib_launch(mm_few_cols_kernel<8>, dim3(grid), dim3(256), (size_t) 0, st, d);
-        else if (a.N <= 16) pib_launch(mm_few_cols_kernel<16>, dim3(grid), dim3(256), (size_t) 0, st, d);
-        else                pib_launch(mm_few_cols_kernel<32>, dim3(grid), dim3(256), (size_t) 0, st, d);
+    mm_dev d = { a.W, a.ldw, a.wz, a.X, a.ldx, a.xz, a.xrows, a.xdiv < 1 ? 1 : a.xdiv, a.Y, a.ldy, a.yz, a.M, a.N, a.K, a.zrange, a.e0, a.e1, a.zlist, a.Y2, a.ld2, a.Y2 ? a.n2 : 0x7fffffff, a.rows2 };
+    if (a.wtype == PIB_TYPE_F32 && a.exact && !a.Y2 && a.N <= 128 && a.M > MV_MAXB && a.Z == 1 && !a.xrows && !a.zrange && a.epi == PIB_EPI_NONE) {
+        const int  NB = a.N <= 8 ? 8 : a.N <= 16 ? 16 : 24;
+        const bool vec = a.K % 4 == 0 && a.ldw % 4 == 0 && a.ldx % 4 == 0 && (((uintptr_t) a.W | (uintptr_t) a.X) & 15) == 0;
+        dim3 grid((unsigned) ((a.M + 4 * FC_ROWS - 1) / (4 * FC_ROWS)), (unsigned) ((a.N + NB - 1) / NB));
+#define FC_GO(NB) do { if (vec) pib_launch(mm_few_cols_kernel<NB, true>, grid, dim3(128), (size_t) 0, st, d); else pib_launch(mm_few_cols_kernel<NB, false>, grid, dim3(128), (size_t) 0, st, d); } while (0)
+        if (NB == 8) FC_GO(8); else if (NB == 16) FC_GO(16); else FC_GO(24);
+#undef FC_GO
         PIB_CHECK(cudaGetLastError());
         return PIB_OK;
     }
@@ -328,7 +388,7 @@ int pib_dense_mm_pair(const pib_mm & a, const pib_mm & b, cudaStream_t st) {
         const int rc = pib_dense_mm(a, st);
         return rc != PIB_OK ? rc : pib_dense_mm(b, st);
     }
-    auto dev = [](const pib_mm & m) { return mm_dev{ m.W, m.ldw, m.wz, m.X, m.ldx, m.xz, nullptr, 1, m.Y, m.ldy, m.yz, m.M, m.N, m.K, nullptr, m.e0, m.e1, nullptr, 0, 0x7fffffff, nullptr }; };
+    auto dev = [](const pib_mm & m) { return mm_dev{ m.W, m.ldw, m.wz, m.X, m.ldx, m.xz, nullptr, 1, m.Y, m.ldy, m.yz, m.M, m.N, m.K, nullptr, m.e0, m.e1, nullptr, nullptr, 0, 0x7fffffff, nullptr }; };
     auto xvec = [](const pib_mm & m) { return m.ldx % 4 == 0 && ((uintptr_t) m.X & 15) == 0; };
 #define PAIR_GO(WT, ROUND) do { if (b.epi == PIB_EPI_NONE) launch_pair<WT, ROUND, PIB_EPI_NONE>(dev(a), dev(b), xvec(a), xvec(b), st); \
                                 else launch_pair<WT, ROUND, PIB_EPI_GEGLU_PAIR>(dev(a), dev(b), xvec(a), xvec(b), st); } while (0)
@@ -336,6 +396,39 @@ int pib_dense_mm_pair(const pib_mm & a, const pib_mm & b, cudaStream_t st) {
     else if (a.exact) PAIR_GO(float, false);
     else PAIR_GO(float, true);
 #undef PAIR_GO
+    PIB_CHECK(cudaGetLastError());
+    return PIB_OK;
+}
+
+template <typename WT, bool ROUND, int EPI>
+static void launch_experts(const mm_dev & a, const mm_dev & b, bool xva, bool xvb, int za, cudaStream_t st) {
+    const int ba = ((pib_epi_pairs(EPI) ? a.N / 2 : a.N) + 7) / 8, bb = ((pib_epi_pairs(EPI) ? b.N / 2 : b.N) + 7) / 8, rows = a.M > b.M ? a.M : b.M;
+    const dim3 grid((unsigned) (ba * za + bb));
+    if (rows == 1)      pib_launch(mv_experts_kernel<WT, ROUND, EPI, 1>, grid, dim3(256), (size_t) 0, st, a, b, xva, xvb, ba, za);
+    else if (rows == 2) pib_launch(mv_experts_kernel<WT, ROUND, EPI, 2>, grid, dim3(256), (size_t) 0, st, a, b, xva, xvb, ba, za);
+    else if (rows <= 4) pib_launch(mv_experts_kernel<WT, ROUND, EPI, 4>, grid, dim3(256), (size_t) 0, st, a, b, xva, xvb, ba, za);
+    else if (rows <= 8) pib_launch(mv_experts_kernel<WT, ROUND, EPI, 8>, grid, dim3(256), (size_t) 0, st, a, b, xva, xvb, ba, za);
+    else                pib_launch(mv_experts_kernel<WT, ROUND, EPI, MV_MAXB>, grid, dim3(256), (size_t) 0, st, a, b, xva, xvb, ba, za);
+}
+int pib_dense_mm_experts(const pib_mm & a, const pib_mm & b, cudaStream_t st) {
+    const int V = a.wtype == PIB_TYPE_BF16 ? 8 : 4;
+    auto fits = [&](const pib_mm & m) { return m.M >= 1 && m.M <= MV_MAXB && !m.x_bf16 && !m.Y2 && m.ldw % V == 0 && m.wz % V == 0 && ((uintptr_t) m.W & 15) == 0; };
+    const bool epi_ok = a.epi == PIB_EPI_NONE || (a.epi == PIB_EPI_SWIGLU_PAIR && a.N % 2 == 0 && b.N % 2 == 0);
+    if (!fits(a) || !fits(b) || !a.zrange || b.Z != 1 || b.zrange || b.xrows || a.wtype != b.wtype || a.exact != b.exact || a.epi != b.epi || !epi_ok || (a.exact && a.wtype != PIB_TYPE_F32)) {
+        const int rc = pib_dense_mm(a, st);
+        return rc != PIB_OK ? rc : pib_dense_mm(b, st);
+    }
+    auto dev = [](const pib_mm & m) {
+        return mm_dev{ m.W, m.ldw, m.wz, m.X, m.ldx, m.xz, m.xrows, m.xdiv < 1 ? 1 : m.xdiv, m.Y, m.ldy, m.yz, m.M, m.N, m.K, m.zrange, m.e0, m.e1, m.zlist, nullptr, 0, 0x7fffffff, nullptr };
+    };
+    auto xvec = [](const pib_mm & m) { return m.ldx % 4 == 0 && ((uintptr_t) m.X & 15) == 0; };
+    const int za = a.zlist && a.M < a.Z ? a.M : a.Z;
+#define EXPERTS_GO(WT, ROUND) do { if (a.epi == PIB_EPI_NONE) launch_experts<WT, ROUND, PIB_EPI_NONE>(dev(a), dev(b), xvec(a), xvec(b), za, st); \
+                                   else launch_experts<WT, ROUND, PIB_EPI_SWIGLU_PAIR>(dev(a), dev(b), xvec(a), xvec(b), za, st); } while (0)
+    if (a.wtype == PIB_TYPE_BF16) EXPERTS_GO(__nv_bfloat16, true);
+    else if (a.exact) EXPERTS_GO(float, false);
+    else EXPERTS_GO(float, true);
+#undef EXPERTS_GO
     PIB_CHECK(cudaGetLastError());
     return PIB_OK;
 }

@@ -30,7 +30,7 @@ struct pib_hybrid_ctx {
     float * h2 = nullptr, * cv = nullptr, * vfirst = nullptr, * mixes = nullptr;   // parallel layers: second norm (pre-norm layers: the stream's second buffer); convolved q | k | v; first mixing layer's values; token-shift mixes
     float * rg = nullptr, * y2 = nullptr;       // gated frame: the residual gate's logits; the second branch's output
     float * cat = nullptr;                      // [stream ; embedding] rows of models whose layers are walked again
-    int32_t * ids = nullptr, * perm = nullptr, * inv = nullptr, * counts = nullptr, * offs = nullptr;
+    int32_t * ids = nullptr, * perm = nullptr, * inv = nullptr, * counts = nullptr, * offs = nullptr, * act = nullptr, * done = nullptr;   // act: the experts with rows of a small batch; done: 0 between launches
     // batch bookkeeping: pinned staging ring + device copy
     static const int RING = 4;
     int32_t *   meta_host[RING] = { nullptr, nullptr, nullptr, nullptr };
@@ -59,14 +59,14 @@ static const char * const HK_NAMES[] = { "cellmap", "embed_ln", "canon_conv", "m
                                          "hyper_norm", "mm_mamba2_in", "mamba2_conv", "mamba2_prep", "mamba2_scan", "gated_group_norm", "mm_mamba2_o", "qkv_rope", "diff_combine",
                                          "mm_gate_up",
                                          "gated_norm", "input_conv", "mm_res_gate", "mm_attn_mem_proj", "attn_mem_prep", "memory_scan", "attn_mem_gate", "mm_attn_mem_o", "mm_gate_pair", "memory_scan_mm",
-                                         "sandwich_norm", "moe_route_sort" };
+                                         "sandwich_norm", "moe_route_sort", "norm_route", "mm_experts_up_all", "mm_experts_down_all" };
 enum { HK_CELLMAP, HK_EMBED, HK_CANON, HK_DQKV, HK_LPREP, HK_UQ, HK_ABSORB, HK_LATTN, HK_UV, HK_AO, HK_QFV, HK_GATES, HK_SCAN, HK_HO, HK_LNRES, HK_UP, HK_POLY, HK_DOWN,
        HK_ROUTER, HK_ROUTE, HK_SORT, HK_EUP, HK_EDOWN, HK_SUP, HK_SDOWN, HK_COMBINE, HK_FINAL, HK_HEAD, HK_SAMPLE, HK_LATTN_MM,
        HK_EMBSCALE, HK_NORM2, HK_QKV, HK_QKVCONV, HK_APREP, HK_KVATTN, HK_KVATTN_MM, HK_SHIFT, HK_RKVG, HK_DECAY, HK_DECAYACT, HK_WKVSCAN, HK_DPREP, HK_DSCAN, HK_GHNORM, HK_GLU,
        HK_PSUM, HK_EMBPAIR, HK_PRENORM, HK_CONCAT, HK_LOOPIN, HK_SSMIN, HK_SSMCONV, HK_SSMX, HK_SSMDT, HK_SSMSCAN, HK_SSMO, HK_DUALPROJ, HK_DUALPREP, HK_DECAYSCAN, HK_DUALGATE,
        HK_DUALO, HK_HYPER, HK_M2IN, HK_M2CONV, HK_M2PREP, HK_M2SCAN, HK_GGNORM, HK_M2O, HK_QKVROPE, HK_DIFFCOMB, HK_GATEUP,
        HK_GNORM, HK_INCONV, HK_RGATE, HK_AMPROJ, HK_AMPREP, HK_MEMSCAN, HK_AMGATE, HK_AMO, HK_GATE_PAIR, HK_MEMSCAN_MM,
-       HK_SANDWICH, HK_ROUTE_SORT, HK_COUNT };
+       HK_SANDWICH, HK_ROUTE_SORT, HK_NORM_ROUTE, HK_EUP_ALL, HK_EDOWN_ALL, HK_COUNT };
 const char * pib_hybrid_kind_name(int k) { return k >= 0 && k < HK_COUNT ? HK_NAMES[k] : "?"; }
 
 // fetch and clear the records; returns the count (the stream is synchronised)
@@ -164,10 +164,10 @@ static int grow_chunk(pib_context * c, size_t need) {
 static void free_scratch(pib_hybrid_ctx * x) {
     for (void * b : { (void *) x->x, (void *) x->h, (void *) x->y, (void *) x->proj, (void *) x->cq, (void *) x->q, (void *) x->qlat, (void *) x->lat, (void *) x->att,
                       (void *) x->rlog, (void *) x->wts, (void *) x->eup, (void *) x->edn, (void *) x->ysh, (void *) x->ids, (void *) x->perm, (void *) x->inv,
-                      (void *) x->counts, (void *) x->offs, (void *) x->h2, (void *) x->cv, (void *) x->vfirst, (void *) x->mixes, (void *) x->cat, (void *) x->rg, (void *) x->y2 }) if (b) cudaFree(b);
+                      (void *) x->counts, (void *) x->offs, (void *) x->act, (void *) x->done, (void *) x->h2, (void *) x->cv, (void *) x->vfirst, (void *) x->mixes, (void *) x->cat, (void *) x->rg, (void *) x->y2 }) if (b) cudaFree(b);
     x->x = x->h = x->y = x->proj = x->cq = x->q = x->qlat = x->lat = x->att = x->rlog = x->wts = x->eup = x->edn = x->ysh = nullptr;
     x->h2 = x->cv = x->vfirst = x->mixes = x->cat = x->rg = x->y2 = nullptr;
-    x->ids = x->perm = x->inv = x->counts = x->offs = nullptr;
+    x->ids = x->perm = x->inv = x->counts = x->offs = x->act = x->done = nullptr;
     x->cap = 0;
 }
 
@@ -207,7 +207,7 @@ static int grow_scratch(pib_context * c, int T) {
                     fl(&x->qlat, (size_t) hy->w_lat) && fl(&x->lat, (size_t) hy->w_lat) && fl(&x->att, (size_t) hy->w_att) && fl(&x->rlog, (size_t) hy->w_router) &&
                     fl(&x->wts, (size_t) hy->w_pairs) && fl(&x->eup, (size_t) hy->w_eup) && fl(&x->edn, (size_t) hy->w_pairs * W) && fl(&x->ysh, hy->w_pairs ? W : 0) &&
                     in(&x->ids, n * hy->w_pairs) && in(&x->perm, n * hy->w_pairs) && in(&x->inv, n * hy->w_pairs) && in(&x->counts, (size_t) hy->w_router + 1) &&
-                    in(&x->offs, (size_t) hy->w_router + 2) && fl(&x->h2, hy->form == PIB_FORM_PARALLEL || hy->form == PIB_FORM_PRENORM || hy->form == PIB_FORM_GATED ? W : 0) && fl(&x->cv, (size_t) hy->w_conv) &&
+                    in(&x->offs, (size_t) hy->w_router + 2) && in(&x->act, (size_t) hy->w_router + 2) && in(&x->done, hy->w_router ? 4 : 0) && (!x->done || cudaMemset(x->done, 0, 16) == cudaSuccess) && fl(&x->h2, hy->form == PIB_FORM_PARALLEL || hy->form == PIB_FORM_PRENORM || hy->form == PIB_FORM_GATED ? W : 0) && fl(&x->cv, (size_t) hy->w_conv) &&
                     fl(&x->vfirst, (size_t) hy->w_vfirst) && fl(&x->mixes, (size_t) hy->w_shift) && fl(&x->cat, (size_t) hy->w_cat) &&
                     fl(&x->rg, (size_t) hy->w_gate) && fl(&x->y2, (size_t) hy->w_y2);
     if (!ok) { cudaGetLastError(); free_scratch(x); pib_set_error("decode: out of memory for the work buffers of %d tokens", T); return PIB_ERR_NOMEM; }
@@ -560,40 +560,53 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
     // experts: rows gate | up, the router's weight multiplies the expert's input, i.e. both products before the clamp (glu_clamp); silu-gated
     // experts: gate and up rows interleaved, gate and product ride on the matmul's way out, the weights multiply the outputs.  The router may have
     // outputs that are no experts (identity): their pairs sort behind all others and no matmul sees them
-    auto run_experts = [&](const pib_hlayer & L, const float * min, int * ld_shared) -> int {
+    auto router_of = [&](const pib_hlayer & L) { return pib_router{ L.n_experts + L.identity, L.n_experts, L.top, L.route, L.groups, L.keep_groups, L.route_scale, L.correction }; };
+    auto run_experts = [&](const pib_hlayer & L, const float * min, int * ld_shared, bool routed = false) -> int {
         const int  n_exp = L.n_experts, E = n_exp + L.identity, top = L.top, P = T * top;
         const bool clamp = L.expert == PIB_EXPERT_GLU_CLAMP, paired = L.expert == PIB_EXPERT_SWIGLU;
         const int  NU = (clamp || paired ? 2 : 1) * L.ff_e, ldu = paired ? L.ff_e : NU, epi = clamp ? PIB_EPI_NONE : paired ? PIB_EPI_SWIGLU_PAIR : PIB_EPI_RELU2;
         const double Pe = (double) P * n_exp / E;                      // pairs of experts, if the router spreads them evenly
         const double touched = Pe >= n_exp ? 1.0 : Pe / n_exp;         // weights of experts without a row are not read
-        const pib_router R = { E, top, L.route, L.groups, L.keep_groups, L.route_scale, L.correction };
-        RC(HK_ROUTER, mmfl(L.router), mmby(L.router), mm(L.router, min, W, x->rlog, E, PIB_EPI_NONE));
-        if (pib_moe_route_sort_fits(T, R)) {
-            RC(HK_ROUTE_SORT, 0, 4.0 * Td * E + 16.0 * P, pib_moe_route_sort(x->rlog, T, R, x->ids, x->wts, x->offs, x->perm, x->inv, st));
-        } else {
-            RC(HK_ROUTE, 0, 4.0 * Td * E, pib_moe_route(x->rlog, T, R, x->ids, x->wts, st));
-            RC(HK_SORT, 0, 4.0 * P * (E + 3.0), pib_moe_sort(x->ids, P, E, x->counts, x->offs, x->perm, x->inv, st)); nk++;
+        const pib_router R = router_of(L);
+        const bool small = pib_moe_route_sort_fits(T, R);              // the sort of a small batch also lists the experts that have rows
+        if (!routed) {                                                 // (else the norm's launch has done it)
+            RC(HK_ROUTER, mmfl(L.router), mmby(L.router), mm(L.router, min, W, x->rlog, E, PIB_EPI_NONE));
+            if (small) {
+                RC(HK_ROUTE_SORT, 0, 4.0 * Td * E + 16.0 * P, pib_moe_route_sort(x->rlog, T, R, x->ids, x->wts, x->offs, x->perm, x->inv, x->act, st));
+            } else {
+                RC(HK_ROUTE, 0, 4.0 * Td * E, pib_moe_route(x->rlog, T, R, x->ids, x->wts, st));
+                RC(HK_SORT, 0, 4.0 * P * (E + 3.0), pib_moe_sort(x->ids, P, E, x->counts, x->offs, x->perm, x->inv, st)); nk++;
+            }
         }
-        {   // up-projection of every (token, expert) pair, pairs grouped by expert
-            pib_mm a;
-            a.W = L.e_up->base; a.wtype = L.e_up->type; a.ldw = W; a.wz = (int64_t) NU * W; a.X = min; a.ldx = W; a.xrows = x->perm; a.xdiv = top;
-            a.Y = x->eup; a.ldy = ldu; a.M = P; a.N = NU; a.K = W; a.Z = n_exp; a.zrange = x->offs; a.epi = epi; a.exact = exact;
-            RC(HK_EUP, 2.0 * Pe * NU * Wd, wbytes(L.e_up) * touched + 4.0 * Pe * (Wd + ldu), pib_dense_mm(a, st));
-            if (clamp) RC(HK_GLU, 0, 12.0 * P * L.ff_e, pib_glu_clamp(x->eup, NU, L.ff_e, L.limit_e, x->wts, x->perm, P, st));
-            pib_mm b;
-            b.W = L.e_down->base; b.wtype = L.e_down->type; b.ldw = L.ff_e; b.wz = (int64_t) W * L.ff_e; b.X = x->eup; b.ldx = ldu;
-            b.Y = x->edn; b.ldy = W; b.M = P; b.N = W; b.K = L.ff_e; b.Z = n_exp; b.zrange = x->offs; b.exact = exact;
-            RC(HK_EDOWN, 2.0 * Pe * L.ff_e * Wd, wbytes(L.e_down) * touched + 4.0 * Pe * (Wd + L.ff_e), pib_dense_mm(b, st));
-        }
+        // up-projection of every (token, expert) pair, pairs grouped by expert; the shared expert's over all tokens
+        pib_mm a, b, sa, sb;
+        a.W = L.e_up->base; a.wtype = L.e_up->type; a.ldw = W; a.wz = (int64_t) NU * W; a.X = min; a.ldx = W; a.xrows = x->perm; a.xdiv = top;
+        a.Y = x->eup; a.ldy = ldu; a.M = P; a.N = NU; a.K = W; a.Z = n_exp; a.zrange = x->offs; a.epi = epi; a.exact = exact;
+        b.W = L.e_down->base; b.wtype = L.e_down->type; b.ldw = L.ff_e; b.wz = (int64_t) W * L.ff_e; b.X = x->eup; b.ldx = ldu;
+        b.Y = x->edn; b.ldy = W; b.M = P; b.N = W; b.K = L.ff_e; b.Z = n_exp; b.zrange = x->offs; b.exact = exact;
+        if (small) a.zlist = b.zlist = x->act;
+        const double fl_up = 2.0 * Pe * NU * Wd, by_up = wbytes(L.e_up) * touched + 4.0 * Pe * (Wd + ldu), fl_dn = 2.0 * Pe * L.ff_e * Wd, by_dn = wbytes(L.e_down) * touched + 4.0 * Pe * (Wd + L.ff_e);
+        double by_su = 0;
         if (L.s_up) {
             const int ld = ((paired ? L.ff_s : (int) L.s_up->N) + 3) & ~3;
             *ld_shared = ld;
-            RC(HK_SUP, mmfl(L.s_up), wbytes(L.s_up) + 4.0 * Td * (Wd + ld), mm(L.s_up, min, W, x->proj, ld, epi));
-            if (clamp) RC(HK_GLU, 0, 12.0 * Td * L.ff_s, pib_glu_clamp(x->proj, ld, L.ff_s, L.limit_s, nullptr, nullptr, T, st));
-            pib_mm d;
-            d.W = L.s_down->base; d.wtype = L.s_down->type; d.ldw = L.ff_s; d.X = x->proj; d.ldx = ld; d.Y = x->ysh; d.ldy = W; d.M = T; d.N = W; d.K = L.ff_s;
-            d.exact = exact || L.s_down->type == PIB_TYPE_F32;
-            RC(HK_SDOWN, mmfl(L.s_down), mmby(L.s_down), pib_dense_mm(d, st));
+            sa = mm_of(L.s_up, min, W, x->proj, ld, epi);
+            by_su = wbytes(L.s_up) + 4.0 * Td * (Wd + ld);
+            sb.W = L.s_down->base; sb.wtype = L.s_down->type; sb.ldw = L.ff_s; sb.X = x->proj; sb.ldx = ld; sb.Y = x->ysh; sb.ldy = W; sb.M = T; sb.N = W; sb.K = L.ff_s;
+            sb.exact = exact || L.s_down->type == PIB_TYPE_F32;
+        }
+        if (L.s_up && paired && P <= 16) {       // decode steps: routed and shared experts share both launches
+            RC(HK_EUP_ALL, fl_up + mmfl(L.s_up), by_up + by_su, pib_dense_mm_experts(a, sa, st));
+            RC(HK_EDOWN_ALL, fl_dn + mmfl(L.s_down), by_dn + mmby(L.s_down), pib_dense_mm_experts(b, sb, st));
+            return PIB_OK;
+        }
+        RC(HK_EUP, fl_up, by_up, pib_dense_mm(a, st));
+        if (clamp) RC(HK_GLU, 0, 12.0 * P * L.ff_e, pib_glu_clamp(x->eup, NU, L.ff_e, L.limit_e, x->wts, x->perm, P, st));
+        RC(HK_EDOWN, fl_dn, by_dn, pib_dense_mm(b, st));
+        if (L.s_up) {
+            RC(HK_SUP, mmfl(L.s_up), by_su, pib_dense_mm(sa, st));
+            if (clamp) RC(HK_GLU, 0, 12.0 * Td * L.ff_s, pib_glu_clamp(x->proj, sa.ldy, L.ff_s, L.limit_s, nullptr, nullptr, T, st));
+            RC(HK_SDOWN, mmfl(L.s_down), mmby(L.s_down), pib_dense_mm(sb, st));
         }
         return PIB_OK;
     };
@@ -632,8 +645,10 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
     };
     // sandwich frame: what the sublayer before left is normed, scaled and added by the kernel that norms the stream for the next one
     pib_sublayer_y leftn;
-    auto sandwich = [&](const float * w, const float * b) -> int {
-        RC(HK_SANDWICH, 0, 4.0 * Td * Wd * ((leftn.y ? 3.0 : leftn.top ? 2.0 : 1.0) + leftn.top + (w ? 1.0 : 0.0)), pib_sandwich_norm(x->x, leftn, w, b, eps, T, W, w ? x->h : nullptr, st));
+    auto sandwich = [&](const float * w, const float * b, const pib_hlayer * moe = nullptr) -> int {
+        pib_norm_route nr;
+        if (moe) { nr.rows = (const float *) moe->router->base; nr.R = router_of(*moe); nr.ids = x->ids; nr.wts = x->wts; nr.offs = x->offs; nr.perm = x->perm; nr.inv = x->inv; nr.act = x->act; nr.done = x->done; }
+        RC(moe ? HK_NORM_ROUTE : HK_SANDWICH, moe ? mmfl(moe->router) : 0, (moe ? wbytes(moe->router) : 0.0) + 4.0 * Td * Wd * ((leftn.y ? 3.0 : leftn.top ? 2.0 : 1.0) + leftn.top + (w ? 1.0 : 0.0)), pib_sandwich_norm(x->x, leftn, w, b, eps, T, W, w ? x->h : nullptr, st, moe ? &nr : nullptr));
         leftn = pib_sublayer_y();
         return PIB_OK;
     };
@@ -644,13 +659,14 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
             if ((rc = sandwich(L.norm1, L.norm1_b)) != PIB_OK) return rc;
             if ((rc = run_mixer(L, x->h)) != PIB_OK) return rc;
             leftn.y = x->y; leftn.w = L.post1; leftn.b = L.post1_b;
-            if (L.mlp != PIB_MLP_NONE && (rc = sandwich(L.norm2, L.norm2_b)) != PIB_OK) return rc;
+            const bool routed = L.mlp == PIB_MLP_MOE && pib_norm_route_fits(T, W, router_of(L));      // small batches: the router rides on the norm
+            if (L.mlp != PIB_MLP_NONE && (rc = sandwich(L.norm2, L.norm2_b, routed ? &L : nullptr)) != PIB_OK) return rc;
             if (L.mlp == PIB_MLP_RELU2) {
                 RC(HK_UP, mmfl(L.up), mmby(L.up), mm(L.up, x->h, W, x->proj, L.ff, PIB_EPI_RELU2));
                 RC(HK_DOWN, mmfl(L.down), mmby(L.down), mm(L.down, x->proj, L.ff, x->y, W, PIB_EPI_NONE));
                 leftn.y = x->y;
             } else if (L.mlp == PIB_MLP_MOE && L.expert == PIB_EXPERT_SWIGLU) {
-                if ((rc = run_experts(L, x->h, &lds)) != PIB_OK) return rc;
+                if ((rc = run_experts(L, x->h, &lds, routed)) != PIB_OK) return rc;
                 leftn.y = L.s_up ? x->ysh : nullptr; leftn.edn = x->edn; leftn.wts = x->wts; leftn.ids = x->ids; leftn.inv = x->inv; leftn.hin = x->h; leftn.top = L.top; leftn.n_real = L.n_experts;
             } else if (L.mlp != PIB_MLP_NONE) { pib_set_error("decode: feed-forward %d in a sandwich layer", L.mlp); return PIB_ERR_UNSUPP; }
             if (L.mlp != PIB_MLP_NONE) { leftn.w = L.post2; leftn.b = L.post2_b; }

@@ -237,6 +237,7 @@ struct pib_mm {
     const int32_t * xrows = nullptr; int xdiv = 1;       // row m reads X row xrows[m] / xdiv (null: m)
     float *         Y = nullptr; int64_t ldy = 0, yz = 0;
     int             M = 0, N = 0, K = 0, Z = 1;
+    const int32_t * zlist = nullptr;                     // device [1 + Z], with zrange: [how many z have rows | which], so that a few-row launch need not look at the others (at most M of them)
     const int32_t * zrange = nullptr;                    // device [Z + 1]: z owns rows [zrange[z], zrange[z + 1]); null: all M rows, every z
     int             epi = PIB_EPI_NONE;
     float           e0 = 0.f, e1 = 0.f;                  // the epilogue's constants (xIELU: softplus(p), 1/2 + softplus(q))
@@ -268,6 +269,7 @@ template <int EPI, bool FAST> __device__ __forceinline__ float pib_glu_pair(floa
 #endif
 int pib_dense_mm(const pib_mm & a, cudaStream_t st);
 int pib_dense_mm_pair(const pib_mm & a, const pib_mm & b, cudaStream_t st);   // two independent matmuls; in decode steps one launch
+int pib_dense_mm_experts(const pib_mm & routed, const pib_mm & shared, cudaStream_t st);   // a grouped matmul and a plain one with the same epilogue; in decode steps one launch
 int pib_dense_mm_check(cudaStream_t st, int enqueue);   // dense_mma.cu: the error word of the bounded waits (1: copy it in stream order, 0: read the copy)
 pib_weight * pib_dense_upload(int type, const void * host, int64_t N, int64_t K);   // type: PIB_TYPE_BF16 / PIB_TYPE_F32, row-major [N][K]
 
@@ -300,10 +302,12 @@ int pib_hgrn2_gates(float * qfv, int ld, const float * f_bias, const float * low
 int pib_hgrn2_scan(const float * qfv, int ld, const pib_hlayer & L, const pib_hbatch & b, float * state, size_t state_stride, const float * onorm, float eps,
                    float * out, cudaStream_t st);
 int pib_polynorm(float * z, int T, int F, const float * act4, float eps, cudaStream_t st);
-struct pib_router { int E = 0, top = 0, mode = PIB_ROUTE_SOFTMAX_RENORM, groups = 1, keep_groups = 1; float scale = 1.f; const float * correction = nullptr; };   // E: outputs, identity ones included
+struct pib_router { int E = 0, n_real = 0, top = 0, mode = PIB_ROUTE_SOFTMAX_RENORM, groups = 1, keep_groups = 1; float scale = 1.f; const float * correction = nullptr; };   // E outputs, the first n_real of them experts
+int pib_moe_router_check(const pib_router & r);
 int pib_moe_route(const float * logits, int T, const pib_router & r, int32_t * ids, float * wts, cudaStream_t st);
 bool pib_moe_route_sort_fits(int T, const pib_router & r);
-int pib_moe_route_sort(const float * logits, int T, const pib_router & r, int32_t * ids, float * wts, int32_t * offs, int32_t * perm, int32_t * inv, cudaStream_t st);   // both steps of a small batch in one launch
+int pib_moe_route_sort(const float * logits, int T, const pib_router & r, int32_t * ids, float * wts, int32_t * offs, int32_t * perm, int32_t * inv, int32_t * act,
+                       cudaStream_t st);   // both steps of a small batch in one launch; act = [how many experts have pairs | which]
 int pib_moe_sort(const int32_t * ids, int n_pairs, int E, int32_t * counts, int32_t * offs, int32_t * perm, int32_t * inv, cudaStream_t st);
 int pib_moe_combine(const float * shared, const float * edn, const float * wts, const int32_t * inv, int T, int top, int W, float * y, cudaStream_t st);
 int pib_cellmap_set(int32_t * cellmap, int n_ctx, const pib_hbatch & b, cudaStream_t st);
@@ -369,7 +373,13 @@ struct pib_sublayer_y {              // a sublayer's output: y, plus (top > 0) t
     int top = 0, n_real = 0;
     const float * w = nullptr, * b = nullptr;       // the norm behind it (times layer scale and residual multiplier)
 };
-int pib_sandwich_norm(float * x, const pib_sublayer_y & o, const float * w, const float * b, float eps, int T, int W, float * h, cudaStream_t st);
+struct pib_norm_route {              // the router of the mixture that reads h, on the same launch (small batches): float32 rows [E][W]
+    const float * rows = nullptr; pib_router R;
+    int32_t * ids = nullptr, * offs = nullptr, * perm = nullptr, * inv = nullptr, * act = nullptr, * done = nullptr;   // done: a word that is 0 between launches
+    float * wts = nullptr;
+};
+bool pib_norm_route_fits(int T, int W, const pib_router & R);
+int pib_sandwich_norm(float * x, const pib_sublayer_y & o, const float * w, const float * b, float eps, int T, int W, float * h, cudaStream_t st, const pib_norm_route * route = nullptr);
 // chunk_scan.cu: n tokens of one segment (batch rows t0 ..) of a recurrence with one decay per head and token, as matmuls (served mode)
 struct pib_chunk_scan {
     const float * q = nullptr, * k = nullptr, * v = nullptr; int ldq = 0, ldk = 0, ldv = 0;   // rows [G][D], [G][D], [H][V] per token

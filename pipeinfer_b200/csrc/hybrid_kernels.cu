@@ -9,6 +9,7 @@
 //   HGRN2: S_t = diag(f_t) S_{t-1} + (1 - f_t) v_t^T, o_t = S_t^T q_t, per head, state in fp32 per sequence
 //   PolyNorm, mixture-of-experts routing (softmax, top-k, renormalise), grouping of (token, expert) pairs by expert
 #include "hybrid.cuh"
+#include "moe_route.cuh"
 
 #include <algorithm>
 
@@ -684,63 +685,7 @@ int pib_polynorm(float * z, int T, int F, const float * act4, float eps, cudaStr
 }
 
 // ---- mixture of experts ------------------------------------------------------------------------------------------------------------
-// One warp per token: the `top` outputs of the router with the largest choice value (ties: the lower index).
-//   PIB_ROUTE_SOFTMAX_RENORM:  scores = softmax over the E logits, weights = score / (sum of the chosen + 1e-20); chosen by the logits
-//   PIB_ROUTE_SIGMOID:         weights = sigmoid(logit) of the chosen, as they are (the order of the logits is the order of their sigmoids)
-//   PIB_ROUTE_SOFTMAX_GROUPS:  scores = softmax over the E logits; the choice values are score + correction; the outputs form equal groups of neighbours, a group
-//                              stands for its largest choice value, and only members of the keep_groups best groups are chosen; weights = score * scale
-// cv: the warp's scratch in shared memory, E + groups floats.  Output k of the token goes to ids[k], wts[k].
-#define MOE_MAX_TOP 16
-__device__ __forceinline__ void moe_route_token(const float * __restrict__ z, const pib_router & R, float * cv, int lane, int32_t * ids, float * wts) {
-    const int E = R.E;
-    float mx = -INFINITY;
-    for (int i = lane; i < E; i += 32) mx = fmaxf(mx, z[i]);
-    mx = warp_max(mx);
-    float sum = 0.f;
-    for (int i = lane; i < E; i += 32) sum += expf(z[i] - mx);
-    sum = warp_sum(sum);
-    const bool grouped = R.mode == PIB_ROUTE_SOFTMAX_GROUPS;
-    for (int i = lane; i < E; i += 32) cv[i] = grouped ? expf(z[i] - mx) / sum + (R.correction ? R.correction[i] : 0.f) : z[i];
-    if (grouped && R.keep_groups < R.groups) {
-        float *   gv  = cv + E;
-        const int per = E / R.groups;
-        __syncwarp();
-        for (int g = lane; g < R.groups; g += 32) {
-            float best = -INFINITY;
-            for (int i = g * per; i < (g + 1) * per; i++) best = fmaxf(best, cv[i]);
-            gv[g] = best;
-        }
-        __syncwarp();
-        for (int i = lane; i < E; i += 32) {
-            const int g = i / per;
-            int better = 0;
-            for (int o = 0; o < R.groups; o++) better += gv[o] > gv[g] || (gv[o] == gv[g] && o < g);
-            if (better >= R.keep_groups) cv[i] = -INFINITY;
-        }
-    }
-    float tot = 0.f, score[MOE_MAX_TOP];
-    int   chosen[MOE_MAX_TOP];
-    for (int k = 0; k < R.top; k++) {
-        float bv = -INFINITY;
-        int   bi = 0x7fffffff;
-        for (int i = lane; i < E; i += 32) { const float v = cv[i]; if (v > bv || (v == bv && v > -INFINITY && i < bi)) { bv = v; bi = i; } }      // a lane reads back only what it wrote
-        for (int o = 16; o > 0; o >>= 1) {
-            const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
-            const int   oi = __shfl_xor_sync(0xffffffffu, bi, o);
-            if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
-        }
-        if (bi >= E) bi = k;                                // nothing comparable is left (logits that are no numbers): stay inside the arrays
-        if ((bi & 31) == lane) cv[bi] = -INFINITY;
-        chosen[k] = bi;
-        score[k]  = R.mode == PIB_ROUTE_SIGMOID ? 1.0f / (1.0f + expf(-z[bi])) : expf(z[bi] - mx) / sum;
-        tot += score[k];
-    }
-    if (lane == 0)
-        for (int k = 0; k < R.top; k++) {
-            ids[k] = chosen[k];
-            wts[k] = R.mode == PIB_ROUTE_SIGMOID ? score[k] : grouped ? score[k] * R.scale : score[k] / (tot + 1e-20f);
-        }
-}
+// routing of a token, sorting of a small batch's pairs: moe_route.cuh
 __global__ void __launch_bounds__(128) moe_route_kernel(const float * __restrict__ logits, int T, pib_router R, int32_t * __restrict__ ids, float * __restrict__ wts) {
     pib_pdl_wait();
     pib_pdl_trigger();
@@ -749,7 +694,7 @@ __global__ void __launch_bounds__(128) moe_route_kernel(const float * __restrict
     if (t >= T) return;
     moe_route_token(logits + (size_t) t * R.E, R, route_sm + (size_t) warp * (R.E + R.groups), threadIdx.x & 31, ids + (size_t) t * R.top, wts + (size_t) t * R.top);
 }
-static int moe_router_check(const pib_router & R) {
+int pib_moe_router_check(const pib_router & R) {
     if (R.top < 1 || R.top > MOE_MAX_TOP || R.top > R.E) { pib_set_error("router: top %d of %d experts (max %d)", R.top, R.E, MOE_MAX_TOP); return PIB_ERR_UNSUPP; }
     if (R.groups < 1 || R.E % R.groups || R.keep_groups < 1 || R.keep_groups > R.groups || R.top > R.keep_groups * (R.E / R.groups)) {
         pib_set_error("router: %d outputs in %d groups of which %d take part, top %d", R.E, R.groups, R.keep_groups, R.top); return PIB_ERR_UNSUPP;
@@ -758,45 +703,32 @@ static int moe_router_check(const pib_router & R) {
     return PIB_OK;
 }
 int pib_moe_route(const float * logits, int T, const pib_router & R, int32_t * ids, float * wts, cudaStream_t st) {
-    const int rc = moe_router_check(R);
+    const int rc = pib_moe_router_check(R);
     if (rc != PIB_OK) return rc;
     pib_launch(moe_route_kernel, dim3((T + 3) / 4), dim3(128), (size_t) 16 * (R.E + R.groups), st, logits, T, R, ids, wts);
     CKL();
     return PIB_OK;
 }
 
-// routing and sorting of a small batch in one block: a warp per token in turn, then a thread per router output counts and places its pairs (in pair order, as
-// the kernels below do)
-#define MOE_SMALL_T 16
-#define MOE_SMALL_PAIRS 256
+// routing and sorting of a small batch in one block: a warp per token, then the block sorts
 __global__ void __launch_bounds__(512) moe_route_sort_kernel(const float * __restrict__ logits, int T, pib_router R, int32_t * __restrict__ ids, float * __restrict__ wts,
-                                                             int32_t * __restrict__ offs, int32_t * __restrict__ perm, int32_t * __restrict__ inv) {
+                                                             int32_t * __restrict__ offs, int32_t * __restrict__ perm, int32_t * __restrict__ inv, int32_t * __restrict__ act) {
     pib_pdl_wait();
     pib_pdl_trigger();
     extern __shared__ float route_sm[];
-    __shared__ int32_t sid[MOE_SMALL_PAIRS], cnt[512];
+    __shared__ int32_t sid[MOE_SMALL_PAIRS], cnt[MOE_SMALL_E];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, P = T * R.top;
     if (warp < T) moe_route_token(logits + (size_t) warp * R.E, R, route_sm + (size_t) warp * (R.E + R.groups), lane, sid + warp * R.top, wts + (size_t) warp * R.top);
     __syncthreads();
     for (int i = threadIdx.x; i < P; i += blockDim.x) ids[i] = sid[i];
-    const int e = threadIdx.x;
-    int n = 0;
-    for (int i = 0; i < P; i++) n += sid[i] == e;
-    cnt[e] = n;
-    __syncthreads();
-    if (e >= R.E) return;
-    int o = 0;
-    for (int i = 0; i < e; i++) o += cnt[i];
-    offs[e] = o;
-    if (e == R.E - 1) offs[R.E] = o + n;
-    if (n > 0) for (int i = 0; i < P; i++) if (sid[i] == e) { perm[o] = i; inv[i] = o; o++; }
+    moe_sort_small(sid, P, R.E, R.n_real, cnt, offs, perm, inv, act);
 }
-bool pib_moe_route_sort_fits(int T, const pib_router & R) { return T <= MOE_SMALL_T && T * R.top <= MOE_SMALL_PAIRS && R.E <= 512 && (size_t) T * (R.E + R.groups) * 4 <= 40 * 1024; }
-int pib_moe_route_sort(const float * logits, int T, const pib_router & R, int32_t * ids, float * wts, int32_t * offs, int32_t * perm, int32_t * inv, cudaStream_t st) {
-    const int rc = moe_router_check(R);
+bool pib_moe_route_sort_fits(int T, const pib_router & R) { return T <= MOE_SMALL_T && T * R.top <= MOE_SMALL_PAIRS && R.E <= MOE_SMALL_E && (size_t) T * (R.E + R.groups) * 4 <= 40 * 1024; }
+int pib_moe_route_sort(const float * logits, int T, const pib_router & R, int32_t * ids, float * wts, int32_t * offs, int32_t * perm, int32_t * inv, int32_t * act, cudaStream_t st) {
+    const int rc = pib_moe_router_check(R);
     if (rc != PIB_OK) return rc;
     const int threads = ((R.E > 32 * T ? R.E : 32 * T) + 31) & ~31;
-    pib_launch(moe_route_sort_kernel, dim3(1), dim3(threads), (size_t) T * (R.E + R.groups) * 4, st, logits, T, R, ids, wts, offs, perm, inv);
+    pib_launch(moe_route_sort_kernel, dim3(1), dim3(threads), (size_t) T * (R.E + R.groups) * 4, st, logits, T, R, ids, wts, offs, perm, inv, act);
     CKL();
     return PIB_OK;
 }

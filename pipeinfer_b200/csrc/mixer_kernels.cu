@@ -12,6 +12,9 @@
 //   the parallel layer's sum: x += mixer + shared expert * sigmoid(gate logit) + routed experts
 #include "hybrid.cuh"
 
+#include <algorithm>
+
+#include <cooperative_groups.h>
 #include <cuda_bf16.h>
 
 #define CKL() do { cudaError_t e__ = cudaGetLastError(); if (e__ != cudaSuccess) { pib_set_error("%s:%d: launch failed: %s", __FILE__, __LINE__, cudaGetErrorString(e__)); return PIB_ERR_CUDA; } } while (0)
@@ -110,7 +113,8 @@ int pib_swa_prep(const float * cv, int ldc, const pib_hlayer & L, float eps, con
 // grid (token, head group); a block holds HPB query heads x KS key shares, one warp each.  A warp walks its share of the window
 // [max(0, p - window + 1), p] (chunk mask: of the token's chunk [p - p % window, p]) and the kept first positions [0, keep) through the slot's position -> cell table, UK
 // keys per trip (their rows are in flight together and their sums cross the lanes side by side), keeps a running maximum / denominator / weighted sum of value
-// rows, and the shares of a head are merged in shared memory.  A sink (optional) is one more logit without a row: the running state of
+// rows, and the shares of a head are merged in shared memory; CL blocks of a thread-block cluster may divide a head's shares further (few tokens over a long
+// window: decoding) and are merged through distributed shared memory.  A sink (optional) is one more logit without a row: the running state of
 // share 0 starts at (max = sink, denominator = 1).  softcap > 0: a score becomes softcap tanh(score / softcap).  Distance biases (optional) join the score
 // behind the cap: -slopes[h] (p - j), or rel[h][min(p - j, n_rel - 1)].  gate (optional): every output value is multiplied by sigmoid(gate).
 struct kva_args {
@@ -120,18 +124,34 @@ struct kva_args {
     const float * sink, * slopes, * rel; int n_rel;
     const int32_t * pos, * slot;
     const float * cache; int cache_row;
-    const int32_t * cellmap; int n_ctx, HPB, KS;
+    const int32_t * cellmap; int n_ctx, HPB, KS, CL;
     float * out;
     const int32_t * skip;
 };
+// one warp merges n <= 32 partial states (max at [V], denominator at [V + 1]); a share that saw no key has max -inf and counts for nothing
+template <int RPL> __device__ __forceinline__ void kva_merge(const float * base, int n, int V, int lane, float & M, float & L, float (&o)[RPL]) {
+    const float * mine = base + (size_t) lane * (V + 2);
+    const float   mk = lane < n ? mine[V] : -INFINITY;
+    M = warp_max(mk);
+    const float f = mk == -INFINITY ? 0.f : expf(mk - M);
+    L = warp_sum(lane < n ? mine[V + 1] * f : 0.f);
+#pragma unroll
+    for (int i = 0; i < RPL; i++) o[i] = 0.f;
+    for (int k = 0; k < n; k++) {
+        const float   fk = __shfl_sync(0xffffffffu, f, k);
+        const float * pk = base + (size_t) k * (V + 2);
+#pragma unroll
+        for (int i = 0; i < RPL; i++) { const int r = i * 32 + lane; if (r < V) o[i] = fmaf(pk[r], fk, o[i]); }
+    }
+}
 template <int RPL, int UK>
 __global__ void __launch_bounds__(512) kv_attn_kernel(kva_args A) {
     pib_pdl_wait();
     pib_pdl_trigger();
-    extern __shared__ float sm[];                 // [HPB * KS][V + 2] partial states
-    const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, H = A.H, D = A.D, V = A.V, KS = A.KS;
+    extern __shared__ float sm[];                 // [HPB * KS (+ 1 in a cluster: the block's own merged state)][V + 2] partial states
+    const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, H = A.H, D = A.D, V = A.V, KS = A.KS, CL = A.CL, rank = blockIdx.y % CL;
     if (A.skip && A.skip[t]) return;              // this token's segment goes through the matmul form
-    const int hl = warp / KS, ks = warp % KS, h = blockIdx.y * A.HPB + hl;
+    const int hl = warp / KS, ks = warp % KS, h = blockIdx.y / CL * A.HPB + hl;
     const int p = A.pos[t], lo = A.mask == PIB_MASK_CHUNK ? p - p % A.window : max(0, p - A.window + 1);
     const bool live = h < H;
     float qv[RPL], acc[RPL];
@@ -142,18 +162,19 @@ __global__ void __launch_bounds__(512) kv_attn_kernel(kva_args A) {
         const float * qp = A.q.q + (size_t) t * A.q.ldq + (size_t) h * D;
 #pragma unroll
         for (int i = 0; i < RPL; i++) { const int r = i * 32 + lane; qv[i] = r < D ? qp[r] * A.scale : 0.f; acc[i] = 0.f; }
-        if (ks == 0 && A.sink) { m = A.sink[h]; l = 1.f; }
+        if (ks == 0 && rank == 0 && A.sink) { m = A.sink[h]; l = 1.f; }
         const int32_t * map = A.cellmap + (size_t) A.slot[t] * A.n_ctx;
         const float *   rel = A.rel ? A.rel + (size_t) h * A.n_rel : nullptr;
         const float     slope = A.slopes ? A.slopes[h] : 0.f;
         const size_t ko = (size_t) (g * A.maps + mp) * D, vo = (size_t) A.G * A.maps * D + (size_t) g * V;
         const int nf = min(A.keep, lo), n_keys = nf + p - lo + 1;        // kept positions in front of the window, then the window
-        for (int e0 = ks; e0 < n_keys; e0 += KS * UK) {
+        const int all = KS * CL;                                         // shares of a head
+        for (int e0 = rank * KS + ks; e0 < n_keys; e0 += all * UK) {
             float s[UK], c[UK][RPL];
             int   dist[UK];
 #pragma unroll
             for (int u = 0; u < UK; u++) {
-                const int e = min(e0 + u * KS, n_keys - 1), j = e < nf ? e : lo + e - nf;      // a trip past the end reads the last key again; its score is dropped below
+                const int e = min(e0 + u * all, n_keys - 1), j = e < nf ? e : lo + e - nf;      // a trip past the end reads the last key again; its score is dropped below
                 dist[u] = p - j;
                 const float * row = A.cache + (size_t) map[j] * A.cache_row;
                 s[u] = 0.f;
@@ -167,7 +188,7 @@ __global__ void __launch_bounds__(512) kv_attn_kernel(kva_args A) {
                 if (A.softcap > 0.f) s[u] = A.softcap * tanhf(s[u] / A.softcap);
                 if (A.slopes) s[u] -= slope * (float) dist[u];
                 if (rel) s[u] += rel[min(dist[u], A.n_rel - 1)];
-                if (UK > 1 && e0 + u * KS >= n_keys) s[u] = -INFINITY;
+                if (UK > 1 && e0 + u * all >= n_keys) s[u] = -INFINITY;
                 mn = fmaxf(mn, s[u]);
             }
             const float a = expf(m - mn);                                              // m == -inf only before the first key: a = 0
@@ -189,22 +210,34 @@ __global__ void __launch_bounds__(512) kv_attn_kernel(kva_args A) {
         if (lane == 0) { part[V] = m; part[V + 1] = l; }
     }
     __syncthreads();
-    if (live && ks == 0) {
-        const float * base = sm + (size_t) (hl * KS) * (V + 2);
-        float M = -INFINITY;
-        for (int k = 0; k < KS; k++) M = fmaxf(M, base[(size_t) k * (V + 2) + V]);
-        float Lsum = 0.f, o[RPL];
+    float M = -INFINITY, Lsum = 0.f, o[RPL];
+    if (live && ks == 0) kva_merge<RPL>(sm + (size_t) (hl * KS) * (V + 2), KS, V, lane, M, Lsum, o);
+    if (CL > 1) {
+        cooperative_groups::cluster_group cl = cooperative_groups::this_cluster();
+        float * mine = sm + (size_t) KS * (V + 2);
+        if (warp == 0) {
 #pragma unroll
-        for (int i = 0; i < RPL; i++) o[i] = 0.f;
-        for (int k = 0; k < KS; k++) {
-            const float * pk = base + (size_t) k * (V + 2);
-            const float   mk = pk[V];
-            if (mk == -INFINITY) continue;           // a share that saw no key
-            const float f = expf(mk - M);
-            Lsum = fmaf(pk[V + 1], f, Lsum);
-#pragma unroll
-            for (int i = 0; i < RPL; i++) { const int r = i * 32 + lane; if (r < V) o[i] = fmaf(pk[r], f, o[i]); }
+            for (int i = 0; i < RPL; i++) { const int r = i * 32 + lane; if (r < V) mine[r] = o[i]; }
+            if (lane == 0) { mine[V] = M; mine[V + 1] = Lsum; }
         }
+        cl.sync();
+        if (warp == 0 && rank == 0) {
+            const float mk = lane < CL ? cl.map_shared_rank(mine, lane)[V] : -INFINITY;
+            M = warp_max(mk);
+            const float f = mk == -INFINITY ? 0.f : expf(mk - M);
+            Lsum = warp_sum(lane < CL ? cl.map_shared_rank(mine, lane)[V + 1] * f : 0.f);
+#pragma unroll
+            for (int i = 0; i < RPL; i++) o[i] = 0.f;
+            for (int k = 0; k < CL; k++) {
+                const float   fk = __shfl_sync(0xffffffffu, f, k);
+                const float * pk = cl.map_shared_rank(mine, k);
+#pragma unroll
+                for (int i = 0; i < RPL; i++) { const int r = i * 32 + lane; if (r < V) o[i] = fmaf(pk[r], fk, o[i]); }
+            }
+        }
+        cl.sync();                                       // the other blocks' states were read
+    }
+    if (live && ks == 0 && rank == 0) {
         const float inv = 1.0f / Lsum;
         float * op = A.out + ((size_t) t * H + h) * V;
         const float * gp = A.q.gate ? A.q.gate + (size_t) t * A.q.ldg + (size_t) h * V : nullptr;
@@ -219,14 +252,19 @@ int pib_kv_attention(const pib_kv_query & q, const pib_hlayer & L, const pib_hba
     const int HPB = (long long) b.T * H <= 1024 ? 1 : (H < 4 ? H : 4);
     int KS = 16 / HPB;
     if (L.window + L.keep < 64) KS = 1;
-    const size_t smem = (size_t) HPB * KS * (V + 2) * 4;
-    dim3 grid((unsigned) b.T, (unsigned) ((H + HPB - 1) / HPB));
+    // few tokens over a long reach: up to 8 blocks of a cluster share a head's keys, as long as the machine has room for them
+    const int64_t reach = std::min<int64_t>((int64_t) L.window + L.keep, n_ctx);
+    int CL = 1;
+    while (HPB == 1 && KS == 16 && CL < 8 && reach >= 128 * CL && (long long) b.T * H * CL * 2 <= 2 * 148) CL *= 2;
+    const size_t smem = (size_t) (HPB * KS + (CL > 1)) * (V + 2) * 4;
+    dim3 grid((unsigned) b.T, (unsigned) ((H + HPB - 1) / HPB * CL));
     const int threads = HPB * KS * 32;
     const kva_args A = { q, H, L.kv_heads, L.maps, L.dim, V, L.scale, L.window, L.mask, L.keep, L.softcap, L.sink, L.slopes, L.rel, L.n_rel, b.pos, b.slot, cache, cache_row, cellmap, n_ctx,
-                         HPB, KS, out, skip };
+                         HPB, KS, CL, out, skip };
 #define KA_GO(RPL, UK) do {                                                                                                              \
         if (smem > 48 * 1024) cudaFuncSetAttribute(kv_attn_kernel<RPL, UK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int) smem);   \
-        pib_launch(kv_attn_kernel<RPL, UK>, dim3(grid), dim3(threads), (size_t) smem, st, A);                                           \
+        if (CL > 1) pib_launch_cluster(kv_attn_kernel<RPL, UK>, dim3(grid), dim3(threads), dim3(1, (unsigned) CL, 1), (size_t) smem, st, A); \
+        else pib_launch(kv_attn_kernel<RPL, UK>, dim3(grid), dim3(threads), (size_t) smem, st, A);                                      \
     } while (0)
     if (R <= 32) KA_GO(1, 4); else if (R <= 64) KA_GO(2, 4); else if (R <= 128) KA_GO(4, 4); else if (R <= 256) KA_GO(8, 2); else if (R <= 512) KA_GO(16, 1);
     else { pib_set_error("attention: head size %d (max 512)", R); return PIB_ERR_UNSUPP; }

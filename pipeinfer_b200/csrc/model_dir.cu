@@ -14,6 +14,7 @@
 
 #include <algorithm>
 #include <memory>
+#include <thread>
 
 // ---- a small JSON reader ---------------------------------------------------------------------------------------------------------
 struct Json {
@@ -179,34 +180,48 @@ struct TensorSource {
     }
     static bool ends(const std::string & s, const char * e) { const size_t n = strlen(e); return s.size() >= n && !s.compare(s.size() - n, n, e); }
     void synth(const std::string & name, std::initializer_list<int64_t> shape, std::vector<float> & out) {
-        uint64_t h = seed * 0x9E3779B97F4A7C15ull + 0x1234567;
-        for (char ch : name) h = (h ^ (uint8_t) ch) * 0x100000001B3ull;
-        auto next = [&]() { h ^= h << 13; h ^= h >> 7; h ^= h << 17; return (float) ((h >> 11) & 0xFFFFFF) / 16777216.0f; };     // [0, 1)
+        uint64_t h0 = seed * 0x9E3779B97F4A7C15ull + 0x1234567;
+        for (char ch : name) h0 = (h0 ^ (uint8_t) ch) * 0x100000001B3ull;
         const int64_t last = shape.size() ? *(shape.end() - 1) : 1;
         const bool norm = ends(name, "norm") || ends(name, "norm1") || ends(name, "norm2") || ends(name, "norm1b") || ends(name, "norm2b") || ends(name, ".ls1") || ends(name, ".ls2");
         const bool norm_bias = ends(name, "norm.b") || ends(name, "norm1.b") || ends(name, "norm2.b") || ends(name, "norm1b.b") || ends(name, "norm2b.b");
         const bool around_zero = norms_around_zero && (ends(name, "norm1") || ends(name, "norm2") || name == "final.norm");
         const float amp = 1.5f * sqrtf(3.0f / (float) last);
-        for (size_t i = 0; i < out.size(); i++) {
-            const float u = next() * 2.f - 1.f;
-            float v;
-            if (around_zero || norm_bias || ends(name, ".correction")) v = 0.2f * u;
-            else if (norm) v = 1.0f + 0.2f * u;
-            else if (name.find(".mu.") != std::string::npos) v = 0.5f + 0.5f * u;
-            else if (name.find(".hc") != std::string::npos)                // hyper-connections: read about evenly, write with weights near 1, mix near the identity
-                v = ends(name, ".in") ? 1.0f / (float) last + 0.1f * u : ends(name, ".out") ? 0.8f + 0.2f * u : ((i / (size_t) last == i % (size_t) last) ? 0.9f : 0.f) + 0.1f * u;
-            else if (ends(name, "vmix")) v = 0.3f;
-            else if (ends(name, ".conv")) v = 0.5f * u + ((int64_t) (i % (size_t) last) == last - 1 ? 0.5f : 0.f);
-            else if (ends(name, "w0") || ends(name, "A_log") || ends(name, "dt_bias") || ends(name, "mix.u")) v = u;
-            else if (ends(name, "lower")) v = 0.45f + 0.45f * u;
-            else if (ends(name, ".act")) v = (i == 0 ? 0.6f : i == 1 ? 0.3f : i == 2 ? 0.2f : 0.05f);
-            else if (ends(name, "sink") || ends(name, "f.b")) v = u;
-            else if (ends(name, "canon1") || ends(name, "canon2")) v = 0.3f * u;
-            else if (ends(name, ".out") && name.find(".mix.") != std::string::npos) v = 1.0f + 0.2f * u;
-            else if (name == "embed") v = 1.7f * u;
-            else v = amp * u;
-            out[i] = __bfloat162float(__float2bfloat16_rn(v));
-        }
+        // value = centre + width * u, u uniform in [-1, 1); a few kinds have a centre that depends on the place
+        float centre = 0.f, width = amp;
+        const bool hc = name.find(".hc") != std::string::npos, hc_mix = hc && !ends(name, ".in") && !ends(name, ".out"), conv = ends(name, ".conv"), act = ends(name, ".act");
+        if (around_zero || norm_bias || ends(name, ".correction")) width = 0.2f;
+        else if (norm) { centre = 1.0f; width = 0.2f; }
+        else if (name.find(".mu.") != std::string::npos) centre = width = 0.5f;
+        else if (hc) { centre = ends(name, ".in") ? 1.0f / (float) last : ends(name, ".out") ? 0.8f : 0.f; width = ends(name, ".out") ? 0.2f : 0.1f; }      // hyper-connections: read about evenly, write with weights near 1, mix near the identity
+        else if (ends(name, "vmix")) { centre = 0.3f; width = 0.f; }
+        else if (conv) width = 0.5f;
+        else if (ends(name, "w0") || ends(name, "A_log") || ends(name, "dt_bias") || ends(name, "mix.u")) width = 1.0f;
+        else if (ends(name, "lower")) centre = width = 0.45f;
+        else if (act) width = 0.f;
+        else if (ends(name, "sink") || ends(name, "f.b")) width = 1.0f;
+        else if (ends(name, "canon1") || ends(name, "canon2")) width = 0.3f;
+        else if (ends(name, ".out") && name.find(".mix.") != std::string::npos) { centre = 1.0f; width = 0.2f; }
+        else if (name == "embed") width = 1.7f;
+        // runs of SYNTH_RUN values have a stream of their own each, so that large tensors are drawn by several threads
+        const size_t SYNTH_RUN = 1 << 18, runs = (out.size() + SYNTH_RUN - 1) / SYNTH_RUN;
+        auto draw = [&](size_t run) {
+            uint64_t h = h0 ^ (run * 0xD1342543DE82EF95ull);
+            auto next = [&]() { h ^= h << 13; h ^= h >> 7; h ^= h << 17; return (float) ((h >> 11) & 0xFFFFFF) / 16777216.0f; };     // [0, 1)
+            for (size_t i = run * SYNTH_RUN; i < std::min(out.size(), (run + 1) * SYNTH_RUN); i++) {
+                const float u = next() * 2.f - 1.f;
+                float c = centre;
+                if (hc_mix) c = i / (size_t) last == i % (size_t) last ? 0.9f : 0.f;
+                else if (conv) c = (int64_t) (i % (size_t) last) == last - 1 ? 0.5f : 0.f;
+                else if (act) c = i == 0 ? 0.6f : i == 1 ? 0.3f : i == 2 ? 0.2f : 0.05f;
+                out[i] = __bfloat162float(__float2bfloat16_rn(c + width * u));
+            }
+        };
+        const size_t n_threads = std::min<size_t>(runs, std::min(16u, std::max(1u, std::thread::hardware_concurrency())));
+        std::vector<std::thread> pool;
+        for (size_t k = 1; k < n_threads; k++) pool.emplace_back([&, k]() { for (size_t run = k; run < runs; run += n_threads) draw(run); });
+        for (size_t run = 0; run < runs; run += std::max<size_t>(1, n_threads)) draw(run);
+        for (std::thread & th : pool) th.join();
     }
 };
 
