@@ -281,11 +281,9 @@ __global__ void __launch_bounds__(128) mm_few_cols_kernel(mm_dev a) {
             for (int r = 0; r < FC_ROWS; r++) xv[r] = *reinterpret_cast<const float4 *>(x[r] + k);
 #pragma unroll
             for (int n = 0; n < NB; n++) {
-                if (n < nn) {
-                    const float4 w = *reinterpret_cast<const float4 *>(W + (size_t) n * a.ldw + k);
+                const float4 w = *reinterpret_cast<const float4 *>(W + (size_t) min(n, nn - 1) * a.ldw + k);      // no branch: the loads of a trip are in flight together
 #pragma unroll
-                    for (int r = 0; r < FC_ROWS; r++) acc[r][n] = fmaf(xv[r].w, w.w, fmaf(xv[r].z, w.z, fmaf(xv[r].y, w.y, fmaf(xv[r].x, w.x, acc[r][n]))));
-                }
+                for (int r = 0; r < FC_ROWS; r++) acc[r][n] = fmaf(xv[r].w, w.w, fmaf(xv[r].z, w.z, fmaf(xv[r].y, w.y, fmaf(xv[r].x, w.x, acc[r][n]))));
             }
         }
     } else {
@@ -295,11 +293,9 @@ __global__ void __launch_bounds__(128) mm_few_cols_kernel(mm_dev a) {
             for (int r = 0; r < FC_ROWS; r++) xv[r] = x[r][k];
 #pragma unroll
             for (int n = 0; n < NB; n++) {
-                if (n < nn) {
-                    const float w = W[(size_t) n * a.ldw + k];
+                const float w = W[(size_t) min(n, nn - 1) * a.ldw + k];
 #pragma unroll
-                    for (int r = 0; r < FC_ROWS; r++) acc[r][n] = fmaf(xv[r], w, acc[r][n]);
-                }
+                for (int r = 0; r < FC_ROWS; r++) acc[r][n] = fmaf(xv[r], w, acc[r][n]);
             }
         }
     }

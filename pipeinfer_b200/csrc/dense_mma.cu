@@ -21,49 +21,12 @@
 #include <utility>
 
 #include "hybrid.cuh"
+#include "tc_common.cuh"
 
 #define DT_BM        128
 #define DT_BK        64
 #define DT_THREADS   192
-#define DT_SPIN      (1u << 22)
 #define DT_ROWS_MAX  16
-
-__device__ __forceinline__ uint32_t dt_smem(const void * p) { return (uint32_t) __cvta_generic_to_shared(p); }
-__device__ __forceinline__ void dt_mbar_init(uint32_t bar, uint32_t count) { asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(bar), "r"(count) : "memory"); }
-__device__ __forceinline__ void dt_mbar_expect_tx(uint32_t bar, uint32_t bytes) { asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar), "r"(bytes) : "memory"); }
-// bounded: false when the phase did not complete within DT_SPIN polls or another role gave up
-__device__ __forceinline__ bool dt_mbar_wait(uint32_t bar, uint32_t parity, volatile int * abort_s) {
-    for (uint32_t it = 0; it < DT_SPIN; it++) {
-        uint32_t ok;
-        asm volatile("{\n\t.reg .pred p;\n\tmbarrier.try_wait.parity.shared::cta.b64 p, [%1], %2;\n\tselp.u32 %0, 1, 0, p;\n\t}" : "=r"(ok) : "r"(bar), "r"(parity) : "memory");
-        if (ok) return true;
-        if ((it & 63) == 63 && *abort_s) return false;
-    }
-    *abort_s = 1;
-    return false;
-}
-__device__ __forceinline__ void dt_tma_3d(uint32_t dst, const CUtensorMap * map, uint32_t bar, int x, int y, int z) {
-    asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5}], [%2];"
-                 ::"r"(dst), "l"(map), "r"(bar), "r"(x), "r"(y), "r"(z) : "memory");
-}
-// shared-memory matrix descriptor: K-major operand, 128-byte swizzle, 8-row groups 1024 bytes apart
-__device__ __forceinline__ uint64_t dt_desc(uint32_t smem_addr) {
-    uint64_t d = 0;
-    d |= (uint64_t) ((smem_addr >> 4) & 0x3fff);
-    d |= (uint64_t) 1 << 16;
-    d |= (uint64_t) (1024 >> 4) << 32;
-    d |= (uint64_t) 1 << 46;
-    d |= (uint64_t) 2 << 61;
-    return d;
-}
-__device__ __forceinline__ void dt_mma(uint32_t tmem_d, uint64_t adesc, uint64_t bdesc, uint32_t idesc, uint32_t accumulate) {
-    asm volatile("{\n\t.reg .pred p;\n\tsetp.ne.b32 p, %4, 0;\n\t"
-                 "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, {%5, %5, %5, %5}, p;\n\t}"
-                 ::"r"(tmem_d), "l"(adesc), "l"(bdesc), "r"(idesc), "r"(accumulate), "r"(0u) : "memory");
-}
-__device__ __forceinline__ void dt_commit(uint32_t bar) {
-    asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar) : "memory");
-}
 
 // ---- fp32 rows -> bfloat16 rows [Zs][M][Kp] (Kp = K rounded up to 8, the tail zero), gathered through xrows ---------------------------
 __global__ void dense_cast_kernel(const float * __restrict__ X, int64_t ldx, int64_t xz, const int32_t * __restrict__ xrows, int xdiv, int M, int K, int Kp,
@@ -235,18 +198,20 @@ static dt_scratch * dt_scratch_of(cudaStream_t st, size_t bytes) {
     return &s;
 }
 
-static int dt_map3(CUtensorMap * map, const void * base, uint64_t d0, uint64_t d1, uint64_t d2, uint64_t s1_bytes, uint64_t s2_bytes, uint32_t box1) {
+int pib_tma_map3(CUtensorMap * map, const void * base, uint64_t d0, uint64_t d1, uint64_t d2, uint64_t s1_bytes, uint64_t s2_bytes, uint32_t box1) {
     dt_encode_fn enc = dt_encode();
-    if (!enc) { pib_set_error("dense matmul: cuTensorMapEncodeTiled not available"); return PIB_ERR_UNSUPP; }
+    if (!enc) { pib_set_error("tensor map: cuTensorMapEncodeTiled not available"); return PIB_ERR_UNSUPP; }
     const cuuint64_t gdim[3] = { d0, d1, d2 };
     const cuuint64_t gstr[2] = { s1_bytes, s2_bytes };
-    const cuuint32_t box[3]  = { DT_BK, box1, 1 };
+    const cuuint32_t box[3]  = { 64, box1, 1 };
     const cuuint32_t estr[3] = { 1, 1, 1 };
     const CUresult r = enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void *>(base), gdim, gstr, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
                            CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
-    if (r != CUDA_SUCCESS) { pib_set_error("dense matmul: cuTensorMapEncodeTiled failed (%d)", (int) r); return PIB_ERR_UNSUPP; }
+    if (r != CUDA_SUCCESS) { pib_set_error("tensor map: cuTensorMapEncodeTiled failed (%d)", (int) r); return PIB_ERR_UNSUPP; }
     return PIB_OK;
 }
+
+int * pib_tc_error_word(cudaStream_t st) { dt_scratch * sc = dt_scratch_of(st, 0); return sc ? sc->err : nullptr; }
 
 template <int NB>
 static int dt_launch(const pib_mm & a, const CUtensorMap & wmap, const CUtensorMap & xmap, int x_has_z, int * err, cudaStream_t st) {
@@ -296,9 +261,9 @@ int pib_dense_mm_tc(const pib_mm & a, cudaStream_t st) {
     const int per = grouped ? (a.M + a.Z - 1) / a.Z : a.M;
     const int NB = per <= 32 ? 32 : per <= 64 ? 64 : 128;
     CUtensorMap wmap, xmap;
-    int rc = dt_map3(&wmap, a.W, (uint64_t) a.K, (uint64_t) a.N, (uint64_t) a.Z, (uint64_t) a.ldw * 2, (uint64_t) (a.Z > 1 ? a.wz : (int64_t) a.N * a.ldw) * 2, DT_BM);
-    if (rc == PIB_OK && a.x_bf16) rc = dt_map3(&xmap, a.X, (uint64_t) a.K, (uint64_t) a.M, (uint64_t) a.Z, (uint64_t) a.ldx * 2, (uint64_t) (a.Z > 1 ? a.xz : (int64_t) a.M * a.ldx) * 2, (uint32_t) NB);
-    else if (rc == PIB_OK) rc = dt_map3(&xmap, sc->xs, (uint64_t) Kp, (uint64_t) a.M, (uint64_t) Zs, (uint64_t) Kp * 2, (uint64_t) a.M * Kp * 2, (uint32_t) NB);
+    int rc = pib_tma_map3(&wmap, a.W, (uint64_t) a.K, (uint64_t) a.N, (uint64_t) a.Z, (uint64_t) a.ldw * 2, (uint64_t) (a.Z > 1 ? a.wz : (int64_t) a.N * a.ldw) * 2, DT_BM);
+    if (rc == PIB_OK && a.x_bf16) rc = pib_tma_map3(&xmap, a.X, (uint64_t) a.K, (uint64_t) a.M, (uint64_t) a.Z, (uint64_t) a.ldx * 2, (uint64_t) (a.Z > 1 ? a.xz : (int64_t) a.M * a.ldx) * 2, (uint32_t) NB);
+    else if (rc == PIB_OK) rc = pib_tma_map3(&xmap, sc->xs, (uint64_t) Kp, (uint64_t) a.M, (uint64_t) Zs, (uint64_t) Kp * 2, (uint64_t) a.M * Kp * 2, (uint32_t) NB);
     if (rc != PIB_OK) return rc;
     switch (NB) {
         case 32:  return dt_launch<32>(a, wmap, xmap, grouped ? 0 : 1, sc->err, st);

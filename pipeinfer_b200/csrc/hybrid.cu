@@ -59,14 +59,14 @@ static const char * const HK_NAMES[] = { "cellmap", "embed_ln", "canon_conv", "m
                                          "hyper_norm", "mm_mamba2_in", "mamba2_conv", "mamba2_prep", "mamba2_scan", "gated_group_norm", "mm_mamba2_o", "qkv_rope", "diff_combine",
                                          "mm_gate_up",
                                          "gated_norm", "input_conv", "mm_res_gate", "mm_attn_mem_proj", "attn_mem_prep", "memory_scan", "attn_mem_gate", "mm_attn_mem_o", "mm_gate_pair", "memory_scan_mm",
-                                         "sandwich_norm", "moe_route_sort", "norm_route", "mm_experts_up_all", "mm_experts_down_all" };
+                                         "sandwich_norm", "moe_route_sort", "norm_route", "mm_experts_up_all", "mm_experts_down_all", "flash_attention" };
 enum { HK_CELLMAP, HK_EMBED, HK_CANON, HK_DQKV, HK_LPREP, HK_UQ, HK_ABSORB, HK_LATTN, HK_UV, HK_AO, HK_QFV, HK_GATES, HK_SCAN, HK_HO, HK_LNRES, HK_UP, HK_POLY, HK_DOWN,
        HK_ROUTER, HK_ROUTE, HK_SORT, HK_EUP, HK_EDOWN, HK_SUP, HK_SDOWN, HK_COMBINE, HK_FINAL, HK_HEAD, HK_SAMPLE, HK_LATTN_MM,
        HK_EMBSCALE, HK_NORM2, HK_QKV, HK_QKVCONV, HK_APREP, HK_KVATTN, HK_KVATTN_MM, HK_SHIFT, HK_RKVG, HK_DECAY, HK_DECAYACT, HK_WKVSCAN, HK_DPREP, HK_DSCAN, HK_GHNORM, HK_GLU,
        HK_PSUM, HK_EMBPAIR, HK_PRENORM, HK_CONCAT, HK_LOOPIN, HK_SSMIN, HK_SSMCONV, HK_SSMX, HK_SSMDT, HK_SSMSCAN, HK_SSMO, HK_DUALPROJ, HK_DUALPREP, HK_DECAYSCAN, HK_DUALGATE,
        HK_DUALO, HK_HYPER, HK_M2IN, HK_M2CONV, HK_M2PREP, HK_M2SCAN, HK_GGNORM, HK_M2O, HK_QKVROPE, HK_DIFFCOMB, HK_GATEUP,
        HK_GNORM, HK_INCONV, HK_RGATE, HK_AMPROJ, HK_AMPREP, HK_MEMSCAN, HK_AMGATE, HK_AMO, HK_GATE_PAIR, HK_MEMSCAN_MM,
-       HK_SANDWICH, HK_ROUTE_SORT, HK_NORM_ROUTE, HK_EUP_ALL, HK_EDOWN_ALL, HK_COUNT };
+       HK_SANDWICH, HK_ROUTE_SORT, HK_NORM_ROUTE, HK_EUP_ALL, HK_EDOWN_ALL, HK_FLASH, HK_COUNT };
 const char * pib_hybrid_kind_name(int k) { return k >= 0 && k < HK_COUNT ? HK_NAMES[k] : "?"; }
 
 // fetch and clear the records; returns the count (the stream is synchronised)
@@ -134,9 +134,9 @@ static bool scan_split_enabled() { static const int on = getenv("PIB_SCAN_SPLIT"
 static bool chunk_scan_enabled() { static const int on = getenv("PIB_SCAN_MM") ? atoi(getenv("PIB_SCAN_MM")) : 1; return on != 0; }
 static bool attn_mm_enabled() { static const int on = getenv("PIB_ATTN_MM") ? atoi(getenv("PIB_ATTN_MM")) : 1; return on != 0; }
 
-// operands of the matmul form of an attention: key rows of `kw` (+ `kx` extra) bfloat16 each, transposed values [kw][2 NKp], query and
-// score rows
-static int grow_attn_mm(pib_context * c, size_t kw, size_t kx, int q_rows, int s_rows, int NK) {
+// operands of the matmul form of an attention: key rows of `kw` (+ `kx` extra) bfloat16 each, transposed values [kw][2 NKp], query rows of q_row bytes
+// (0: as many floats as a key row has numbers) and score rows
+static int grow_attn_mm(pib_context * c, size_t kw, size_t kx, int q_rows, int s_rows, int NK, size_t q_row = 0) {
     pib_hybrid_ctx * x = c->hy;
     const size_t R = kw, RK = kw + kx, NKp = ((size_t) NK + 7) & ~(size_t) 7, rows = (size_t) s_rows;
     auto grow = [&](void ** p, size_t * cap, size_t need) {
@@ -147,7 +147,7 @@ static int grow_attn_mm(pib_context * c, size_t kw, size_t kx, int q_rows, int s
         if (cudaMalloc(p, *cap) != cudaSuccess) { cudaGetLastError(); *p = nullptr; *cap = 0; return false; }
         return true;
     };
-    if (!grow(&x->am_kb, &x->am_kb_cap, NKp * RK * 2) || !grow(&x->am_vt, &x->am_vt_cap, R * NKp * 4) || !grow((void **) &x->am_q, &x->am_q_cap, (size_t) q_rows * RK * 4) ||
+    if (!grow(&x->am_kb, &x->am_kb_cap, NKp * RK * 2) || !grow(&x->am_vt, &x->am_vt_cap, R * NKp * 4) || !grow((void **) &x->am_q, &x->am_q_cap, (size_t) q_rows * (q_row ? q_row : RK * 4)) ||
         !grow((void **) &x->am_s, &x->am_s_cap, rows * NKp * 8) || !grow(&x->am_p, &x->am_p_cap, rows * NKp * 4)) { pib_set_error("decode: out of memory for the attention's score rows"); return PIB_ERR_NOMEM; }
     return PIB_OK;
 }
@@ -223,6 +223,7 @@ static int grow_scratch(pib_context * c, int T) {
 #define MM_ATTN_MIN_LEN 128
 #define MM_ATTN_MIN_ROW 192
 #define MM_ATTN_BLOCK   512
+#define FLASH_ATTN_BLOCK 4096     // the form that keeps its scores on chip
 // a recurrence's matmul form works through a segment in blocks of at most MM_SCAN_BLOCK tokens (its operands take a few hundred MB per block)
 #define MM_SCAN_BLOCK   2048
 struct pib_hseg { int start, len, seq, slot; bool fresh; };
@@ -340,17 +341,20 @@ static int run_layers(pib_context * c, pib_run & run, const pib_hbatch & B, cons
                pib_kv_attention(q, L, B, cache, row, x->cellmap, (int) c->n_ctx, out, any_mm ? B.mmflag : nullptr, st));
         for (const pib_hseg & g : segs) {
             if (!mm_ok || g.len < MM_ATTN_MIN_LEN) continue;
-            const int nb = (g.len + MM_ATTN_BLOCK - 1) / MM_ATTN_BLOCK, per = (g.len + nb - 1) / nb;      // blocks of equal size: none is left with a handful of rows
+            const bool flash = pib_flash_attention_fits(L);                                                 // no score rows in memory: longer blocks
+            const int block = flash ? FLASH_ATTN_BLOCK : MM_ATTN_BLOCK, nb = (g.len + block - 1) / block, per = (g.len + nb - 1) / nb;      // blocks of equal size: none is left with a handful of rows
             for (int o = 0; o < g.len; o += per) {
                 const int nq = std::min(per, g.len - o), p0 = B_pos_host[g.start + o];
                 int j0 = L.mask == PIB_MASK_CHUNK ? p0 - p0 % L.window : std::max(0, p0 - L.window + 1), n_front = 0;
                 if (L.keep > 0) { if (j0 <= L.keep) j0 = 0; else n_front = L.keep; }        // kept first positions: columns of their own in front of the window's
                 const int NK = n_front + p0 + nq - j0;
-                if ((rc = grow_attn_mm(c, (size_t) G * std::max(D, V), (size_t) 3 * G * D + V, nq * H, nq * H, NK)) != PIB_OK) return rc;
-                RC(HK_KVATTN_MM, 2.0 * nq * H * (double) NK * (D + 2.0 * V), 2.0 * NK * G * (D + 2.0 * V) + 8.0 * nq * H * (D + V) + 8.0 * nq * H * (double) NK,
-                   pib_kv_attention_mm(q, L, B, cache, row, x->cellmap + (size_t) g.slot * c->n_ctx, g.start + o, nq, j0, n_front, NK, x->am_kb, x->am_vt, x->am_q, x->am_s,
+                if ((rc = grow_attn_mm(c, (size_t) G * std::max(D, V), (size_t) 3 * G * D, nq * H, flash ? 0 : nq * H, NK, (size_t) std::max(6 * D, 4 * V))) != PIB_OK) return rc;
+                double pairs = 0;                                            // (token, key) pairs of the block, for the profile: the two products the attention is
+                for (int i = 0; i < nq; i++) pairs += L.mask == PIB_MASK_CHUNK ? (p0 + i) % L.window + 1 : std::min<int64_t>(p0 + i + 1, (int64_t) L.window + L.keep);
+                RC(flash ? HK_FLASH : HK_KVATTN_MM, 2.0 * H * pairs * (D + V), 4.0 * NK * G * (D + V) + 4.0 * nq * H * (D + V),
+                   pib_kv_attention_mm(q, L, B, cache, row, x->cellmap + (size_t) g.slot * c->n_ctx, g.start + o, nq, p0, j0, n_front, NK, x->am_kb, x->am_vt, x->am_q, x->am_s,
                                        x->am_p, out, st));
-                nk += 5;
+                nk += flash ? 2 : 5;
             }
         }
         return PIB_OK;

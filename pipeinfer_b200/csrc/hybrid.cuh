@@ -321,8 +321,11 @@ struct pib_kv_query {                // query rows [heads * maps][dim] of token 
 };
 int pib_kv_attention(const pib_kv_query & q, const pib_hlayer & L, const pib_hbatch & b, const float * cache, int cache_row, const int32_t * cellmap, int n_ctx, float * out,
                      const int32_t * skip, cudaStream_t st);
-int pib_kv_attention_mm(const pib_kv_query & q, const pib_hlayer & L, const pib_hbatch & b, const float * cache, int cache_row, const int32_t * map, int t0, int nq, int j0, int n_front, int NK,
+int pib_kv_attention_mm(const pib_kv_query & q, const pib_hlayer & L, const pib_hbatch & b, const float * cache, int cache_row, const int32_t * map, int t0, int nq, int p0, int j0, int n_front, int NK,
                         void * Kb, void * Vt, float * Qc, float * S, void * P, float * out, cudaStream_t st);
+// flash_attn.cu: the same for heads of up to 128 coordinates, scores and weights in tensor memory
+bool pib_flash_attention_fits(const pib_hlayer & L);
+int pib_flash_attention(const pib_kv_query & q, const pib_hlayer & L, int t0, int nq, int p0, int j0, int n_front, int NK, const void * Kb, const void * Vt, const void * Qc, float * out, cudaStream_t st);
 int pib_token_shift(const float * h, const float * mu, int n_mix, const pib_hbatch & b, float * state, size_t state_stride, size_t shift_off, int W, float * mixes, cudaStream_t st);
 int pib_rows_act(float * z, int ld, int n, int T, int op, const float * bias, cudaStream_t st);           // op 0: tanh; 1: exp(-exp(z + bias))
 int pib_delta_prep(float * cv, int ldc, const pib_hlayer & L, const float * proj, int ldp, int b_off, int a_off, float * bg, int T, cudaStream_t st);

@@ -252,10 +252,11 @@ int pib_kv_attention(const pib_kv_query & q, const pib_hlayer & L, const pib_hba
     const int HPB = (long long) b.T * H <= 1024 ? 1 : (H < 4 ? H : 4);
     int KS = 16 / HPB;
     if (L.window + L.keep < 64) KS = 1;
-    // few tokens over a long reach: up to 8 blocks of a cluster share a head's keys, as long as the machine has room for them
+    // few tokens over a long reach: up to 8 blocks of a cluster share a head's keys, as long as all clusters find room at once (a cluster lives in one GPC and a
+    // block of 16 warps takes most of an SM)
     const int64_t reach = std::min<int64_t>((int64_t) L.window + L.keep, n_ctx);
     int CL = 1;
-    while (HPB == 1 && KS == 16 && CL < 8 && reach >= 128 * CL && (long long) b.T * H * CL * 2 <= 2 * 148) CL *= 2;
+    while (HPB == 1 && KS == 16 && CL < 8 && reach >= 128 * CL && (long long) b.T * H * CL * 2 <= 96) CL *= 2;
     const size_t smem = (size_t) (HPB * KS + (CL > 1)) * (V + 2) * 4;
     dim3 grid((unsigned) b.T, (unsigned) ((H + HPB - 1) / HPB * CL));
     const int threads = HPB * KS * 32;
@@ -278,7 +279,8 @@ int pib_kv_attention(const pib_kv_query & q, const pib_hlayer & L, const pib_hba
 // scores [nq * rep][NK] = (scale * queries of the rep heads that share g) x keys^T, the masked softmax over each row, outputs = weights x
 // values.  Scores keep fp32 accuracy on bfloat16 tensor cores: a number enters as its bfloat16 part and the remainder of that rounding,
 // queries as rows [hi | lo | hi], keys as rows [hi | hi | lo] (3 D wide: hi.hi + lo.hi + hi.lo), and a weight enters the value matmul as
-// [hi | lo] against the values twice side by side.  These kernels prepare the operands -- keys [G][NKp][3 D], values transposed
+// [hi | lo] against the values twice side by side.  Heads of up to 128 coordinates take these operands to flash_attn.cu, which keeps scores and weights on chip; others
+// go through score rows in memory.  These kernels prepare the operands -- keys [G][NKp][3 D], values transposed
 // [G][V][2 NKp], query rows [G][nq * rep][3 D], all bfloat16 -- and put the outputs [G][nq * rep][V] back in token order.
 __device__ __forceinline__ void mk_split(float x, __nv_bfloat16 & hi, __nv_bfloat16 & lo) { hi = __float2bfloat16_rn(x); lo = __float2bfloat16_rn(x - __bfloat162float(hi)); }
 // columns [0, n_front) are positions 0 .. n_front - 1, the columns behind them positions j0, j0 + 1, ...
@@ -359,7 +361,7 @@ __global__ void __launch_bounds__(256) kv_token_order_kernel(const float * __res
         for (int i = threadIdx.x & 31; i < V; i += 32) dst[i] = gp ? src[i] * mk_sigmoid(gp[i]) : src[i];
     }
 }
-int pib_kv_attention_mm(const pib_kv_query & q, const pib_hlayer & L, const pib_hbatch & b, const float * cache, int cache_row, const int32_t * map, int t0, int nq, int j0, int n_front, int NK,
+int pib_kv_attention_mm(const pib_kv_query & q, const pib_hlayer & L, const pib_hbatch & b, const float * cache, int cache_row, const int32_t * map, int t0, int nq, int p0, int j0, int n_front, int NK,
                         void * Kb, void * Vt, float * Qc, float * S, void * P, float * out, cudaStream_t st) {
     const int maps = L.maps, H = L.heads * maps, G = L.kv_heads, GK = G * maps, D = L.dim, V = L.vdim, rep = L.heads / G, NKp = (NK + 7) & ~7, M = nq * rep;
     if (maps > 1 && L.sink) { pib_set_error("attention: a sink with several maps per head"); return PIB_ERR_UNSUPP; }
@@ -367,6 +369,7 @@ int pib_kv_attention_mm(const pib_kv_query & q, const pib_hlayer & L, const pib_
     CKL();
     pib_launch(kv_query_rows_kernel, dim3((unsigned) nq), dim3(256), (size_t) 0, st, q.q, q.ldq, (__nv_bfloat16 *) Qc, H, maps, rep, nq, D, t0, L.scale);
     CKL();
+    if (pib_flash_attention_fits(L)) return pib_flash_attention(q, L, t0, nq, p0, j0, n_front, NK, Kb, Vt, Qc, out, st);
     pib_mm a;
     a.W = Kb; a.wtype = PIB_TYPE_BF16; a.ldw = 3 * D; a.wz = (int64_t) NKp * 3 * D; a.X = Qc; a.ldx = 3 * D; a.xz = (int64_t) M * 3 * D; a.x_bf16 = 1;
     a.Y = S; a.ldy = NKp; a.yz = (int64_t) M * NKp; a.M = M; a.N = NK; a.K = 3 * D; a.Z = GK;

@@ -96,6 +96,12 @@ def medium():
                             (slopes(4, 2, 32, 24, 40, kv_from=0), moe(6, 2, 56, shared=40))], mult=0.4)
 
 
+def big_heads():
+    """heads of up to 128 coordinates, value sizes unlike them, groups of three query heads, many rows per key: the tensor-core attention's widest tiles"""
+    return model(64, 150, [(slopes(2, 1, 128, 128, 100), None), (buckets(3, 1, 96, 80, 170, 7, n=24, reach=200), dense(40)), (slopes(4, 4, 72, 40, scale=0.15), None),
+                           (buckets(12, 4, 120, 8, 64, 130, n=12, reach=90, scale=0.12), None)], mult=0.6)
+
+
 def drawn(seed):
     """a configuration drawn from a seed: every size and constant varies"""
     import numpy as np
@@ -129,4 +135,4 @@ def drawn(seed):
     return model(pick([24, 40, 53, 96, 136]), int(r.integers(30, 400)), layers, eps=pick([1e-6, 1e-5, 1e-3]), mult=float(pick([0.2, 0.5, 1.0])))
 
 
-CONFIGS = {f.__name__: f for f in (mixed_small, slope_only, bucket_only, experts_only, shared_cells, ones, far_keys, wide_heads, medium)}
+CONFIGS = {f.__name__: f for f in (mixed_small, slope_only, bucket_only, experts_only, shared_cells, ones, far_keys, wide_heads, big_heads, medium)}

@@ -389,10 +389,11 @@ def test_long_decoding(tmp_path):
     assert e.max() < TOL32
 
 
-def test_long_portions_take_the_matmul_forms(tmp_path):
+@pytest.mark.parametrize("name", ["wide_heads", "big_heads"])
+def test_long_portions_take_the_matmul_forms(tmp_path, name):
     """served mode: portions of 128 tokens and more run as tensor-core matmuls; shorter portions and decoded tokens stay with the per-token
     kernels.  Both against the oracle, against each other, and mixed in one batch"""
-    cfg = CONFIGS["wide_heads"]()
+    cfg = CONFIGS[name]()
     W = O.random_weights(cfg, 23)
     toks, other = tokens(cfg, 450, 10), tokens(cfg, 60, 11)
     ref, ref_o = oracle_logits(cfg, W, toks), oracle_logits(cfg, W, other)
