@@ -1,11 +1,12 @@
 // flash_attn.cu -- attention of long portions over cached key / value heads (served mode) with scores and weights in tensor memory.
 //
 // One block takes 128 query rows of one problem (key / value head, map): rows are (token, head of the group), the `rep` heads that share the keys next to each other.
-// It walks the key columns its tokens can see in tiles of 64 with one pass and a running maximum:
-//   warp 0       one lane brings the query rows once and every tile's keys and values by TMA (two stages)
-//   warp 1       one lane issues tcgen05.mma: scores S = Q K^T of the NEXT tile into the other half of a double buffer, then O += P V of this one
-//   warps 2..5   a thread per query row: scores from tensor memory, cap, distance bias and mask, running maximum, weights as two bfloat16 parts into shared memory
-//                (the operand of the second product); the accumulator in tensor memory is rescaled only when a maximum has grown by more than 2^FA_LAZY
+// It walks the key columns its tokens can see in tiles of 64 with one pass and running maxima:
+//   warp 0       one lane brings the query rows once and every tile's keys and values by TMA (two stages each)
+//   warp 1       one lane issues tcgen05.mma: scores S = Q K^T of a tile, then O += P V of the tile before the last
+//   warps 2..9   two groups of 128 threads, one for the even and one for the odd tiles, a thread per query row: scores from tensor memory, cap, distance bias and
+//                mask, running maximum, weights as two bfloat16 parts into shared memory (the operand of the second product).  Each group has its own accumulator
+//                in tensor memory, rescaled only when a maximum has grown by more than 2^FA_LAZY; both are merged on the way out
 // Scores keep fp32 accuracy on bfloat16 operands: queries and keys enter as their bfloat16 part and the remainder of that rounding, three products are summed
 // (hi.hi + lo.hi + hi.lo); weights enter as two parts against the bfloat16 values.  The sink is the running state's start (maximum = sink, denominator = 1).
 // The result leaves in token order, divided by the denominator and (optionally) gated.
@@ -19,7 +20,7 @@
 
 #define FA_ROWS    128
 #define FA_KEYS    64
-#define FA_THREADS 192
+#define FA_THREADS 320
 #define FA_LAZY    8.0f
 #define FA_LOG2E   1.4426950408889634f
 
@@ -38,7 +39,7 @@ __device__ __forceinline__ int fa_low(const fa_args & A, int p) { return A.mask 
 template <int NC> struct fa_cfg {                    // NC: 64-wide column chunks of a head (1 or 2)
     static constexpr int Q_TILE = FA_ROWS * 128, K_TILE = FA_KEYS * 128, V_TILE = 128 * 128, P_TILE = FA_ROWS * 128;
     static constexpr int Q_BYTES = 2 * NC * Q_TILE, K_BYTES = 2 * NC * K_TILE, STAGE = K_BYTES + V_TILE;
-    static constexpr size_t SMEM = (size_t) Q_BYTES + 2 * STAGE + 2 * P_TILE + 16 * 8 + 32 + 1024;
+    static constexpr size_t SMEM = (size_t) Q_BYTES + 2 * STAGE + 4 * P_TILE + 16 * 8 + 32 + 1024;      // weights: two parts per group; the last tiles' shared memory also carries a group's maxima and denominators
 };
 
 template <int NC>
@@ -52,11 +53,13 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap qh, const __grid_constant_
     uint8_t *  sQ  = fa_dsm + ((1024u - (dt_smem(fa_dsm) & 1023u)) & 1023u);
     uint8_t *  sKV = sQ + C::Q_BYTES;
     uint8_t *  sP  = sKV + 2 * C::STAGE;
-    uint64_t * bar = reinterpret_cast<uint64_t *>(sP + 2 * C::P_TILE);
+    uint64_t * bar = reinterpret_cast<uint64_t *>(sP + 4 * C::P_TILE);
     uint32_t * tmem_slot = reinterpret_cast<uint32_t *>(bar + 16);
     volatile int * abort_s = reinterpret_cast<volatile int *>(tmem_slot + 1);
-    const uint32_t b0 = dt_smem(bar), bar_q = b0, bar_kv = b0 + 8, bar_free = b0 + 24, bar_s = b0 + 40, bar_p = b0 + 56, bar_o = b0 + 64;
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, z = blockIdx.y, row0 = blockIdx.x * FA_ROWS, n_rows = A.nq * A.rep;
+    // barriers: queries; keys arrived / read, values arrived / read (per stage); scores ready, weights written, product done (per group)
+    const uint32_t b0 = dt_smem(bar), bar_q = b0, bar_k = b0 + 8, bar_kf = b0 + 24, bar_v = b0 + 40, bar_vf = b0 + 56, bar_s = b0 + 72, bar_p = b0 + 88, bar_o = b0 + 104;
+    // the longest rows' blocks (the portion's last tokens) start first
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, z = blockIdx.y, row0 = (gridDim.x - 1 - blockIdx.x) * FA_ROWS, n_rows = A.nq * A.rep;
     // the tiles this block's tokens see: [0, front) hold kept positions, [first, last] the window
     const int pa = A.p0 + row0 / A.rep, pb = A.p0 + min(n_rows - 1, row0 + FA_ROWS - 1) / A.rep;
     const int first = (A.n_front + fa_low(A, pa) - A.j0) / FA_KEYS, last = (A.n_front + pb - A.j0) / FA_KEYS;
@@ -67,20 +70,21 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap qh, const __grid_constant_
 
     if (threadIdx.x == 0) {
         dt_mbar_init(bar_q, 1);
-        for (int s = 0; s < 2; s++) { dt_mbar_init(bar_kv + 8 * s, 1); dt_mbar_init(bar_free + 8 * s, 1); dt_mbar_init(bar_s + 8 * s, 1); }
-        dt_mbar_init(bar_p, FA_ROWS);
-        dt_mbar_init(bar_o, 1);
+        for (int k = 0; k < 2; k++) {
+            for (uint32_t b : { bar_k, bar_kf, bar_v, bar_vf, bar_s, bar_o }) dt_mbar_init(b + 8 * k, 1);
+            dt_mbar_init(bar_p + 8 * k, FA_ROWS);
+        }
         *abort_s = 0;
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
     }
     if (warp == 1) {
-        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(dt_smem(tmem_slot)), "r"(256u) : "memory");
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(dt_smem(tmem_slot)), "r"(512u) : "memory");
         asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
     }
     dt_fence_before();
     __syncthreads();
     dt_fence_after();
-    const uint32_t tmem = *tmem_slot, tm_o = tmem + 128;          // columns: scores 0..63 and 64..127, outputs 128..255
+    const uint32_t tmem = *tmem_slot, tm_o = tmem + 128;          // columns: scores 0..63 and 64..127, outputs 128..255 and 256..383
 
     if (warp == 0) {
         if (lane == 0) {
@@ -90,15 +94,18 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap qh, const __grid_constant_
                 dt_tma_3d(dt_smem(sQ + (NC + c) * C::Q_TILE), &ql, bar_q, c * 64, row0, z);
             }
             for (int j = 0; j < n_tiles; j++) {
-                const int s = j & 1, col = tile_of(j) * FA_KEYS;
-                if (j >= 2 && !dt_mbar_wait(bar_free + 8 * s, ((j >> 1) - 1) & 1, abort_s)) break;
-                uint8_t * st = sKV + s * C::STAGE;
-                dt_mbar_expect_tx(bar_kv + 8 * s, C::K_BYTES + A.VN * 128);
+                const int k = 8 * (j & 1), col = tile_of(j) * FA_KEYS;
+                const uint32_t again = ((j >> 1) - 1) & 1;
+                uint8_t * st = sKV + (j & 1) * C::STAGE;
+                if (j >= 2 && !dt_mbar_wait(bar_kf + k, again, abort_s)) break;
+                dt_mbar_expect_tx(bar_k + k, C::K_BYTES);
                 for (int c = 0; c < NC; c++) {
-                    dt_tma_3d(dt_smem(st + c * C::K_TILE), &kh, bar_kv + 8 * s, c * 64, col, z);
-                    dt_tma_3d(dt_smem(st + (NC + c) * C::K_TILE), &kl, bar_kv + 8 * s, c * 64, col, z);
+                    dt_tma_3d(dt_smem(st + c * C::K_TILE), &kh, bar_k + k, c * 64, col, z);
+                    dt_tma_3d(dt_smem(st + (NC + c) * C::K_TILE), &kl, bar_k + k, c * 64, col, z);
                 }
-                dt_tma_3d(dt_smem(st + C::K_BYTES), &vm, bar_kv + 8 * s, col, 0, z);
+                if (j >= 2 && !dt_mbar_wait(bar_vf + k, again, abort_s)) break;
+                dt_mbar_expect_tx(bar_v + k, A.VN * 128);
+                dt_tma_3d(dt_smem(st + C::K_BYTES), &vm, bar_v + k, col, 0, z);
             }
         }
     } else if (warp == 1) {
@@ -106,7 +113,9 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap qh, const __grid_constant_
             constexpr uint32_t id_s = dt_idesc(FA_ROWS, FA_KEYS);
             const uint32_t id_o = dt_idesc(FA_ROWS, A.VN);
             const uint64_t dq = dt_desc(dt_smem(sQ)), dp = dt_desc(dt_smem(sP));
-            auto scores = [&](int j) {                             // S(j): three products over the head's columns
+            auto scores = [&](int j) {                             // S(j), once its keys are there: three products over the head's columns
+                if (!dt_mbar_wait(bar_k + 8 * (j & 1), (j >> 1) & 1, abort_s)) return false;
+                dt_fence_after();
                 const uint64_t dk = dt_desc(dt_smem(sKV + (j & 1) * C::STAGE));
                 bool acc = false;
 #pragma unroll
@@ -118,46 +127,46 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap qh, const __grid_constant_
                         for (int k = 0; k < 4; k++) { dt_mma(tmem + 64 * (j & 1), a + (c * C::Q_TILE >> 4) + 2 * k, b + (c * C::K_TILE >> 4) + 2 * k, id_s, acc); acc = true; }
                 }
                 dt_commit(bar_s + 8 * (j & 1));
+                dt_commit(bar_kf + 8 * (j & 1));
+                return true;
             };
-            bool ok = dt_mbar_wait(bar_q, 0, abort_s) && dt_mbar_wait(bar_kv, 0, abort_s);
-            if (ok) { dt_fence_after(); scores(0); }
+            bool ok = dt_mbar_wait(bar_q, 0, abort_s) && scores(0) && (n_tiles < 2 || scores(1));
             for (int j = 0; j < n_tiles && ok; j++) {
-                if (j + 1 < n_tiles) {                             // its half of the score buffer was read before the weights of tile j - 1 arrived
-                    ok = dt_mbar_wait(bar_kv + 8 * ((j + 1) & 1), ((j + 1) >> 1) & 1, abort_s);
-                    if (!ok) break;
-                    dt_fence_after();
-                    scores(j + 1);
-                }
-                ok = dt_mbar_wait(bar_p, j & 1, abort_s);
+                ok = dt_mbar_wait(bar_p + 8 * (j & 1), (j >> 1) & 1, abort_s);       // the group has read its scores, too: their columns are free
+                if (!ok) break;
+                if (j + 2 < n_tiles && !(ok = scores(j + 2))) break;
+                ok = dt_mbar_wait(bar_v + 8 * (j & 1), (j >> 1) & 1, abort_s);
                 if (!ok) break;
                 dt_fence_after();
-                const uint64_t dv = dt_desc(dt_smem(sKV + (j & 1) * C::STAGE + C::K_BYTES));
+                const uint64_t dv = dt_desc(dt_smem(sKV + (j & 1) * C::STAGE + C::K_BYTES)), dw = dp + ((j & 1) * 2 * C::P_TILE >> 4);
 #pragma unroll
                 for (int part = 0; part < 2; part++)
 #pragma unroll
-                    for (int k = 0; k < 4; k++) dt_mma(tm_o, dp + (part * C::P_TILE >> 4) + 2 * k, dv + 2 * k, id_o, (j | part | k) != 0);
-                dt_commit(bar_o);
-                dt_commit(bar_free + 8 * (j & 1));
+                    for (int k = 0; k < 4; k++) dt_mma(tm_o + 128 * (j & 1), dw + (part * C::P_TILE >> 4) + 2 * k, dv + 2 * k, id_o, (j > 1) | ((part | k) != 0));
+                dt_commit(bar_o + 8 * (j & 1));
+                dt_commit(bar_vf + 8 * (j & 1));
             }
         }
     } else {
-        const int q4 = warp & 3, rt = q4 * 32 + lane, R = row0 + rt, Rc = min(R, n_rows - 1);
+        const int w = (warp - 2) >> 2, q4 = warp & 3, rt = q4 * 32 + lane, R = row0 + rt, Rc = min(R, n_rows - 1);
         const int p = A.p0 + Rc / A.rep, h = (z / A.maps * A.rep + Rc % A.rep) * A.maps + z % A.maps;
         const int pmin = A.p0 + min(n_rows - 1, row0 + q4 * 32) / A.rep, pmax = A.p0 + min(n_rows - 1, row0 + q4 * 32 + 31) / A.rep;      // of this warp's rows
         const uint32_t lane_off = (uint32_t) (q4 * 32) << 16;
         const float slope2 = A.slopes ? A.slopes[h] * FA_LOG2E : 0.f;
         const float * rel = A.rel ? A.rel + (size_t) h * A.n_rel : nullptr;
-        float m = A.sink ? A.sink[h] * FA_LOG2E : -INFINITY, l = A.sink ? 1.f : 0.f;                                                     // maximum in units of log2
-        uint8_t * prow = sP + (rt >> 3) * 1024 + (rt & 7) * 128;
+        const bool sunk = A.sink && w == 0;                                                                                              // the sink counts once
+        float m = sunk ? A.sink[h] * FA_LOG2E : -INFINITY, l = sunk ? 1.f : 0.f;                                                         // maximum in units of log2
+        const uint32_t tm_s = tmem + lane_off + 64 * w, tm_w = tm_o + lane_off + 128 * w;
+        uint8_t * prow = sP + w * 2 * C::P_TILE + (rt >> 3) * 1024 + (rt & 7) * 128;
         bool ok = true;
-        for (int j = 0; j < n_tiles; j++) {
+        for (int j = w; j < n_tiles; j += 2) {
             const int c0 = tile_of(j) * FA_KEYS, xb = A.j0 + c0 - A.n_front;       // column c0 + i holds position xb + i (i when it is a kept column in front)
-            ok = dt_mbar_wait(bar_s + 8 * (j & 1), (j >> 1) & 1, abort_s);
+            ok = dt_mbar_wait(bar_s + 8 * w, (j >> 1) & 1, abort_s);
             if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
             dt_fence_after();
             float t[FA_KEYS];
-            dt_ld32(tmem + lane_off + 64 * (j & 1), reinterpret_cast<uint32_t *>(t));
-            dt_ld32(tmem + lane_off + 64 * (j & 1) + 32, reinterpret_cast<uint32_t *>(t) + 32);
+            dt_ld32(tm_s, reinterpret_cast<uint32_t *>(t));
+            dt_ld32(tm_s + 32, reinterpret_cast<uint32_t *>(t) + 32);
             dt_wait_ld();
             if (A.softcap > 0.f) {
                 const float ic = 1.0f / A.softcap;
@@ -208,57 +217,74 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap qh, const __grid_constant_
             float f = 1.f;
             if (grow) { f = fa_exp2(m - mt); m = mt; l *= f; }
             const float ms = m == -INFINITY ? 0.f : m;
-            uint32_t hi[FA_KEYS / 2], lo2[FA_KEYS / 2];
-#pragma unroll
-            for (int i = 0; i < FA_KEYS; i += 2) {
-                const float a = fa_exp2(t[i] - ms), b = fa_exp2(t[i + 1] - ms);
-                l += a + b;
-                const __nv_bfloat162 h2 = __floats2bfloat162_rn(a, b);
-                const uint32_t hb = *reinterpret_cast<const uint32_t *>(&h2);
-                const __nv_bfloat162 r2 = __floats2bfloat162_rn(a - __uint_as_float(hb << 16), b - __uint_as_float(hb & 0xffff0000u));
-                hi[i / 2] = hb;
-                lo2[i / 2] = *reinterpret_cast<const uint32_t *>(&r2);
-            }
-            if (j > 0) {                                             // the product before has read its weights and left the accumulator
-                ok = dt_mbar_wait(bar_o, (j - 1) & 1, abort_s);
+            if (j > 1) {                                             // the group's product before has read its weights and left the accumulator
+                ok = dt_mbar_wait(bar_o + 8 * w, ((j >> 1) - 1) & 1, abort_s);
                 if (!__all_sync(0xffffffffu, ok)) { ok = false; break; }
                 if (rescale) {
                     dt_fence_after();
                     for (int c = 0; c < A.VN; c += 32) {
                         uint32_t v[32];
-                        dt_ld32(tm_o + lane_off + c, v);
+                        dt_ld32(tm_w + c, v);
                         dt_wait_ld();
 #pragma unroll
                         for (int i = 0; i < 32; i++) v[i] = __float_as_uint(__uint_as_float(v[i]) * f);
-                        dt_st32(tm_o + lane_off + c, v);
+                        dt_st32(tm_w + c, v);
                     }
                     dt_wait_st();
                 }
             }
+            float l2 = 0.f;
 #pragma unroll
             for (int c = 0; c < 8; c++) {                            // 16-byte pieces, swizzled as the descriptor expects them
+                uint32_t hi[4], lo4[4];
+#pragma unroll
+                for (int i = 0; i < 4; i++) {
+                    const float a = fa_exp2(t[8 * c + 2 * i] - ms), b = fa_exp2(t[8 * c + 2 * i + 1] - ms);
+                    l += a; l2 += b;
+                    const __nv_bfloat162 h2 = __floats2bfloat162_rn(a, b);
+                    hi[i] = *reinterpret_cast<const uint32_t *>(&h2);
+                    const __nv_bfloat162 r2 = __floats2bfloat162_rn(a - __uint_as_float(hi[i] << 16), b - __uint_as_float(hi[i] & 0xffff0000u));
+                    lo4[i] = *reinterpret_cast<const uint32_t *>(&r2);
+                }
                 const int off = (c ^ (rt & 7)) * 16;
-                *reinterpret_cast<uint4 *>(prow + off) = make_uint4(hi[4 * c], hi[4 * c + 1], hi[4 * c + 2], hi[4 * c + 3]);
-                *reinterpret_cast<uint4 *>(prow + C::P_TILE + off) = make_uint4(lo2[4 * c], lo2[4 * c + 1], lo2[4 * c + 2], lo2[4 * c + 3]);
+                *reinterpret_cast<uint4 *>(prow + off) = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+                *reinterpret_cast<uint4 *>(prow + C::P_TILE + off) = make_uint4(lo4[0], lo4[1], lo4[2], lo4[3]);
             }
+            l += l2;
             asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
             dt_fence_before();
-            dt_arrive(bar_p);
+            dt_arrive(bar_p + 8 * w);
         }
-        if (ok) ok = dt_mbar_wait(bar_o, (n_tiles - 1) & 1, abort_s);
-        if (__all_sync(0xffffffffu, ok)) {
+        // both groups' products are done; maxima and denominators cross through shared memory (the weights' place), then each group writes half of the columns
+        const int mine = (n_tiles - 1 - w) >> 1;                     // index of the group's last tile among its own (none: -1)
+        if (ok && n_tiles > w) ok = dt_mbar_wait(bar_o + 8 * w, mine & 1, abort_s);
+        ok = __all_sync(0xffffffffu, ok);
+        asm volatile("bar.sync 1, 256;" ::: "memory");
+        float2 * ml = reinterpret_cast<float2 *>(sP);
+        ml[w * FA_ROWS + rt] = make_float2(m, l);
+        asm volatile("bar.sync 1, 256;" ::: "memory");
+        if (ok && !*abort_s) {
             dt_fence_after();
-            const float inv = 1.0f / l;
+            const float2 o = ml[(1 - w) * FA_ROWS + rt];
+            const float  M = fmaxf(m, o.x), fm = m == -INFINITY ? 0.f : fa_exp2(m - M), fo = o.x == -INFINITY ? 0.f : fa_exp2(o.x - M), inv = 1.0f / (l * fm + o.y * fo);
+            const float  f0 = (w == 0 ? fm : fo) * inv, f1 = (w == 0 ? fo : fm) * inv;
             const size_t t_row = (size_t) (A.t0 + Rc / A.rep);
             float * op = A.out + (t_row * A.H + h) * A.V;
             const float * gp = A.gate ? A.gate + t_row * A.ldg + (size_t) h * A.V : nullptr;
-            for (int c = 0; c < A.VN; c += 32) {
+            for (int c = 32 * w; c < A.VN; c += 64) {
                 float v[32];
                 dt_ld32(tm_o + lane_off + c, reinterpret_cast<uint32_t *>(v));
                 dt_wait_ld();
-                if (R >= n_rows) continue;
 #pragma unroll
-                for (int i = 0; i < 32; i++) v[i] *= inv;
+                for (int i = 0; i < 32; i++) v[i] *= f0;
+                if (n_tiles > 1) {
+                    float u[32];
+                    dt_ld32(tm_o + lane_off + 128 + c, reinterpret_cast<uint32_t *>(u));
+                    dt_wait_ld();
+#pragma unroll
+                    for (int i = 0; i < 32; i++) v[i] = fmaf(u[i], f1, v[i]);
+                }
+                if (R >= n_rows) continue;
                 if (gp) {
 #pragma unroll
                     for (int i = 0; i < 32; i++) if (c + i < A.V) v[i] *= 1.0f / (1.0f + __expf(-gp[c + i]));
@@ -281,7 +307,7 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap qh, const __grid_constant_
         for (int i = 0; i < 2000; i++) __nanosleep(1000);
         __syncthreads();
     }
-    if (warp == 1) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(256u) : "memory");
+    if (warp == 1) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(512u) : "memory");
 }
 
 bool pib_flash_attention_fits(const pib_hlayer & L) {
