@@ -3,7 +3,7 @@
 // More than DT_ROWS_MAX rows (prompt portions): dense_tc_kernel, tcgen05.  A CTA owns 128 weight rows x NB tokens of one problem z:
 //   warp 0       one lane streams both operands by TMA (cp.async.bulk.tensor.3d, 128-byte swizzle): the weight tile [128 n][64 k] and
 //                the activation tile [NB m][64 k] of every k-step land in one stage and complete one mbarrier
-//   warp 1       allocates tensor memory; one lane issues tcgen05.mma.cta_group::1.kind::f16 (bf16 x bf16 -> fp32, M 128, N NB, 4 x K 16 per
+//   warp 1       allocates tensor memory; an elected lane issues tcgen05.mma.cta_group::1.kind::f16 (bf16 x bf16 -> fp32, M 128, N NB, 4 x K 16 per
 //                k-step) and commits each stage back to the producer, the last one to the epilogue
 //   warps 2..5   read the accumulators (tcgen05.ld.32x32b: a lane is a weight row, a column a token) and store Y, optionally relu^2
 // The activations are fp32 in the layer buffers (a producer that can write bfloat16 rows itself passes them as they are: x_bf16);
@@ -98,22 +98,20 @@ dense_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_constant_
             }
         }
     } else if (warp == 1) {
-        // instruction descriptor: fp32 accumulators, bfloat16 x bfloat16, both operands K-major, N = NB, M = 128
-        constexpr uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t) (NB >> 3) << 17) | ((uint32_t) (DT_BM >> 4) << 24);
-        if (lane == 0) {
-            bool ok = true;
-            for (int kt = 0; kt < n_ksteps && ok; kt++) {
-                const int s = kt % C::STAGES;
-                ok = dt_mbar_wait(bar_f + s * 8, (kt / C::STAGES) & 1, abort_s);
-                if (!ok) break;
-                asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-                const uint64_t ad = dt_desc(dt_smem(sA + s * C::A_BYTES)), bd = dt_desc(dt_smem(sB + s * C::B_BYTES));
+        constexpr uint32_t idesc = dt_idesc(DT_BM, NB);
+        const uint64_t ad0 = dt_desc(dt_smem(sA)), bd0 = dt_desc(dt_smem(sB));
+        bool ok = true;
+        for (int kt = 0; kt < n_ksteps && ok; kt++) {
+            const int s = kt % C::STAGES;
+            ok = __all_sync(0xffffffffu, dt_mbar_wait(bar_f + s * 8, (kt / C::STAGES) & 1, abort_s));
+            if (!ok) break;
+            dt_fence_after();
+            const uint64_t ad = ad0 + (uint64_t) (s * C::A_BYTES >> 4), bd = bd0 + (uint64_t) (s * C::B_BYTES >> 4);
 #pragma unroll
-                for (int k = 0; k < DT_BK / 16; k++) dt_mma(tmem_d, ad + 2 * k, bd + 2 * k, idesc, (kt | k) != 0);
-                dt_commit(bar_e + s * 8);
-            }
-            if (ok) dt_commit(bar_t);
+            for (int k = 0; k < DT_BK / 16; k++) dt_mma(tmem_d, ad + 2 * k, bd + 2 * k, idesc, (kt | k) != 0);
+            dt_commit(bar_e + s * 8);
         }
+        if (ok) dt_commit(bar_t);
     } else {
         const bool ok = dt_mbar_wait(bar_t, 0, abort_s);
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");

@@ -3,7 +3,7 @@
 // One block takes 128 query rows of one problem (key / value head, map): rows are (token, head of the group), the `rep` heads that share the keys next to each other.
 // It walks the key columns its tokens can see in tiles of 64 with one pass and running maxima:
 //   warp 0       one lane brings the query rows once and every tile's keys and values by TMA (two stages each)
-//   warp 1       one lane issues tcgen05.mma: scores S = Q K^T of a tile, then O += P V of the tile before the last
+//   warp 1       an elected lane issues tcgen05.mma: scores S = Q K^T of a tile, then O += P V of the tile before the last
 //   warps 2..9   two groups of 128 threads, one for the even and one for the odd tiles, a thread per query row: scores from tensor memory, cap, distance bias and
 //                mask, running maximum, weights as two bfloat16 parts into shared memory (the operand of the second product).  Each group has its own accumulator
 //                in tensor memory, rescaled only when a maximum has grown by more than 2^FA_LAZY; both are merged on the way out
@@ -93,59 +93,62 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap qh, const __grid_constant_
                 dt_tma_3d(dt_smem(sQ + c * C::Q_TILE), &qh, bar_q, c * 64, row0, z);
                 dt_tma_3d(dt_smem(sQ + (NC + c) * C::Q_TILE), &ql, bar_q, c * 64, row0, z);
             }
-            for (int j = 0; j < n_tiles; j++) {
+            auto keys = [&](int j) {
                 const int k = 8 * (j & 1), col = tile_of(j) * FA_KEYS;
-                const uint32_t again = ((j >> 1) - 1) & 1;
                 uint8_t * st = sKV + (j & 1) * C::STAGE;
-                if (j >= 2 && !dt_mbar_wait(bar_kf + k, again, abort_s)) break;
+                if (j >= 2 && !dt_mbar_wait(bar_kf + k, ((j >> 1) - 1) & 1, abort_s)) return false;
                 dt_mbar_expect_tx(bar_k + k, C::K_BYTES);
                 for (int c = 0; c < NC; c++) {
                     dt_tma_3d(dt_smem(st + c * C::K_TILE), &kh, bar_k + k, c * 64, col, z);
                     dt_tma_3d(dt_smem(st + (NC + c) * C::K_TILE), &kl, bar_k + k, c * 64, col, z);
                 }
-                if (j >= 2 && !dt_mbar_wait(bar_vf + k, again, abort_s)) break;
+                return true;
+            };
+            bool ok = keys(0);
+            for (int j = 0; j < n_tiles && ok; j++) {               // the keys run one tile ahead: their place is free as soon as the scores before are formed
+                const int k = 8 * (j & 1);
+                if (j + 1 < n_tiles && !(ok = keys(j + 1))) break;
+                if (j >= 2 && !dt_mbar_wait(bar_vf + k, ((j >> 1) - 1) & 1, abort_s)) break;
                 dt_mbar_expect_tx(bar_v + k, A.VN * 128);
-                dt_tma_3d(dt_smem(st + C::K_BYTES), &vm, bar_v + k, col, 0, z);
+                dt_tma_3d(dt_smem(sKV + (j & 1) * C::STAGE + C::K_BYTES), &vm, bar_v + k, tile_of(j) * FA_KEYS, 0, z);
             }
         }
     } else if (warp == 1) {
-        if (lane == 0) {
-            constexpr uint32_t id_s = dt_idesc(FA_ROWS, FA_KEYS);
-            const uint32_t id_o = dt_idesc(FA_ROWS, A.VN);
-            const uint64_t dq = dt_desc(dt_smem(sQ)), dp = dt_desc(dt_smem(sP));
-            auto scores = [&](int j) {                             // S(j), once its keys are there: three products over the head's columns
-                if (!dt_mbar_wait(bar_k + 8 * (j & 1), (j >> 1) & 1, abort_s)) return false;
-                dt_fence_after();
-                const uint64_t dk = dt_desc(dt_smem(sKV + (j & 1) * C::STAGE));
-                bool acc = false;
+        constexpr uint32_t id_s = dt_idesc(FA_ROWS, FA_KEYS);
+        const uint32_t id_o = dt_idesc(FA_ROWS, A.VN);
+        const uint64_t dq = dt_desc(dt_smem(sQ)), dp = dt_desc(dt_smem(sP));
+        auto scores = [&](int j) {                             // S(j), once its keys are there: three products over the head's columns
+            if (!__all_sync(0xffffffffu, dt_mbar_wait(bar_k + 8 * (j & 1), (j >> 1) & 1, abort_s))) return false;
+            dt_fence_after();
+            const uint64_t dk = dt_desc(dt_smem(sKV + (j & 1) * C::STAGE));
+            bool acc = false;
 #pragma unroll
-                for (int part = 0; part < 3; part++) {
-                    const uint64_t a = dq + (part == 1 ? (uint64_t) (NC * C::Q_TILE >> 4) : 0), b = dk + (part == 2 ? (uint64_t) (NC * C::K_TILE >> 4) : 0);
+            for (int part = 0; part < 3; part++) {
+                const uint64_t a = dq + (part == 1 ? (uint64_t) (NC * C::Q_TILE >> 4) : 0), b = dk + (part == 2 ? (uint64_t) (NC * C::K_TILE >> 4) : 0);
 #pragma unroll
-                    for (int c = 0; c < NC; c++)
+                for (int c = 0; c < NC; c++)
 #pragma unroll
-                        for (int k = 0; k < 4; k++) { dt_mma(tmem + 64 * (j & 1), a + (c * C::Q_TILE >> 4) + 2 * k, b + (c * C::K_TILE >> 4) + 2 * k, id_s, acc); acc = true; }
-                }
-                dt_commit(bar_s + 8 * (j & 1));
-                dt_commit(bar_kf + 8 * (j & 1));
-                return true;
-            };
-            bool ok = dt_mbar_wait(bar_q, 0, abort_s) && scores(0) && (n_tiles < 2 || scores(1));
-            for (int j = 0; j < n_tiles && ok; j++) {
-                ok = dt_mbar_wait(bar_p + 8 * (j & 1), (j >> 1) & 1, abort_s);       // the group has read its scores, too: their columns are free
-                if (!ok) break;
-                if (j + 2 < n_tiles && !(ok = scores(j + 2))) break;
-                ok = dt_mbar_wait(bar_v + 8 * (j & 1), (j >> 1) & 1, abort_s);
-                if (!ok) break;
-                dt_fence_after();
-                const uint64_t dv = dt_desc(dt_smem(sKV + (j & 1) * C::STAGE + C::K_BYTES)), dw = dp + ((j & 1) * 2 * C::P_TILE >> 4);
-#pragma unroll
-                for (int part = 0; part < 2; part++)
-#pragma unroll
-                    for (int k = 0; k < 4; k++) dt_mma(tm_o + 128 * (j & 1), dw + (part * C::P_TILE >> 4) + 2 * k, dv + 2 * k, id_o, (j > 1) | ((part | k) != 0));
-                dt_commit(bar_o + 8 * (j & 1));
-                dt_commit(bar_vf + 8 * (j & 1));
+                    for (int k = 0; k < 4; k++) { dt_mma(tmem + 64 * (j & 1), a + (c * C::Q_TILE >> 4) + 2 * k, b + (c * C::K_TILE >> 4) + 2 * k, id_s, acc); acc = true; }
             }
+            dt_commit(bar_s + 8 * (j & 1));
+            dt_commit(bar_kf + 8 * (j & 1));
+            return true;
+        };
+        bool ok = __all_sync(0xffffffffu, dt_mbar_wait(bar_q, 0, abort_s)) && scores(0) && (n_tiles < 2 || scores(1));
+        for (int j = 0; j < n_tiles && ok; j++) {
+            ok = __all_sync(0xffffffffu, dt_mbar_wait(bar_p + 8 * (j & 1), (j >> 1) & 1, abort_s));       // the group has read its scores, too: their columns are free
+            if (!ok) break;
+            if (j + 2 < n_tiles && !(ok = scores(j + 2))) break;
+            ok = __all_sync(0xffffffffu, dt_mbar_wait(bar_v + 8 * (j & 1), (j >> 1) & 1, abort_s));
+            if (!ok) break;
+            dt_fence_after();
+            const uint64_t dv = dt_desc(dt_smem(sKV + (j & 1) * C::STAGE + C::K_BYTES)), dw = dp + ((j & 1) * 2 * C::P_TILE >> 4);
+#pragma unroll
+            for (int part = 0; part < 2; part++)
+#pragma unroll
+                for (int k = 0; k < 4; k++) dt_mma(tm_o + 128 * (j & 1), dw + (part * C::P_TILE >> 4) + 2 * k, dv + 2 * k, id_o, (j > 1) | ((part | k) != 0));
+            dt_commit(bar_o + 8 * (j & 1));
+            dt_commit(bar_vf + 8 * (j & 1));
         }
     } else {
         const int w = (warp - 2) >> 2, q4 = warp & 3, rt = q4 * 32 + lane, R = row0 + rt, Rc = min(R, n_rows - 1);
