@@ -184,7 +184,7 @@ int pib_sandwich_norm(float * x, const pib_sublayer_y & o, const float * w, cons
     while (nv < 8 && (pieces + nv - 1) / nv > want) nv *= 2;
     int threads = ((pieces + nv - 1) / nv + 31) & ~31;
     if (threads > (nv >= 4 ? 512 : 1024)) { pib_set_error("sandwich norm: width %d not supported", W); return PIB_ERR_UNSUPP; }
-    if (route) threads = std::max(threads, nv >= 4 || route->R.E <= 16 ? 512 : 1024);      // a warp per row of the router
+    if (route) threads = std::max(threads, 512);                       // 16 warps over the router's rows
 #define SW_GO(VEC, NV) pib_launch(sandwich_norm_kernel<VEC, NV, false>, dim3((unsigned) T), dim3((unsigned) threads), (size_t) 0, st, A)
 #define SW_GO_ROUTE(NV) pib_launch(sandwich_norm_kernel<4, NV, true>, dim3((unsigned) T), dim3((unsigned) threads), sw_route_smem(T, W, route->R), st, A)
     if (route)         { if (nv == 1) SW_GO_ROUTE(1); else if (nv == 2) SW_GO_ROUTE(2); else if (nv == 4) SW_GO_ROUTE(4); else SW_GO_ROUTE(8); }
